@@ -6,7 +6,8 @@ Storage.  Layers whose mixers ask for the same `CacheSpec` form a group with
 storage of its own: a kv group owns `k`/`v` tensors
 `[layers_in_group, pages, kv_heads, PAGE_TOKENS, head_dim]` and one page list per
 slot (all layers of the group use the same page numbers); a group with a window
-gives pages back as soon as every position on them has left the window.  A state
+gives pages back as soon as every position on them has left the window (a spec may keep the
+sequence's first positions beside it: their pages stay).  A state
 layer owns a tensor `[slots + 1, *shape]`, a slot's row zeroed when the slot is
 handed out.  Page 0 of every kv group is never handed out, and neither is the last
 row of a state tensor (`null_slot`): the padding rows of a captured step point at them.
@@ -59,6 +60,7 @@ class KVLayerCache:
     block_table: torch.Tensor                   # int32 [seqs of the step, pages per sequence]
     window: Optional[int]
     writable: bool                              # False: the layer reads another layer's cache
+    keep_first: int = 0                         # first positions of a sequence that stay beside the window
 
 
 @dataclass
@@ -183,7 +185,7 @@ class SequenceCache:
 
     def advance(self, slot: int, n_new: int) -> None:
         """The step wrote `n_new` positions of `slot`.  Pages of windowed groups
-        whose every position has left the window go back to the pool."""
+        whose every position has left the window go back to the pool (those that hold kept first positions stay)."""
         self.lengths[slot] += n_new
         new_len = self.lengths[slot]
         for g in self.kv_groups:
@@ -192,7 +194,7 @@ class SequenceCache:
                 continue
             first_needed = max(0, new_len - w + 1)      # the next query (position new_len) reads from here
             pages = g.pages[slot]
-            for b in range(min(first_needed // PAGE_TOKENS, len(pages))):
+            for b in range(pages_for(g.spec.keep_first), min(first_needed // PAGE_TOKENS, len(pages))):
                 if pages[b]:
                     g.pool.give_back(pages[b])
                     pages[b] = 0

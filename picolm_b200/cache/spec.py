@@ -18,6 +18,7 @@ class CacheSpec:
     num_kv_heads: int = 0                       # kv
     head_dim: int = 0                           # kv
     window: Optional[int] = None                # kv: keep only the last `window` positions
+    keep_first: int = 0                         # kv: beside a window, keep the first positions of a sequence too
     values: bool = True                         # kv: False = one row per position that serves as key and as value
     shape: Tuple[int, ...] = ()                 # state: per-sequence shape
     dtype: str = "float32"                      # state: element type
@@ -26,16 +27,21 @@ class CacheSpec:
     private: bool = False
 
     @staticmethod
-    def kv(num_kv_heads: int, head_dim: int, window: Optional[int] = None, values: bool = True) -> "CacheSpec":
+    def kv(num_kv_heads: int, head_dim: int, window: Optional[int] = None, values: bool = True,
+           keep_first: int = 0) -> "CacheSpec":
         if num_kv_heads <= 0 or head_dim <= 0:
             raise ValueError("a kv cache needs positive num_kv_heads and head_dim")
         if window is not None and window <= 0:
             raise ValueError("a window must be positive")
-        return CacheSpec("kv", num_kv_heads=num_kv_heads, head_dim=head_dim, window=window, values=bool(values))
+        if keep_first < 0 or (keep_first and window is None):
+            raise ValueError("keep_first must not be negative, and only a window has first positions to keep")
+        return CacheSpec("kv", num_kv_heads=num_kv_heads, head_dim=head_dim, window=window, values=bool(values),
+                         keep_first=int(keep_first))
 
     @staticmethod
     def state(shape, dtype: str = "float32", private: bool = False) -> "CacheSpec":
         return CacheSpec("state", shape=tuple(int(s) for s in shape), dtype=dtype, private=bool(private))
 
     def group_key(self):
-        return (self.kind, self.num_kv_heads, self.head_dim, self.window, self.shape, self.dtype, self.values)
+        return (self.kind, self.num_kv_heads, self.head_dim, self.window, self.shape, self.dtype, self.values,
+                self.keep_first)

@@ -170,11 +170,12 @@ __device__ __forceinline__ void pv_tile_sw(float (&o)[HD / 8][4], const float (&
 // Scale, mask and fold one block of scores into the running softmax of the thread's two rows
 // (row_lo = lane/4, row_hi = lane/4 + 8).  Scores become probabilities in place.
 // key_base: position of the block's first key; pos_*: each row's own position (keys above it are
-// masked); lo_*: first key each row may see.
-template <int NKT>
+// masked); lo_*: first key of each row's window; keys before `keep` are seen whatever the window.
+// BIAS: a score also loses slope_* (in log2 units) times the distance of its key.
+template <int NKT, bool BIAS>
 __device__ __forceinline__ void softmax_block(float (&s)[NKT][4], float (&o)[HD / 8][4], float (&m)[2], float (&l)[2],
                                               float scale_log2, int key_base, int pos_lo, int pos_hi, int lo_lo,
-                                              int lo_hi, int lane) {
+                                              int lo_hi, int lane, int keep, float slope_lo, float slope_hi) {
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int j = 0; j < NKT; ++j) {
@@ -182,8 +183,10 @@ __device__ __forceinline__ void softmax_block(float (&s)[NKT][4], float (&o)[HD 
         for (int e = 0; e < 4; ++e) {
             const int key = key_base + j * 8 + (lane & 3) * 2 + (e & 1);
             const int hi = e >> 1;
-            const bool ok = hi ? (key <= pos_hi && key >= lo_hi) : (key <= pos_lo && key >= lo_lo);
-            const float v = ok ? s[j][e] * scale_log2 : -INFINITY;
+            const bool ok = hi ? (key <= pos_hi && (key >= lo_hi || key < keep)) : (key <= pos_lo && (key >= lo_lo || key < keep));
+            float raw = s[j][e] * scale_log2;
+            if (BIAS) raw = fmaf(s[j][e], scale_log2, (hi ? slope_hi : slope_lo) * (float)(key - (hi ? pos_hi : pos_lo)));
+            const float v = ok ? raw : -INFINITY;
             s[j][e] = v;
             mx[hi] = fmaxf(mx[hi], v);
         }
@@ -240,7 +243,7 @@ __global__ void __launch_bounds__(NT)
 attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const bf16* __restrict__ vc,
                     bf16* __restrict__ out, const int* __restrict__ seq_start, const int* __restrict__ seq_kv_len,
                     const int* __restrict__ block_table, int max_pages, int H, int G, float scale_log2, int window,
-                    const float* __restrict__ sink) {
+                    const float* __restrict__ sink, int keep, const float* __restrict__ slopes) {
     extern __shared__ __align__(16) uint8_t smem_raw[];
     bf16* q_s = reinterpret_cast<bf16*>(smem_raw);
     bf16* k_s = q_s + TILE_ELEMS;                     // [PF_STAGES][64][LDS]
@@ -279,11 +282,13 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, con
     const int pos_min = pos0 + row0 / R, pos_max = pos0 + last_row / R;
     const int first_key = plm_first_key(pos_min, window);
     const int page_first = first_key / PLM_PAGE, page_last = pos_max / PLM_PAGE;
-    const int n_pages = page_last - page_first + 1;
+    const int n_kept = plm_kept_pages(first_key, keep);     // pages of kept first positions in front of the window's
+    const int n_pages = n_kept + page_last - page_first + 1;
+    auto page_at = [&](int i) { return i < n_kept ? i : page_first + i - n_kept; };
 
-    auto issue = [&](int i) {                          // page i of this tile's range into stage i % PF_STAGES
-        const size_t base = ((size_t)PLM_PAGE_NO(pages[page_first + i]) * G + g) * PLM_PAGE * HD;
-        const int valid = kv_len - (page_first + i) * PLM_PAGE;
+    auto issue = [&](int i) {                          // the i-th page of this tile's walk into stage i % PF_STAGES
+        const size_t base = ((size_t)PLM_PAGE_NO(pages[page_at(i)]) * G + g) * PLM_PAGE * HD;
+        const int valid = kv_len - page_at(i) * PLM_PAGE;
         load_tile(k_s + (i % PF_STAGES) * TILE_ELEMS, kc + base, valid);
         load_tile(v_s + (i % PF_STAGES) * TILE_ELEMS, vc + base, valid);
     };
@@ -296,6 +301,11 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, con
     const int pos_hi = r_hi < rows_total ? pos0 + r_hi / R : -1;
     const int lo_lo = plm_first_key(pos_lo, window);
     const int lo_hi = plm_first_key(pos_hi, window);
+    float slope_lo = 0.f, slope_hi = 0.f;
+    if (slopes) {
+        if (r_lo < rows_total) slope_lo = slopes[g * R + r_lo % R] * LOG2E;
+        if (r_hi < rows_total) slope_hi = slopes[g * R + r_hi % R] * LOG2E;
+    }
 
     float o[HD / 8][4];
 #pragma unroll
@@ -309,7 +319,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, con
         __syncthreads();
         const bf16* kt = k_s + (i % PF_STAGES) * TILE_ELEMS;
         const bf16* vt = v_s + (i % PF_STAGES) * TILE_ELEMS;
-        const int key_base = (page_first + i) * PLM_PAGE;
+        const int key_base = page_at(i) * PLM_PAGE;
         // a warp whose rows all lie before this page has nothing to do here (causal)
         const int warp_pos_max = pos0 + min(last_row, row0 + warp * 16 + 15) / R;
         if (key_base <= warp_pos_max && row0 + warp * 16 < rows_total) {
@@ -317,7 +327,10 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, con
 #pragma unroll
             for (int j = 0; j < 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
             qk_tile<8>(s, q_s + warp * 16 * LDS, kt, 0, lane, lane & 15);
-            softmax_block<8>(s, o, m, l, scale_log2, key_base, pos_lo, pos_hi, lo_lo, lo_hi, lane);
+            if (slopes)
+                softmax_block<8, true>(s, o, m, l, scale_log2, key_base, pos_lo, pos_hi, lo_lo, lo_hi, lane, keep, slope_lo, slope_hi);
+            else
+                softmax_block<8, false>(s, o, m, l, scale_log2, key_base, pos_lo, pos_hi, lo_lo, lo_hi, lane, keep, 0.f, 0.f);
             pv_tile<8>(o, s, vt, 0, lane);
         }
         __syncthreads();                               // the stage may be overwritten by the next issue
@@ -410,7 +423,7 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, cons
                    const int* __restrict__ tok_pos, const int* __restrict__ tok_seq, const int* __restrict__ block_table,
                    int max_pages, int H, int G, float scale_log2, int window, int row_groups, const Rotary rot,
                    int q_rows, const __grid_constant__ PageMaps maps, int* __restrict__ status,
-                   const float* __restrict__ sink) {
+                   const float* __restrict__ sink, int keep, const float* __restrict__ slopes) {
     extern __shared__ __align__(16) uint8_t smem_raw[];
     const size_t q_bytes = (size_t)q_rows * LDS * sizeof(bf16);          // q_rows: 16, or 9 (8 heads and a row of zeros)
     bf16* q_s = reinterpret_cast<bf16*>(smem_raw);
@@ -441,11 +454,14 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, cons
     const int pos = PLM_POSITION(tok_pos[t]);
     const int lo = plm_first_key(pos, window);
     const int page_first = lo / PLM_PAGE, page_last = pos / PLM_PAGE;
-    const int total_pages = page_last - page_first + 1;
+    // the walk: the pages of kept first positions that lie before the window's, then the window's; a split takes `per`
+    // of them in a row, from the w_begin-th on
+    const int n_kept = plm_kept_pages(lo, keep);
+    const int total_pages = n_kept + page_last - page_first + 1;
     const int per = (total_pages + n_splits - 1) / n_splits;
-    const int p_begin = page_first + split * per;
-    const int p_end = min(page_last + 1, p_begin + per);
-    const int n_pages = p_end - p_begin;
+    const int w_begin = split * per;
+    const int n_pages = min(total_pages, w_begin + per) - w_begin;
+    auto page_at = [&](int i) { return w_begin + i < n_kept ? w_begin + i : page_first + w_begin + i - n_kept; };
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int* pages = block_table + (size_t)PLM_SEQ_NO(tok_seq[t]) * max_pages;
 
@@ -453,7 +469,7 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, cons
         if constexpr (TMA) {
             if (threadIdx.x == 0) {                     // a page's keys and values: HD / 64 boxes each, one barrier
                 const int st = i % DC_STAGES;
-                const int row0 = (PLM_PAGE_NO(pages[p_begin + i]) * G + g) * PLM_PAGE;
+                const int row0 = (PLM_PAGE_NO(pages[page_at(i)]) * G + g) * PLM_PAGE;
                 const uint32_t kd = ring + (uint32_t)(2 * st) * SW_TILE_BYTES, vd = kd + SW_TILE_BYTES;
                 plm_tc::mbar_expect_tx(full0 + 8 * st, 2 * SW_TILE_BYTES);
 #pragma unroll
@@ -463,14 +479,14 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, cons
                 }
             }
         } else {
-            const size_t base = ((size_t)PLM_PAGE_NO(pages[p_begin + i]) * G + g) * PLM_PAGE * HD;
-            const int valid = pos + 1 - (p_begin + i) * PLM_PAGE;
+            const size_t base = ((size_t)PLM_PAGE_NO(pages[page_at(i)]) * G + g) * PLM_PAGE * HD;
+            const int valid = pos + 1 - page_at(i) * PLM_PAGE;
             load_tile(k_s + (i % DC_STAGES) * TILE_ELEMS, kc + base, valid);
             load_tile(v_s + (i % DC_STAGES) * TILE_ELEMS, vc + base, valid);
         }
     };
     const int n_first = min(n_pages, DC_STAGES - 1);                    // pages asked for before the loop
-    const bool early = ROPE || n_first <= 0 || p_begin + n_first - 1 < page_last;  // none of them is written in this step
+    const bool early = ROPE || n_first <= 0 || page_at(n_first - 1) < page_last;  // none of them is written in this step
     if (!early) pdl_wait();
 #pragma unroll
     for (int i = 0; i < DC_STAGES - 1; ++i) {
@@ -513,6 +529,17 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, cons
 #pragma unroll
     for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    float slope_lo = 0.f, slope_hi = 0.f;               // of this lane's two rows (heads)
+    if (slopes) {
+        if ((lane >> 2) < n_rows) slope_lo = slopes[h0 + (lane >> 2)] * LOG2E;
+        if ((lane >> 2) + 8 < n_rows) slope_hi = slopes[h0 + (lane >> 2) + 8] * LOG2E;
+    }
+    auto fold = [&](float (&s)[2][4], int key_base) {
+        if (slopes)
+            softmax_block<2, true>(s, o, m, l, scale_log2, key_base, pos, pos, lo, lo, lane, keep, slope_lo, slope_hi);
+        else
+            softmax_block<2, false>(s, o, m, l, scale_log2, key_base, pos, pos, lo, lo, lane, keep, 0.f, 0.f);
+    };
 
     for (int i = 0; i < n_pages; ++i) {
         if (i + DC_STAGES - 1 < n_pages) issue(i + DC_STAGES - 1);
@@ -521,7 +548,7 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, cons
             // (the stage that was just asked for again was released by the barrier that ended the iteration before)
             plm_tc::mbar_wait(full0 + 8 * (i % DC_STAGES), (uint32_t)((i / DC_STAGES) & 1), status, 5);
             if (i == 0) __syncthreads();                // the query rows, written with plain stores above
-            if (p_begin + i == page_last) {
+            if (page_at(i) == page_last) {
                 // Places of the page that hold no key yet may hold whatever an earlier owner of the page left:
                 // zeros instead, so that nothing of it reaches a sum (a masked score times a stale value).
                 const int first_free = pos + (ROPE ? 0 : 1) - page_last * PLM_PAGE;     // ROPE: this step's row is written below
@@ -539,7 +566,7 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, cons
         }
         const bf16* kt = k_s + (i % DC_STAGES) * TILE_ELEMS;
         const bf16* vt = v_s + (i % DC_STAGES) * TILE_ELEMS;
-        if (ROPE && p_begin + i == page_last) {
+        if (ROPE && page_at(i) == page_last) {
             // the step's own key (rotated) and value: into this CTA's copy of the page, and from the
             // first row group into the cache as well
             constexpr int GRP = HD / 16;
@@ -579,18 +606,18 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, cons
             }
             __syncthreads();
         }
-        const int key_base = (p_begin + i) * PLM_PAGE + warp * 16;       // this warp's 16 keys of the page
+        const int key_base = page_at(i) * PLM_PAGE + warp * 16;       // this warp's 16 keys of the page
         if (key_base <= pos) {
             float s[2][4];
 #pragma unroll
             for (int j = 0; j < 2; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
             if constexpr (TMA) {
                 qk_tile_sw<2>(s, q_s, kt_sw, warp * 16, lane, min(lane & 15, q_rows - 1));
-                softmax_block<2>(s, o, m, l, scale_log2, key_base, pos, pos, lo, lo, lane);
+                fold(s, key_base);
                 pv_tile_sw<2>(o, s, vt_sw, warp * 16, lane);
             } else {
                 qk_tile<2>(s, q_s, kt, warp * 16, lane, min(lane & 15, q_rows - 1));
-                softmax_block<2>(s, o, m, l, scale_log2, key_base, pos, pos, lo, lo, lane);
+                fold(s, key_base);
                 pv_tile<2>(o, s, vt, warp * 16, lane);
             }
         }
@@ -788,9 +815,10 @@ extern "C" int plm_attn_head_dim() { return HD; }
 // max_new is the largest number of new tokens of a sequence.
 extern "C" int plm_attn_prefill(const void* q, const void* kc, const void* vc, void* out, const int* seq_start,
                                 const int* seq_kv_len, const int* block_table, int max_pages, int n_seqs, int max_new,
-                                int H, int G, float scale, int window, const float* sink, cudaStream_t stream) {
+                                int H, int G, float scale, int window, const float* sink, int keep, const float* slopes,
+                                cudaStream_t stream) {
     if (n_seqs <= 0 || max_new <= 0) return PLM_OK;
-    if (H <= 0 || G <= 0 || H % G || n_seqs > 65535 || G > 65535) return PLM_ERR_SHAPE;
+    if (H <= 0 || G <= 0 || H % G || n_seqs > 65535 || G > 65535 || keep < 0) return PLM_ERR_SHAPE;
     static bool configured = false;
     if (!configured) {
         int rc = set_smem(attn_prefill_kernel, PF_SMEM);
@@ -801,7 +829,7 @@ extern "C" int plm_attn_prefill(const void* q, const void* kc, const void* vc, v
     dim3 grid(((size_t)max_new * R + 63) / 64, G, n_seqs);
     return plm_status_of(launch_pdl(attn_prefill_kernel, grid, dim3(NT), PF_SMEM, stream, (const bf16*)q, (const bf16*)kc,
                                     (const bf16*)vc, (bf16*)out, seq_start, seq_kv_len, block_table, max_pages, H, G,
-                                    scale * LOG2E, window, sink));
+                                    scale * LOG2E, window, sink, keep, slopes));
 }
 
 // Floats of workspace that plm_attn_decode needs for (tokens, H, splits): acc then (m, l).
@@ -817,9 +845,9 @@ extern "C" long plm_attn_decode_workspace(int n_tokens, int H, int n_splits) {
 extern "C" int plm_attn_decode(const void* q, const void* kc, const void* vc, void* out, float* workspace,
                                const int* tok_pos, const int* tok_seq, const int* block_table, int max_pages,
                                int n_tokens, int H, int G, float scale, int window, int n_splits, int n_pages,
-                               int* status, const float* sink, cudaStream_t stream) {
+                               int* status, const float* sink, int keep, const float* slopes, cudaStream_t stream) {
     if (n_tokens <= 0) return PLM_OK;
-    if (H <= 0 || G <= 0 || H % G || n_splits < 1 || n_tokens > 65535) return PLM_ERR_SHAPE;
+    if (H <= 0 || G <= 0 || H % G || n_splits < 1 || n_tokens > 65535 || keep < 0) return PLM_ERR_SHAPE;
     constexpr bool TMA = HAS_TMA;
     static bool configured = false;
     if (!configured) {
@@ -845,13 +873,13 @@ extern "C" int plm_attn_decode(const void* q, const void* kc, const void* vc, vo
         return plm_status_of(launch_pdl_cluster(attn_decode_kernel<true, false, TMA>, grid, dim3(NT), dim3(n_splits, 1, 1), smem,
                                                 stream, (const bf16*)q, (const bf16*)kc, (const bf16*)vc, (bf16*)out,
                                                 (float*)nullptr, (float*)nullptr, tok_pos, tok_seq, block_table,
-                                                max_pages, H, G, scale * LOG2E, window, row_groups, Rotary{}, q_rows, maps, status, sink));
+                                                max_pages, H, G, scale * LOG2E, window, row_groups, Rotary{}, q_rows, maps, status, sink, keep, slopes));
     }
     float* ws_o = workspace;
     float* ws_ml = workspace ? workspace + (size_t)n_tokens * H * n_splits * HD : nullptr;
     int rc = plm_status_of(launch_pdl(attn_decode_kernel<false, false, TMA>, grid, dim3(NT), smem, stream, (const bf16*)q,
                                       (const bf16*)kc, (const bf16*)vc, (bf16*)out, ws_o, ws_ml, tok_pos, tok_seq,
-                                      block_table, max_pages, H, G, scale * LOG2E, window, row_groups, Rotary{}, q_rows, maps, status, sink));
+                                      block_table, max_pages, H, G, scale * LOG2E, window, row_groups, Rotary{}, q_rows, maps, status, sink, keep, slopes));
     if (rc != PLM_OK || n_splits == 1) return rc;
     return plm_status_of(launch_pdl(attn_merge_kernel, dim3(n_tokens * H), dim3(MERGE_THREADS),
                                     (size_t)(n_splits + MERGE_THREADS) * sizeof(float), stream,
@@ -893,13 +921,13 @@ extern "C" int plm_attn_decode_rope(const void* qkv, void* kc, void* vc, void* o
         return plm_status_of(launch_pdl_cluster(attn_decode_kernel<true, true, TMA>, grid, dim3(NT), dim3(n_splits, 1, 1), smem,
                                                 stream, (const bf16*)qkv, (const bf16*)kc, (const bf16*)vc, (bf16*)out,
                                                 (float*)nullptr, (float*)nullptr, tok_pos, tok_seq, block_table,
-                                                max_pages, H, G, scale * LOG2E, window, row_groups, rot, q_rows, maps, status, (const float*)nullptr));
+                                                max_pages, H, G, scale * LOG2E, window, row_groups, rot, q_rows, maps, status, (const float*)nullptr, 0, (const float*)nullptr));
     }
     float* ws_o = workspace;
     float* ws_ml = workspace ? workspace + (size_t)n_tokens * H * n_splits * HD : nullptr;
     int rc = plm_status_of(launch_pdl(attn_decode_kernel<false, true, TMA>, grid, dim3(NT), smem, stream, (const bf16*)qkv,
                                       (const bf16*)kc, (const bf16*)vc, (bf16*)out, ws_o, ws_ml, tok_pos, tok_seq,
-                                      block_table, max_pages, H, G, scale * LOG2E, window, row_groups, rot, q_rows, maps, status, (const float*)nullptr));
+                                      block_table, max_pages, H, G, scale * LOG2E, window, row_groups, rot, q_rows, maps, status, (const float*)nullptr, 0, (const float*)nullptr));
     if (rc != PLM_OK || n_splits == 1) return rc;
     return plm_status_of(launch_pdl(attn_merge_kernel, dim3(n_tokens * H), dim3(MERGE_THREADS),
                                     (size_t)(n_splits + MERGE_THREADS) * sizeof(float), stream,

@@ -6,7 +6,8 @@
 // with the running (max, sum, acc) update of the reference's `attn_core`
 // (picolm/model_attention.c:43-140; max starts at -1e30, causal by the loop
 // bound) taken 32 keys at a time.  lo = 0, or p - window + 1 for a sliding
-// window, or the start of p's chunk for a mask of chunks (plm_first_key).  Keys and values of position t of sequence b live at
+// window, or the start of p's chunk for a mask of chunks (plm_first_key); with `keep` > 0 the positions before
+// min(keep, lo) are seen too; with `slopes` [H] a score loses slopes[h] * (p - t).  Keys and values of position t of sequence b live at
 //   cache[block_table[b][t / PLM_PAGE]][g][t % PLM_PAGE][0..hd)
 // and the new tokens' own K/V are already there when this kernel runs.
 //
@@ -27,7 +28,7 @@ __global__ void __launch_bounds__(WARPS * 32)
 attention_rows_kernel(const Ta* __restrict__ q, const Tc* __restrict__ kc, const Tc* __restrict__ vc,
                       Ta* __restrict__ out, const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                       const int* __restrict__ block_table, int max_pages, int H, int G, int hd, float scale,
-                      int window, const float* __restrict__ sink) {
+                      int window, const float* __restrict__ sink, int keep, const float* __restrict__ slopes) {
     extern __shared__ float q_sm[];                 // [WARPS][hd]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x;
@@ -46,17 +47,23 @@ attention_rows_kernel(const Ta* __restrict__ q, const Tc* __restrict__ kc, const
     for (int i = 0; i < MAX_HD / 32; ++i) acc[i] = 0.f;
     float m = -1e30f, l = 0.f;
     const int lo = plm_first_key(pos, window);
+    const int n_kept = min(keep, lo);               // kept first positions in front of the window
+    const int n_keys_all = n_kept + pos - lo + 1;
+    const int skip = lo - n_kept;                   // the n-th key this row sees: n, or n + skip from n_kept on
+    const float slope = slopes ? slopes[h] : 0.f;
 
-    for (int base = lo; base <= pos; base += 32) {
-        const int key = base + lane;
+    for (int base = 0; base < n_keys_all; base += 32) {
+        const int nth = base + lane;
+        const int key = nth < n_kept ? nth : nth + skip;
         float s = -1e30f;
-        const bool valid = key <= pos;
+        const bool valid = nth < n_keys_all;
         if (valid) {
             const int page = PLM_PAGE_NO(pages[key / PLM_PAGE]);
             const Tc* kr = kc + (((size_t)page * G + g) * PLM_PAGE + key % PLM_PAGE) * hd;
             float dot = 0.f;
             for (int i = 0; i < hd; ++i) dot = fmaf(qs[i], to_f32<Tc>(kr[i]), dot);
             s = dot * scale;
+            if (slopes) s -= slope * (float)(pos - key);
         }
         const float m_new = fmaxf(m, warp_max(s));
         const float corr = expf(m - m_new);
@@ -64,10 +71,10 @@ attention_rows_kernel(const Ta* __restrict__ q, const Tc* __restrict__ kc, const
         l = l * corr + warp_sum(p);
 #pragma unroll
         for (int i = 0; i < MAX_HD / 32; ++i) acc[i] *= corr;
-        const int n_keys = min(32, pos - base + 1);
+        const int n_keys = min(32, n_keys_all - base);
         for (int j = 0; j < n_keys; ++j) {
             const float pj = __shfl_sync(0xffffffffu, p, j);
-            const int kj = base + j;
+            const int kj = base + j < n_kept ? base + j : base + j + skip;
             const int page = PLM_PAGE_NO(pages[kj / PLM_PAGE]);
             const Tc* vr = vc + (((size_t)page * G + g) * PLM_PAGE + kj % PLM_PAGE) * hd;
 #pragma unroll
@@ -102,15 +109,15 @@ attention_rows_kernel(const Ta* __restrict__ q, const Tc* __restrict__ kc, const
 extern "C" int plm_attention_rows(const void* q, const void* kc, const void* vc, void* out, int dtype,
                                   const int* tok_pos, const int* tok_seq, const int* block_table, int max_pages,
                                   int n_tokens, int H, int G, int hd, float scale, int window, const float* sink,
-                                  cudaStream_t stream) {
+                                  int keep, const float* slopes, cudaStream_t stream) {
     if (n_tokens <= 0) return PLM_OK;
-    if (H <= 0 || G <= 0 || H % G || hd <= 0 || hd > MAX_HD) return PLM_ERR_SHAPE;
+    if (H <= 0 || G <= 0 || H % G || hd <= 0 || hd > MAX_HD || keep < 0) return PLM_ERR_SHAPE;
     dim3 grid(n_tokens, (H + WARPS - 1) / WARPS);
     const size_t smem = (size_t)WARPS * hd * sizeof(float);
 #define ROWS_LAUNCH(Ta_, MAXHD_)                                                                                       \
     attention_rows_kernel<Ta_, Ta_, MAXHD_><<<grid, WARPS * 32, smem, stream>>>(                                       \
         (const Ta_*)q, (const Ta_*)kc, (const Ta_*)vc, (Ta_*)out, tok_pos, tok_seq, block_table, max_pages, H, G, hd, \
-        scale, window, sink)
+        scale, window, sink, keep, slopes)
 #define ROWS_BY_SIZE(Ta_)                          \
     do {                                           \
         if (hd <= 256) ROWS_LAUNCH(Ta_, 256);      \

@@ -20,6 +20,11 @@
 // barriers of their own.  Keys of a KV head are shared by its
 // query heads through L2 (consecutive CTAs work on the heads of one group).
 //
+// A sliding window may keep the sequence's first positions in sight: the walk then starts with their pages.  With
+// slopes (BIAS: a score loses its head's slope times the key's distance) the walk goes backwards, from the tile's own
+// page to the oldest: the scores' level falls along it, so that the reference maximum is found on the first pages and
+// O is hardly ever rescaled.
+//
 // Waits on mbarriers are bounded as in gemm_tc.cu: a wait that runs out records where in
 // `status`, the CTA stops issuing work, lets what is in flight land, frees its TMEM and returns.
 #include "tc_common.cuh"
@@ -160,12 +165,13 @@ __device__ long long plm_attn_trace[5][TRACE_PAGES][8];
 #endif
 
 // grid = (query tiles of the longest sequence, heads, sequences)
+template <bool BIAS>
 __global__ void __launch_bounds__(NUM_THREADS, 2)
 attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out,
                        const int* __restrict__ seq_start, const int* __restrict__ seq_kv_len,
                        const int* __restrict__ block_table, int max_pages, int H, int G, float scale_log2, int window,
-                       int* __restrict__ status, const float* __restrict__ sink) {
+                       int* __restrict__ status, const float* __restrict__ sink, int keep, const float* __restrict__ slopes) {
     extern __shared__ uint8_t smem_raw[];
     const uint32_t raw = smem_u32(smem_raw);
     const uint32_t base = (raw + 1023u) & ~1023u;
@@ -196,7 +202,12 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     const int pos_last = pos0 + rows - 1;
     const int first_key = plm_first_key(pos0, window);
     const int page_first = first_key / BKV, page_last = pos_last / BKV;
-    const int n_pages = page_last - page_first + 1;
+    const int n_kept = plm_kept_pages(first_key, keep);                  // pages of kept first positions before the window's
+    const int n_pages = n_kept + page_last - page_first + 1;
+    auto page_at = [&](int i) {                                          // the i-th page of the walk
+        const int w = BIAS ? n_pages - 1 - i : i;
+        return w < n_kept ? w : page_first + w - n_kept;
+    };
     const int* pages = block_table + (size_t)b * max_pages;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
 #ifdef PLM_ATTN_TRACE
@@ -238,7 +249,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             int issued_k = 0, issued_v = 0;
             for (int i = 0; i < n_pages; ++i) {
                 const int ks = i % KS, vs = i % VS;
-                const int row = (PLM_PAGE_NO(pages[page_first + i]) * G + g) * BKV;
+                const int row = (PLM_PAGE_NO(pages[page_at(i)]) * G + g) * BKV;
                 if (*(volatile int*)&s_abort) break;
                 if (!mbar_wait(k_empty0 + 8 * ks, ((i / KS) & 1) ^ 1, status, 1)) { s_abort = 1; break; }
                 mbar_expect_tx(k_full0 + 8 * ks, SPLIT_RINGS ? K_BYTES : K_BYTES + V_BYTES);
@@ -328,6 +339,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         const int r = quarter * 32 + lane;                               // this thread's query row
         const int pos = r < rows ? pos0 + r : -1;                        // -1: no such row, everything masked
         const int lo = plm_first_key(pos, window);
+        const float slope2 = BIAS ? slopes[h] * LOG2E : 0.f;             // what a key loses per position of distance, log2 units
         const uint32_t lane_bits = (uint32_t)(quarter * 32) << 16;
         // O stays in tensor memory and the MMAs accumulate into it across pages.  Probabilities are
         // taken relative to a reference maximum m_ref that is raised (and O rescaled) only when a
@@ -339,20 +351,38 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             if (!mbar_spin(s_full0 + 8 * (i % NSB), (i / NSB) & 1, status, 3)) { ok = false; break; }
             tc_fence_after();
             ATTN_TRACE(softmax_warp, i, 0);
-            const int key0 = (page_first + i) * BKV;
-            const bool need_mask = key0 + BKV - 1 > pos0 || key0 < plm_first_key(pos_last, window);
+            const int key0 = page_at(i) * BKV;
+            const bool need_mask = key0 + BKV - 1 > pos0 || (key0 < plm_first_key(pos_last, window) && key0 + BKV > keep);
             float mx = -INFINITY;
             uint32_t s0[32], s1[32];
             tc_ld32(tmem + lane_bits + TM_S + (i % NSB) * 64, s0);
             tc_ld32(tmem + lane_bits + TM_S + (i % NSB) * 64 + 32, s1);
             tc_wait_ld();
             ATTN_TRACE(softmax_warp, i, 1);
+            if (BIAS) {                                                  // scores in log2 units, the distance's share taken off
+                const uint64_t sc2 = pack2(__float_as_uint(scale_log2), __float_as_uint(scale_log2));
+                const uint64_t sl2 = pack2(__float_as_uint(slope2), __float_as_uint(slope2));
+                const float off = slope2 * (float)(key0 - pos), off_hi = slope2 * (float)(key0 + 32 - pos);
+                const uint64_t off2 = pack2(__float_as_uint(off), __float_as_uint(off));
+                const uint64_t off2h = pack2(__float_as_uint(off_hi), __float_as_uint(off_hi));
+#pragma unroll
+                for (int j = 0; j < 32; j += 2) {
+                    const uint64_t jj = pack2(__float_as_uint((float)j), __float_as_uint((float)(j + 1)));
+                    float x0, x1, y0, y1;
+                    unpack2(fma2(pack2(s0[j], s0[j + 1]), sc2, fma2(jj, sl2, off2)), x0, x1);
+                    unpack2(fma2(pack2(s1[j], s1[j + 1]), sc2, fma2(jj, sl2, off2h)), y0, y1);
+                    s0[j] = __float_as_uint(x0);
+                    s0[j + 1] = __float_as_uint(x1);
+                    s1[j] = __float_as_uint(y0);
+                    s1[j + 1] = __float_as_uint(y1);
+                }
+            }
             if (need_mask) {
 #pragma unroll
                 for (int j = 0; j < 32; ++j) {
                     const int ka = key0 + j, kc2 = key0 + 32 + j;
-                    if (ka > pos || ka < lo) s0[j] = 0xff800000u;        // -inf
-                    if (kc2 > pos || kc2 < lo) s1[j] = 0xff800000u;
+                    if (ka > pos || (ka < lo && ka >= keep)) s0[j] = 0xff800000u;        // -inf
+                    if (kc2 > pos || (kc2 < lo && kc2 >= keep)) s1[j] = 0xff800000u;
                 }
             } else if (pos < 0) {
 #pragma unroll
@@ -368,7 +398,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             }
             mx = fmaxf(fmaxf(mx, mx1), fmaxf(mx2, mx3));
             // the scale is positive, so the maximum of the scaled scores is the scaled maximum
-            const float m_cand = fmaxf(m_ref, mx * scale_log2);
+            const float m_cand = fmaxf(m_ref, BIAS ? mx : mx * scale_log2);
             const bool raise = m_cand > m_ref + RESCALE_LOG2 || (m_ref == -INFINITY && m_cand > -INFINITY);
             // P has two buffers: page i writes the one that page i - 2 used, whose P V must be done.  (Written over
             // the scores it is: S(i) was issued after P(i - 2) V(i - 2) by the same thread.)
@@ -400,8 +430,13 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
 #pragma unroll
             for (int j = 0; j < 16; ++j) {                              // p = 2^(s * scale - m_ref): half an FFMA2 and one EX2 each
                 float xa0, xa1, xc0, xc1;
-                unpack2(fma2(pack2(s0[2 * j], s0[2 * j + 1]), scale2, neg_m2), xa0, xa1);
-                unpack2(fma2(pack2(s1[2 * j], s1[2 * j + 1]), scale2, neg_m2), xc0, xc1);
+                if (BIAS) {
+                    unpack2(add2(pack2(s0[2 * j], s0[2 * j + 1]), neg_m2), xa0, xa1);
+                    unpack2(add2(pack2(s1[2 * j], s1[2 * j + 1]), neg_m2), xc0, xc1);
+                } else {
+                    unpack2(fma2(pack2(s0[2 * j], s0[2 * j + 1]), scale2, neg_m2), xa0, xa1);
+                    unpack2(fma2(pack2(s1[2 * j], s1[2 * j + 1]), scale2, neg_m2), xc0, xc1);
+                }
                 const float a0 = ex2(xa0), a1 = ex2(xa1), c0 = ex2(xc0), c1 = ex2(xc1);
                 sum2 = add2(sum2, add2(pack2(__float_as_uint(a0), __float_as_uint(a1)),
                                        pack2(__float_as_uint(c0), __float_as_uint(c1))));
@@ -496,13 +531,15 @@ extern "C" int plm_attn_tc_trace_read(void* host_out) {
 extern "C" int plm_attn_tc_prefill(const void* q, const void* kc, const void* vc, void* out, const int* seq_start,
                                    const int* seq_kv_len, const int* block_table, int max_pages, int n_pages,
                                    int n_tokens, int n_seqs, int max_new, int H, int G, float scale, int window,
-                                   int* status, const float* sink, cudaStream_t stream) {
+                                   int* status, const float* sink, int keep, const float* slopes, cudaStream_t stream) {
     if (n_seqs <= 0 || max_new <= 0 || n_tokens <= 0) return PLM_OK;
-    if (H <= 0 || G <= 0 || H % G || n_seqs > 65535 || H > 65535) return PLM_ERR_SHAPE;
+    if (H <= 0 || G <= 0 || H % G || n_seqs > 65535 || H > 65535 || keep < 0) return PLM_ERR_SHAPE;
     if ((((uintptr_t)q | (uintptr_t)kc | (uintptr_t)vc | (uintptr_t)out)) & 15) return PLM_ERR_ALIGN;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_tc_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM);
+        cudaError_t e = cudaFuncSetAttribute(attn_tc_prefill_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM);
+        if (e == cudaSuccess)
+            e = cudaFuncSetAttribute(attn_tc_prefill_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
@@ -512,6 +549,11 @@ extern "C" int plm_attn_tc_prefill(const void* q, const void* kc, const void* vc
     if ((rc = make_map(&mk, kc, (long)n_pages * G * BKV, HD, HD, BKV)) != PLM_OK) return rc;
     if ((rc = make_map(&mv, vc, (long)n_pages * G * BKV, HD, HD, BKV)) != PLM_OK) return rc;
     dim3 grid((max_new + BQ - 1) / BQ, H, n_seqs);
-    return plm_status_of(launch_pdl(attn_tc_prefill_kernel, grid, dim3(NUM_THREADS), SMEM, stream, mq, mk, mv, (bf16*)out,
-                                    seq_start, seq_kv_len, block_table, max_pages, H, G, scale * LOG2E, window, status, sink));
+    if (slopes)
+        return plm_status_of(launch_pdl(attn_tc_prefill_kernel<true>, grid, dim3(NUM_THREADS), SMEM, stream, mq, mk, mv,
+                                        (bf16*)out, seq_start, seq_kv_len, block_table, max_pages, H, G, scale * LOG2E, window,
+                                        status, sink, keep, slopes));
+    return plm_status_of(launch_pdl(attn_tc_prefill_kernel<false>, grid, dim3(NUM_THREADS), SMEM, stream, mq, mk, mv,
+                                    (bf16*)out, seq_start, seq_kv_len, block_table, max_pages, H, G, scale * LOG2E, window,
+                                    status, sink, keep, slopes));
 }

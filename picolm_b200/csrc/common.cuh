@@ -75,6 +75,14 @@ __device__ __forceinline__ int plm_first_key(int pos, int mask) {
     return 0;
 }
 
+// Beside a window's keys a query may see the first `keep` positions of its sequence.  Pages that such a query (or a
+// tile of queries whose first row's window starts at key `first`) walks: the kept positions' pages that lie before the
+// window's first page, then the window's pages up to the query's own.  plm_kept_pages is how many come first.
+__device__ __forceinline__ int plm_kept_pages(int first, int keep) {
+    const int kept = (keep + PLM_PAGE - 1) / PLM_PAGE, window_page = first / PLM_PAGE;
+    return kept < window_page ? kept : window_page;
+}
+
 // One rotary pair (picolm/tensor.c:3216-3304: x0' = x0 c - x1 s, x1' = x0 s + x1 c) with the roundings spelt
 // out (each product rounded, then the sum: what a plain implementation does), so that every kernel that
 // rotates gives the same bits whatever the compiler would fuse.

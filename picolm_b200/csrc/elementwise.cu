@@ -1291,3 +1291,185 @@ extern "C" int plm_norm_pair_shift(const float* x, const float* w_a, const float
                                             n_tokens, d, eps, stream);
     return PLM_ERR_DTYPE;
 }
+
+// --------------------------------------------------- embedding of a token and of the pair it forms with the one before
+// out[t, :] = (table[id] + pairs[row]) * scale with row = (before * mul_prev + id * mul_cur) mod buckets; a sequence's first
+// token has none before it and takes row `buckets`.  `state` [slots, stride] int32: the sequence's last token + 1, 0 for
+// a sequence that has none yet.  The block of a sequence's first token of the step reads the state and then writes the
+// sequence's last token of the step into it, so no block reads a state that is already new.
+template <typename Tw>
+__global__ void embed_pair_kernel(const int* __restrict__ tok, const Tw* __restrict__ table, const Tw* __restrict__ pairs,
+                                  int* __restrict__ state, long state_stride, const int* __restrict__ tok_seq,
+                                  const int* __restrict__ seq_start, const int* __restrict__ seq_slot, float* __restrict__ out,
+                                  int d, int vocab, long buckets, long mul_prev, long mul_cur, float scale) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    int id = tok[t];
+    if (id < 0 || id >= vocab) id = 0;   // ids are checked on the host; never read outside the table
+    const int b = PLM_SEQ_NO(tok_seq[t]);
+    const bool first = t == seq_start[b];
+    int* st = state + (long)seq_slot[b] * state_stride;
+    const long before = first ? (long)*st - 1 : (long)tok[t - 1];
+    if (first) {
+        __syncthreads();                 // everybody has read the state
+        if (threadIdx.x == 0) {
+            const int last = seq_start[b + 1] - 1;
+            *st = tok[last > t ? last : t] + 1;
+        }
+    }
+    long row = buckets;
+    if (before >= 0) {
+        row = (before * mul_prev + (long)id * mul_cur) % buckets;
+        if (row < 0) row += buckets;
+    }
+    const Tw* a = table + (size_t)id * d;
+    const Tw* p = pairs + (size_t)row * d;
+    float* o = out + (size_t)t * d;
+    if (d % 4 == 0 && (((uintptr_t)table | (uintptr_t)pairs | (uintptr_t)out) & 15) == 0) {
+        for (int i = threadIdx.x * 4; i < d; i += blockDim.x * 4) {
+            const float4 u = load4(a + i), v = load4(p + i);
+            store4(o + i, make_float4((u.x + v.x) * scale, (u.y + v.y) * scale, (u.z + v.z) * scale, (u.w + v.w) * scale));
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < d; i += blockDim.x) o[i] = (to_f32<Tw>(a[i]) + to_f32<Tw>(p[i])) * scale;
+}
+
+extern "C" int plm_embed_pair(const int* tok, const void* table, const void* pairs, int table_dtype, int* state, long state_stride,
+                              const int* tok_seq, const int* seq_start, const int* seq_slot, float* out, int n_tokens, int d,
+                              int vocab, long buckets, long mul_prev, long mul_cur, float scale, cudaStream_t stream) {
+    if (n_tokens <= 0) return PLM_OK;
+    if (d <= 0 || vocab <= 0 || buckets <= 0 || !state) return PLM_ERR_SHAPE;
+    const int nt = d >= 1024 ? 256 : 128;
+    if (table_dtype == PLM_F32)
+        return plm_status_of(launch_pdl(embed_pair_kernel<float>, n_tokens, nt, 0, stream, tok, (const float*)table,
+                                        (const float*)pairs, state, state_stride, tok_seq, seq_start, seq_slot, out, d, vocab,
+                                        buckets, mul_prev, mul_cur, scale));
+    if (table_dtype == PLM_BF16)
+        return plm_status_of(launch_pdl(embed_pair_kernel<bf16>, n_tokens, nt, 0, stream, tok, (const bf16*)table,
+                                        (const bf16*)pairs, state, state_stride, tok_seq, seq_start, seq_slot, out, d, vocab,
+                                        buckets, mul_prev, mul_cur, scale));
+    return PLM_ERR_DTYPE;
+}
+
+// ------------------------------------- two results, each behind a norm of its own, into the stream through a third norm
+// Per row: y = factor * (rms(a) w_a + rms(b) w_b), x += rms(y) w_post, out = rms(x) w_pre, rms(v) being v over its root mean
+// square: what ends a pair of mixers, their sublayer and the add, and opens the next sublayer, in one pass over the
+// row.  Rows of a multiple of 4 and at most 4 * VPT * NT columns, kept in registers; weights fp32.
+__device__ __forceinline__ float dot4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+template <typename To, int NT, int VPT>
+__global__ void __launch_bounds__(NT)
+joined_post_pre_norm_kernel(float* __restrict__ x, const float* __restrict__ a, const float* __restrict__ b,
+                            const float* __restrict__ w_a, const float* __restrict__ w_b, float factor,
+                            const float* __restrict__ w_post, const float* __restrict__ w_pre, To* __restrict__ out, int d,
+                            float eps_a, float eps_b, float eps_post, float eps_pre) {
+    __shared__ float red[66];
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t row = (size_t)blockIdx.x * d;
+    float4 va[VPT], vb[VPT];
+    float sa = 0.f, sb = 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        const int i = (threadIdx.x + k * NT) * 4;
+        if (i < d) {
+            va[k] = load4(a + row + i);
+            vb[k] = load4(b + row + i);
+            sa += dot4(va[k]);
+            sb += dot4(vb[k]);
+        }
+    }
+    const float2 sums = block_sum2<NT>(sa, sb, red);
+    const float ra = 1.0f / sqrtf(sums.x / (float)d + eps_a), rb = 1.0f / sqrtf(sums.y / (float)d + eps_b);
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        const int i = (threadIdx.x + k * NT) * 4;
+        if (i < d) {
+            const float4 wa = load4(w_a + i), wb = load4(w_b + i);
+            va[k].x = factor * (va[k].x * ra * wa.x + vb[k].x * rb * wb.x);
+            va[k].y = factor * (va[k].y * ra * wa.y + vb[k].y * rb * wb.y);
+            va[k].z = factor * (va[k].z * ra * wa.z + vb[k].z * rb * wb.z);
+            va[k].w = factor * (va[k].w * ra * wa.w + vb[k].w * rb * wb.w);
+            ss += dot4(va[k]);
+        }
+    }
+    const float r1 = 1.0f / sqrtf(block_sum<NT>(ss, red) / (float)d + eps_post);
+    ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        const int i = (threadIdx.x + k * NT) * 4;
+        if (i < d) {
+            const float4 wp = load4(w_post + i), xv = load4(x + row + i);
+            va[k] = make_float4(xv.x + va[k].x * r1 * wp.x, xv.y + va[k].y * r1 * wp.y, xv.z + va[k].z * r1 * wp.z,
+                                xv.w + va[k].w * r1 * wp.w);
+            store4(x + row + i, va[k]);
+            ss += dot4(va[k]);
+        }
+    }
+    const float r2 = 1.0f / sqrtf(block_sum<NT>(ss, red) / (float)d + eps_pre);
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        const int i = (threadIdx.x + k * NT) * 4;
+        if (i < d) {
+            const float4 wv = load4(w_pre + i);
+            store4(out + row + i, make_float4(va[k].x * r2 * wv.x, va[k].y * r2 * wv.y, va[k].z * r2 * wv.z, va[k].w * r2 * wv.w));
+        }
+    }
+}
+
+template <typename To>
+static int joined_post_pre_norm_launch(float* x, const float* a, const float* b, const float* w_a, const float* w_b, float factor,
+                                       const float* w_post, const float* w_pre, void* out, int n_rows, int d, float eps_a,
+                                       float eps_b, float eps_post, float eps_pre, cudaStream_t stream) {
+#define JPP_LAUNCH(NT_, VPT_)                                                                                              \
+    return plm_status_of(launch_pdl(joined_post_pre_norm_kernel<To, NT_, VPT_>, dim3(n_rows), dim3(NT_), 0, stream, x, a, b, w_a, \
+                                    w_b, factor, w_post, w_pre, (To*)out, d, eps_a, eps_b, eps_post, eps_pre))
+    if (d <= 4 * 256) JPP_LAUNCH(256, 1);
+    if (d <= 8 * 256) JPP_LAUNCH(256, 2);
+    if (d <= 8 * 512) JPP_LAUNCH(512, 2);
+    if (d <= 8 * 1024) JPP_LAUNCH(1024, 2);
+    JPP_LAUNCH(1024, 4);
+#undef JPP_LAUNCH
+}
+
+extern "C" int plm_joined_post_pre_norm(float* x, const float* a, const float* b, const float* w_a, const float* w_b, float factor,
+                                        const float* w_post, const float* w_pre, void* out, int out_dtype, int n_rows, int d,
+                                        float eps_a, float eps_b, float eps_post, float eps_pre, cudaStream_t stream) {
+    if (n_rows <= 0) return PLM_OK;
+    if (d <= 0 || d % 4 || d > 16 * 1024) return PLM_ERR_SHAPE;
+    if (((uintptr_t)x | (uintptr_t)a | (uintptr_t)b | (uintptr_t)w_a | (uintptr_t)w_b | (uintptr_t)w_post | (uintptr_t)w_pre |
+         (uintptr_t)out) & 15)
+        return PLM_ERR_ALIGN;
+    if (out_dtype == PLM_F32)
+        return joined_post_pre_norm_launch<float>(x, a, b, w_a, w_b, factor, w_post, w_pre, out, n_rows, d, eps_a, eps_b, eps_post,
+                                                  eps_pre, stream);
+    if (out_dtype == PLM_BF16)
+        return joined_post_pre_norm_launch<bf16>(x, a, b, w_a, w_b, factor, w_post, w_pre, out, n_rows, d, eps_a, eps_b, eps_post,
+                                                 eps_pre, stream);
+    return PLM_ERR_DTYPE;
+}
+
+// ------------------------------------------------------------------------- an activation without a gate
+// y = 0.5 x (1 + erf(x / sqrt 2)), the exact GELU
+template <typename T>
+__global__ void gelu_erf_kernel(const T* __restrict__ x, T* __restrict__ out, size_t total) {
+    pdl_launch_dependents();
+    pdl_wait();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+        const float v = to_f32<T>(x[i]);
+        out[i] = from_f32<T>(0.5f * v * (1.f + erff(v * 0.70710678118654752f)));
+    }
+}
+
+extern "C" int plm_gelu_erf(const void* x, void* out, int dtype, long total, cudaStream_t stream) {
+    if (total <= 0) return PLM_OK;
+    const long blocks = (total + 255) / 256;
+    const dim3 grid((unsigned)(blocks < 16 * PLM_SM_COUNT ? blocks : 16 * PLM_SM_COUNT));
+    if (dtype == PLM_F32)
+        return plm_status_of(launch_pdl(gelu_erf_kernel<float>, grid, dim3(256), 0, stream, (const float*)x, (float*)out, (size_t)total));
+    if (dtype == PLM_BF16)
+        return plm_status_of(launch_pdl(gelu_erf_kernel<bf16>, grid, dim3(256), 0, stream, (const bf16*)x, (bf16*)out, (size_t)total));
+    return PLM_ERR_DTYPE;
+}

@@ -206,9 +206,12 @@ extern "C" int plm_causal_conv(const void* u, int dtype, long ldu, const float* 
 //   DECAY_SIGMOID  per key channel: d[n] = exp(log_sigmoid(raw[t, h * N + n] + p0[h * N + n]) * power)
 //   DECAY_GIVEN    per key channel, worked out beforehand: d[n] = raw[t, h * N + n], float32 (plm_sigmoid_decay
 //                  makes these from the raw values where a step's tokens are walked twice)
+//   DECAY_CONST    per head: d = p0[h], the same for every token; nothing is read from raw
 #define DECAY_STEP 1
 #define DECAY_SIGMOID 2
 #define DECAY_GIVEN 3
+#define DECAY_CONST 4
+#define DECAY_PER_CHANNEL(mode) ((mode) == DECAY_SIGMOID || (mode) == DECAY_GIVEN)
 
 // What a launch of the scan kernel does with the tokens of its segment:
 //   SCAN_WHOLE  one segment per sequence: from the cache's state, writes y and the state (decode steps, short prompts)
@@ -232,6 +235,7 @@ struct ScanArgs {
     int n_seqs, H, N, P, heads_per_group;
     int seg_len, max_segs;                // tokens per segment; segments of the longest sequence
     float *seg_state, *seg_decay;         // [seq][segment][H][N][P] and [seq][segment][H][N]
+    int silu;                             // q, k and v pass SiLU as they are read
     int vec8;                             // bf16 rows may be read eight channels at a time (sizes and addresses allow it)
 };
 
@@ -243,7 +247,7 @@ struct ScanArgs {
 template <typename T, int NS, int MODE, int PASS>
 __global__ void __launch_bounds__(SCAN_THREADS, NS <= 8 ? 4 : 1) linear_scan_kernel(const ScanArgs a, int TC) {
     constexpr int ROW = NS == 4 ? 4 : NS + 4;             // padded so that a quarter warp's float4 reads hit different banks
-    constexpr bool PER_CHANNEL = MODE != DECAY_STEP;
+    constexpr bool PER_CHANNEL = DECAY_PER_CHANNEL(MODE);
     extern __shared__ __align__(16) float smem[];
     pdl_launch_dependents();
     const int ptiles = (a.P + SCAN_PTILE - 1) / SCAN_PTILE;
@@ -295,6 +299,14 @@ __global__ void __launch_bounds__(SCAN_THREADS, NS <= 8 ? 4 : 1) linear_scan_ker
     // Rows of bf16 whose channels come in eights on 16-byte boundaries are brought in eight at a time (a.vec8, checked
     // by the host); the channels beyond N, which only pad the 16 lanes' shares, are filled once.
     const bool vec8 = sizeof(T) == 2 && a.vec8;
+    const bool silu = MODE == DECAY_CONST && a.silu;      // (the other modes' callers hand rows that have passed theirs)
+    auto act8 = [&](float* f) {
+        if (silu) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) f[e] = silu_f(f[e]);
+        }
+    };
+    auto act = [&](float x) { return silu ? silu_f(x) : x; };
     if (vec8) {
         for (int idx = threadIdx.x; idx < TC * 16 * NS; idx += SCAN_THREADS) {
             const int tt = idx / (16 * NS), n = idx % (16 * NS);
@@ -317,10 +329,12 @@ __global__ void __launch_bounds__(SCAN_THREADS, NS <= 8 ? 4 : 1) linear_scan_ker
                 float f[8];
                 if (PASS != SCAN_LOCAL) {
                     load8_bf16((const bf16*)q + row * a.ldq + (long)g * N + n, f);
+                    act8(f);
                     *(float4*)(qs + at) = make_float4(f[0] * a.q_scale, f[1] * a.q_scale, f[2] * a.q_scale, f[3] * a.q_scale);
                     *(float4*)(qs + at + 4) = make_float4(f[4] * a.q_scale, f[5] * a.q_scale, f[6] * a.q_scale, f[7] * a.q_scale);
                 }
                 load8_bf16((const bf16*)k + row * a.ldk + (long)g * N + n, f);
+                act8(f);
                 *(float4*)(ks + at) = make_float4(f[0], f[1], f[2], f[3]);
                 *(float4*)(ks + at + 4) = make_float4(f[4], f[5], f[6], f[7]);
                 if (MODE == DECAY_GIVEN) {
@@ -342,8 +356,8 @@ __global__ void __launch_bounds__(SCAN_THREADS, NS <= 8 ? 4 : 1) linear_scan_ker
                 const int at = (tt * 16 + n / NS) * ROW + n % NS;
                 const long row = base + tt;
                 const bool in = n < N;
-                if (PASS != SCAN_LOCAL) qs[at] = in ? to_f32<T>(q[row * a.ldq + (long)g * N + n]) * a.q_scale : 0.f;
-                ks[at] = in ? to_f32<T>(k[row * a.ldk + (long)g * N + n]) : 0.f;
+                if (PASS != SCAN_LOCAL) qs[at] = in ? act(to_f32<T>(q[row * a.ldq + (long)g * N + n])) * a.q_scale : 0.f;
+                ks[at] = in ? act(to_f32<T>(k[row * a.ldk + (long)g * N + n])) : 0.f;
                 if (MODE == DECAY_SIGMOID)
                     ds[at] = in ? expf(log_sigmoid_f(to_f32<T>(raw[row * a.ldraw + (long)h * N + n]) + a.p0[(long)h * N + n]) * a.power) : 1.f;
                 if (MODE == DECAY_GIVEN) ds[at] = in ? ((const float*)a.raw)[row * a.ldraw + (long)h * N + n] : 1.f;
@@ -351,6 +365,11 @@ __global__ void __launch_bounds__(SCAN_THREADS, NS <= 8 ? 4 : 1) linear_scan_ker
         }
         if (!PER_CHANNEL) {
             for (int tt = threadIdx.x; tt < nt; tt += SCAN_THREADS) {
+                if (MODE == DECAY_CONST) {
+                    ds[tt] = a.p0[h];
+                    ds[TC + tt] = 1.f;
+                    continue;
+                }
                 const float dt = softplus_f(to_f32<T>(raw[(long)(base + tt) * a.ldraw + h]) + a.p0[h]);
                 ds[tt] = expf(-expf(a.p1[h]) * dt);
                 ds[TC + tt] = dt;
@@ -361,6 +380,7 @@ __global__ void __launch_bounds__(SCAN_THREADS, NS <= 8 ? 4 : 1) linear_scan_ker
                 const int tt = idx / (SCAN_PTILE / 8), c = (idx % (SCAN_PTILE / 8)) << 3;
                 float f[8];
                 load8_bf16((const bf16*)v + (long)(base + tt) * a.ldv + (long)h * P + ptile * SCAN_PTILE + c, f);
+                act8(f);
                 *(float4*)(vs + tt * SCAN_PTILE + c) = make_float4(f[0], f[1], f[2], f[3]);
                 *(float4*)(vs + tt * SCAN_PTILE + c + 4) = make_float4(f[4], f[5], f[6], f[7]);
             }
@@ -368,7 +388,7 @@ __global__ void __launch_bounds__(SCAN_THREADS, NS <= 8 ? 4 : 1) linear_scan_ker
 #pragma unroll 4
             for (int idx = threadIdx.x; idx < nt * SCAN_PTILE; idx += SCAN_THREADS) {
                 const int tt = idx / SCAN_PTILE, c = idx % SCAN_PTILE, pc = ptile * SCAN_PTILE + c;
-                vs[idx] = pc < P ? to_f32<T>(v[(long)(base + tt) * a.ldv + (long)h * P + pc]) : 0.f;
+                vs[idx] = pc < P ? act(to_f32<T>(v[(long)(base + tt) * a.ldv + (long)h * P + pc])) : 0.f;
             }
         }
         __syncthreads();
@@ -488,7 +508,7 @@ template <int NS>
 static size_t scan_smem(int mode, int* TC) {
     const int ROW = NS == 4 ? 4 : NS + 4;
     // tokens per pass: as many as fit into about 40 KB of shared memory, 16 at most
-    const long per_token = (mode != DECAY_STEP ? 3L : 2L) * 16 * ROW + SCAN_PTILE + (mode != DECAY_STEP ? 0 : 2);
+    const long per_token = (DECAY_PER_CHANNEL(mode) ? 3L : 2L) * 16 * ROW + SCAN_PTILE + (DECAY_PER_CHANNEL(mode) ? 0 : 2);
     int tc = (int)((40 * 1024 / 4 - 4) / per_token);
     tc = tc > 16 ? 16 : tc < 1 ? 1 : tc;
     *TC = tc;
@@ -519,6 +539,7 @@ static int scan_dispatch(const ScanArgs& a, int mode, cudaStream_t stream) {
 #define SCAN_NS(NS_)                                                                       \
     (mode == DECAY_SIGMOID ? scan_launch<T, NS_, DECAY_SIGMOID>(a, stream)                 \
      : mode == DECAY_GIVEN ? scan_launch<T, NS_, DECAY_GIVEN>(a, stream)                   \
+     : mode == DECAY_CONST ? scan_launch<T, NS_, DECAY_CONST>(a, stream)                   \
                            : scan_launch<T, NS_, DECAY_STEP>(a, stream))
     if (ns <= 4) e = SCAN_NS(4);
     else if (ns <= 8) e = SCAN_NS(8);
@@ -588,12 +609,13 @@ extern "C" int plm_linear_scan(const void* q, const void* k, const void* v, cons
                                float q_scale, float power, float* state, long state_stride, float* y, long ldy,
                                const int* seq_start, const int* seq_slot, int n_seqs, int H, int N, int P,
                                int heads_per_group, int seg_len, int max_segs, float* seg_state, float* seg_decay,
-                               cudaStream_t stream) {
+                               int silu, cudaStream_t stream) {
     if (n_seqs <= 0 || H <= 0 || N <= 0 || P <= 0 || heads_per_group <= 0) return PLM_ERR_SHAPE;
-    if (mode != DECAY_STEP && mode != DECAY_SIGMOID && mode != DECAY_GIVEN) return PLM_ERR_UNSUPPORTED;
+    if (mode != DECAY_STEP && mode != DECAY_SIGMOID && mode != DECAY_GIVEN && mode != DECAY_CONST) return PLM_ERR_UNSUPPORTED;
     if (mode == DECAY_STEP && !p1) return PLM_ERR_SHAPE;
     if (mode != DECAY_GIVEN && !p0) return PLM_ERR_SHAPE;
     if (N > 256) return PLM_ERR_UNSUPPORTED;
+    if (silu && mode != DECAY_CONST) return PLM_ERR_UNSUPPORTED;
     if (max_segs > 1 && (!seg_state || !seg_decay || seg_len <= 0 || max_segs > 65535)) return PLM_ERR_SHAPE;
     ScanArgs a;
     a.q = q, a.k = k, a.v = v, a.raw = raw;
@@ -606,9 +628,10 @@ extern "C" int plm_linear_scan(const void* q, const void* k, const void* v, cons
     a.n_seqs = n_seqs, a.H = H, a.N = N, a.P = P, a.heads_per_group = heads_per_group;
     a.seg_len = seg_len, a.max_segs = max_segs < 1 ? 1 : max_segs;
     a.seg_state = seg_state, a.seg_decay = seg_decay;
+    a.silu = silu;
     const auto al = [](const void* p_, long ld, int bytes) { return (uintptr_t)p_ % 16 == 0 && (ld * bytes) % 16 == 0; };
     a.vec8 = dtype == PLM_BF16 && N % 8 == 0 && P % 8 == 0 && al(q, ldq, 2) && al(k, ldk, 2) && al(v, ldv, 2) &&
-             (mode == DECAY_STEP || (mode == DECAY_GIVEN ? al(raw, ldraw, 4) : al(raw, ldraw, 2)));
+             (!DECAY_PER_CHANNEL(mode) || (mode == DECAY_GIVEN ? al(raw, ldraw, 4) : al(raw, ldraw, 2)));
     if (dtype == PLM_F32) return scan_dispatch<float>(a, mode, stream);
     if (dtype == PLM_BF16) return scan_dispatch<bf16>(a, mode, stream);
     return PLM_ERR_DTYPE;

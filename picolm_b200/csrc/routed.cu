@@ -2,7 +2,8 @@
 // expert, the experts' two products over those pairs, and the weighted sum per token.
 //
 //   scores   s_e = sigmoid(z_e), or softmax(z)_e over all router outputs, from the router's logits z (fp32); the choice is
-//            made on c_e = s_e + correction_e
+//            made on c_e = s_e + correction_e.  Or the logits themselves, s_e = z_e + correction_e (the correction is then
+//            a bias of the router): the choice goes by them and the weights are the softmax over the chosen ones alone
 //   groups   the experts form n_groups equal groups of neighbours; a group's score is the sum of its two largest
 //            c_e, or its largest; only experts of the `keep` best groups can be chosen (the others count as -inf)
 //   choice   the `top` largest c_e (the lower index on ties)
@@ -31,7 +32,7 @@ constexpr int ROUTE_WARPS = 4;
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 route_topk_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ correction, int E, int top,
                   int n_groups, int keep, float scale, int* __restrict__ ids, float* __restrict__ weights,
-                  float* __restrict__ gate, int gate_col, int T, int softmax_scores, int group_by_max, int normalize) {
+                  float* __restrict__ gate, int gate_col, int T, int score_mode, int group_by_max, int normalize) {
     extern __shared__ float route_sm[];             // per warp: s[E], c[E], group score[n_groups], group kept[n_groups]
     pdl_launch_dependents();
     pdl_wait();
@@ -43,6 +44,7 @@ route_topk_kernel(const float* __restrict__ logits, int ld, const float* __restr
     float* gs = c + E;
     float* kept = gs + n_groups;
     const float* z = logits + (size_t)t * ld;
+    const bool by_logits = score_mode == 2, softmax_scores = score_mode == 1;
     float zmax = 0.f, zden = 1.f;
     if (softmax_scores) {
         // softmax over all E outputs: the maximum, then the sum of the exponentials, each in an order E alone fixes
@@ -55,8 +57,9 @@ route_topk_kernel(const float* __restrict__ logits, int ld, const float* __restr
         zden = warp_sum(part);
     }
     for (int e = lane; e < E; e += 32) {
-        const float v = softmax_scores ? expf(z[e] - zmax) / zden : 1.0f / (1.0f + expf(-z[e]));
-        float cv = v + (correction ? correction[e] : 0.f);
+        const float bias = correction ? correction[e] : 0.f;
+        const float v = by_logits ? z[e] + bias : softmax_scores ? expf(z[e] - zmax) / zden : 1.0f / (1.0f + expf(-z[e]));
+        float cv = by_logits ? v : v + bias;
         if (!(cv == cv)) cv = -INFINITY;            // a NaN is never chosen before anything else
         s[e] = v;
         c[e] = cv;
@@ -122,8 +125,18 @@ route_topk_kernel(const float* __restrict__ logits, int ld, const float* __restr
         __syncwarp();
     }
     if (lane == 0) {
+        if (by_logits) {                            // (the first choice is the largest)
+            const float zm = weights[(size_t)t * top];
+            sum = 0.f;
+            for (int r = 0; r < top; ++r) {
+                const float wv = expf(weights[(size_t)t * top + r] - zm);
+                weights[(size_t)t * top + r] = wv;
+                sum += wv;
+            }
+            for (int r = 0; r < top; ++r) weights[(size_t)t * top + r] = weights[(size_t)t * top + r] / sum * scale;
+        }
         const float den = sum + 1e-20f;
-        for (int r = 0; r < top; ++r) {
+        for (int r = 0; r < top && !by_logits; ++r) {
             const float wv = weights[(size_t)t * top + r];
             weights[(size_t)t * top + r] = normalize ? wv / den * scale : wv * scale;
         }
@@ -611,7 +624,7 @@ extern "C" int plm_router_logits(const void* h, int h_dtype, const void* w, int 
 
 extern "C" int plm_route_topk(const float* logits, int ld, const float* correction, int E, int top, int n_groups,
                               int keep, float scale, int* ids, float* weights, float* gate, int gate_col, int n_tokens,
-                              int softmax_scores, int group_by_max, int normalize, cudaStream_t stream) {
+                              int score_mode, int group_by_max, int normalize, cudaStream_t stream) {
     if (n_tokens <= 0) return PLM_OK;
     if (E <= 0 || top <= 0 || top > E || n_groups <= 0 || E % n_groups || keep <= 0 || keep > n_groups || ld < E)
         return PLM_ERR_SHAPE;
@@ -621,7 +634,7 @@ extern "C" int plm_route_topk(const float* logits, int ld, const float* correcti
     if (smem > 48 * 1024) cudaFuncSetAttribute(route_topk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     return plm_status_of(launch_pdl(route_topk_kernel, dim3((n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32),
                                     smem, stream, logits, ld, correction, E, top, n_groups, keep, scale, ids, weights, gate,
-                                    gate_col, n_tokens, softmax_scores, group_by_max, normalize));
+                                    gate_col, n_tokens, score_mode, group_by_max, normalize));
 }
 
 // The most tiles of `bm` rows that `n_entries` pairs over `n_experts` experts can fill: every tile holds at least

@@ -46,7 +46,10 @@ class Engine:
         self.vocab_size = spec.vocab_size
         # Decode steps replay a CUDA graph when every part of every block says that its forward only
         # launches work that depends on the step through device buffers (`graph_safe`).
-        safe = all(getattr(part, "graph_safe", False) for b in model.blocks for _, part in b.parts())
+        parts = [part for b in model.blocks for _, part in b.parts()]
+        if hasattr(model.embedding, "cache_specs"):
+            parts.append(model.embedding)                    # an embedding that keeps something reads the step like a mixer
+        safe = all(getattr(part, "graph_safe", False) for part in parts)
         self.use_graphs = safe if use_graphs is None else (use_graphs and safe)
         from ..ops import _lib
         if _lib.CHECKED or _lib.TRACED:
@@ -59,7 +62,7 @@ class Engine:
         # float32 runs launch them kernel by kernel (their kernels take longer than the launches)
         import os
         self.prompt_graphs = (os.environ.get("PICOLM_B200_PROMPT_GRAPHS", "1") != "0" and self.runtime.dtype == torch.bfloat16 and
-                              all(getattr(part, "graph_safe_prompts", False) for b in model.blocks for _, part in b.parts()))
+                              all(getattr(part, "graph_safe_prompts", False) for part in parts))
         # one id per live sequence, and never fewer than the largest captured batch size (its padding rows read it)
         from .decode_graph import BUCKETS
         self._tokens = torch.zeros(max(BUCKETS[-1], self.cache.max_seqs), dtype=torch.int32,

@@ -45,6 +45,7 @@ class Model:
         self.run_input = build_part("run_input", spec.run_input, runtime) if spec.run_input is not None else None
         self._run_inputs = {run: (index, bool(first)) for run, index, first in spec.run_input_at}
         self.loaded = False
+        self._embedding_caches: List[Tuple[int, bool]] = []       # (cache number, may write it), numbered by `cache_specs`
         # Called as layer_hook(run, layer, done) before (done False) and after (done True) every scheduled layer
         # of a step: the reference's per-layer benchmark callback (bench_layer_cb_t, picolm/model.h:528-533,
         # fired around each layer in picolm/model_core.c:235-252).  While it is set, steps are not replayed
@@ -133,7 +134,10 @@ class Model:
                 else:
                     entries.append((lent.pop(0), False))
             self._run_caches.append(entries)
-        return out
+        # what the embedding keeps (the token before, for one that looks at pairs)
+        own = list(self.embedding.cache_specs()) if hasattr(self.embedding, "cache_specs") else []
+        self._embedding_caches = [(len(out) + n, True) for n in range(len(own))]
+        return out + own
 
     def prepare(self, max_seq_tokens: int) -> None:
         for block in self.blocks:
@@ -142,13 +146,18 @@ class Model:
     def layer_caches(self, run: int, cache: SequenceCache, step) -> list:
         """What the parts of a run see of the cache: one `KVLayerCache` or `StateLayerCache` per entry of
         the arrangement's `cache_specs()`, in that order."""
+        return self._views(self._run_caches[run], cache, step)
+
+    @staticmethod
+    def _views(entries, cache: SequenceCache, step) -> list:
         out = []
-        for c, writable in self._run_caches[run]:
+        for c, writable in entries:
             if c in cache.layer_group:
                 gi = cache.layer_group[c]
                 g = cache.kv_groups[gi]
                 o = g.ordinal(c)
-                out.append(KVLayerCache(g.k[o], g.v[o], step.block_tables[gi], g.spec.window, writable))
+                out.append(KVLayerCache(g.k[o], g.v[o], step.block_tables[gi], g.spec.window, writable,
+                                        g.spec.keep_first))
             else:
                 out.append(StateLayerCache(cache.state[c], writable))
         return out
@@ -157,7 +166,8 @@ class Model:
     def forward(self, step, cache: SequenceCache) -> Optional[torch.Tensor]:
         """Run the step's tokens through the scheduled layers; returns fp32 logits
         [wanted rows, vocab] (None if no row is wanted)."""
-        stream = ResidualStream(self.embedding.forward(step))
+        kept = self._views(self._embedding_caches, cache, step)
+        stream = ResidualStream(self.embedding.forward(step, kept) if kept else self.embedding.forward(step))
         hook = self.layer_hook
         last = len(self.spec.schedule) - 1
         # a later run may add the embedding's output once more: the layers change the stream in place, so keep a copy

@@ -18,6 +18,9 @@ _vp, _i, _l, _f = ctypes.c_void_p, ctypes.c_int, ctypes.c_long, ctypes.c_float
 
 _SIGNATURES = {
     "plm_embed": [_vp, _vp, _i, _vp, _i, _i, _i, _f, _vp],
+    "plm_embed_pair": [_vp, _vp, _vp, _i, _vp, _l, _vp, _vp, _vp, _vp, _i, _i, _i, _l, _l, _l, _f, _vp],
+    "plm_joined_post_pre_norm": [_vp, _vp, _vp, _vp, _vp, _f, _vp, _vp, _vp, _i, _i, _i, _f, _f, _f, _f, _vp],
+    "plm_gelu_erf": [_vp, _vp, _i, _l, _vp],
     "plm_rmsnorm": [_vp, _vp, _vp, _i, _vp, _i, _vp, _i, _i, _f, _vp],
     "plm_post_pre_norm": [_vp, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _f, _f, _vp],
     "plm_swiglu": [_vp, _vp, _i, _i, _i, _i, _f, _f, _vp],
@@ -58,10 +61,10 @@ _SIGNATURES = {
     "plm_gemm_tc_wide_splits": [_i, _i, _i],
     "plm_gemm_tc_pair": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _l, _l, _l, _vp, _vp],
     "plm_gemm_simt": [_vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _l, _l, _l, _vp],
-    "plm_attention_rows": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _vp, _vp],
-    "plm_attn_prefill": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _vp, _vp],
-    "plm_attn_tc_prefill": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _vp, _vp],
-    "plm_attn_decode": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _i, _i, _vp, _vp, _vp],
+    "plm_attention_rows": [_vp, _vp, _vp, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _vp, _i, _vp, _vp],
+    "plm_attn_prefill": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _vp, _i, _vp, _vp],
+    "plm_attn_tc_prefill": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _vp, _i, _vp, _vp],
+    "plm_attn_decode": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _i, _i, _vp, _vp, _i, _vp, _vp],
     "plm_attn_decode_rope": [_vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _f, _i, _i, _i, _vp, _vp],
     "plm_check_bounds": [_i, _i, _i, _i, _vp, _vp],
     "plm_decode_chain": [_vp, _i, _i, _vp, _vp, _vp, _vp],
@@ -74,7 +77,7 @@ _SIGNATURES = {
     "plm_delta_chunk_scan": [_vp, _vp, _vp, _vp, _vp, _i, _l, _vp, _l, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
     "plm_delta_scan": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _l, _vp, _l, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
     "plm_linear_scan": [_vp, _vp, _vp, _vp, _i, _l, _l, _l, _l, _i, _vp, _vp, _vp, _f, _f, _vp, _l, _vp, _l, _vp, _vp,
-                        _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp],
+                        _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _i, _vp],
     "plm_sigmoid_decay": [_vp, _i, _l, _vp, _f, _vp, _i, _i, _vp],
     "plm_linear_scan_plan": [_i, _i, _i, _i, _i, _i, _vp],
     "plm_gated_norm": [_vp, _i, _l, _vp, _i, _l, _vp, _i, _vp, _i, _l, _i, _i, _i, _f, _i, _i, _i, _vp],

@@ -81,6 +81,65 @@ def post_pre_norm(x: torch.Tensor, delta: torch.Tensor, w_post: torch.Tensor, ep
     return out
 
 
+def embed_pair(step, table: torch.Tensor, pairs: torch.Tensor, state: torch.Tensor, mul_prev: int, mul_cur: int,
+               scale: float = 1.0) -> torch.Tensor:
+    """out[t, :] = (table[token] + pairs[row]) * scale as the fp32 residual stream, with
+    row = (token before * mul_prev + token * mul_cur) mod buckets for `pairs` [buckets + 1, d]; a sequence's first token
+    takes the last row.  `state` int32 [slots + 1, >= 1] with contiguous rows holds every sequence's last token + 1 (0:
+    none yet) and is brought up to date."""
+    _dev(table, "table"), _dev(pairs, "pairs"), _i32(step.tok_ids, "tok_ids")
+    T, (vocab, d) = step.tok_ids.numel(), table.shape
+    if pairs.dim() != 2 or pairs.shape[1] != d or pairs.shape[0] < 2 or pairs.dtype != table.dtype:
+        raise KernelError(f"embed_pair: the pair table must be [buckets + 1, {d}] of {table.dtype}")
+    if not state.is_cuda or state.dtype != torch.int32 or state.dim() != 2 or state.stride(1) != 1:
+        raise KernelError("embed_pair: the state must be int32 [slots, 1] on the device")
+    out = torch.empty((T, d), dtype=torch.float32, device=table.device)
+    set_bounds("elementwise", n_seqs=step.n_seqs, device=table.device)
+    _check(_fn("elementwise", "plm_embed_pair")(
+        _p(step.tok_ids), _p(table), _p(pairs), _dt(table, "table"), _p(state), state.stride(0), _p(step.tok_seq),
+        _p(step.seq_start), _p(step.seq_slot), _p(out), T, d, vocab, pairs.shape[0] - 1, int(mul_prev), int(mul_cur),
+        float(scale), _stream()), f"embed_pair T={T} d={d}", nbytes=T * d * (4 + 2 * table.element_size()))
+    return out
+
+
+def joined_post_pre_norm_supported(x: torch.Tensor, a, b, *weights) -> bool:
+    """Whether `joined_post_pre_norm` takes this case: float32 stream and rows of one shape, a multiple of 4 and at most
+    16,384 columns, float32 weights."""
+    d = x.shape[1]
+    return (d % 4 == 0 and d <= 16384
+            and all(isinstance(t, torch.Tensor) and t.dtype == torch.float32 and t.shape == x.shape and t.is_contiguous()
+                    and t.data_ptr() % 16 == 0 for t in (x, a, b))
+            and all(w.dtype == torch.float32 and w.shape == (d,) and w.data_ptr() % 16 == 0 for w in weights))
+
+
+def joined_post_pre_norm(x: torch.Tensor, a: torch.Tensor, w_a: torch.Tensor, eps_a: float, b: torch.Tensor, w_b: torch.Tensor,
+                         eps_b: float, factor: float, w_post: torch.Tensor, eps_post: float, w_pre: torch.Tensor,
+                         eps_pre: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """y = factor * (RMSNorm(a; w_a) + RMSNorm(b; w_b)); x += RMSNorm(y; w_post) in place on the fp32 stream; returns
+    RMSNorm(x; w_pre) of the new x as [T, d] of `out_dtype`: what joins two mixers' results, closes their sublayer, adds
+    it and opens the next one, in one kernel.  All rows and weights float32."""
+    for t, n in ((x, "x"), (a, "a"), (b, "b"), (w_a, "w_a"), (w_b, "w_b"), (w_post, "w_post"), (w_pre, "w_pre")):
+        _dev(t, n)
+    if not joined_post_pre_norm_supported(x, a, b, w_a, w_b, w_post, w_pre):
+        raise KernelError("joined_post_pre_norm: not a case the fused kernel takes")
+    T, d = x.shape
+    out = torch.empty((T, d), dtype=out_dtype, device=x.device)
+    _check(_fn("elementwise", "plm_joined_post_pre_norm")(
+        _p(x), _p(a), _p(b), _p(w_a), _p(w_b), float(factor), _p(w_post), _p(w_pre), _p(out), _dt(out, "out"), T, d, float(eps_a),
+        float(eps_b), float(eps_post), float(eps_pre), _stream()), f"joined_post_pre_norm rows={T} d={d}",
+        nbytes=T * d * (16 + out.element_size()))
+    return out
+
+
+def gelu_erf(x: torch.Tensor) -> torch.Tensor:
+    """0.5 x (1 + erf(x / sqrt 2)) element by element, in x's type (float32 inside)."""
+    _dev(x, "x")
+    out = torch.empty_like(x)
+    _check(_fn("elementwise", "plm_gelu_erf")(_p(x), _p(out), _dt(x, "x"), x.numel(), _stream()), "gelu_erf",
+           nbytes=2 * x.numel() * x.element_size())
+    return out
+
+
 def gather_rows(x: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:
     """x[rows] for a 2-D `x` with contiguous rows and int32 `rows` on the device: [len(rows), x.shape[1]]."""
     _i32(rows, "rows")

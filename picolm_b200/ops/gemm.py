@@ -10,6 +10,7 @@ from . import chain as _chain
 from ._lib import (SM_COUNT, KernelError, _check, _dev, _dt, _fn, _p, _stream, status_word, stream_space,
                    stream_space_enabled)
 from .chain import LazyRows
+from .elementwise import gelu_erf
 
 
 def _work(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, extra: int = 0) -> dict:
@@ -373,6 +374,16 @@ def linear_swiglu(a, w_gate_up: torch.Tensor, defer: bool = False, activation: s
         return gemm_tc_skinny(a, w_gate_up, torch.bfloat16, swiglu=True, activation=activation, limit=limit, slope=slope)
     return gemm_tc_wide(a, w_gate_up, torch.bfloat16, swiglu=True, pair=pair_pays(M, N, K, 1), activation=activation,
                         limit=limit, slope=slope)
+
+
+PLAIN_ACTIVATIONS = ("gelu_erf",)
+
+
+def linear_act(a, w: torch.Tensor, out_dtype: torch.dtype, activation: str):
+    """act(a [M, K] times w [N, K]^T) -> [M, N]: a product with an activation that has no gate behind it."""
+    if activation not in PLAIN_ACTIVATIONS:
+        raise KernelError(f"activation {activation!r} without a gate has no kernel; known: {', '.join(PLAIN_ACTIVATIONS)}")
+    return gelu_erf(linear(a, w, out_dtype))
 
 
 def linear(a, w: torch.Tensor, out_dtype: torch.dtype, defer: bool = False):

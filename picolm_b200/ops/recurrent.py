@@ -9,7 +9,7 @@ import torch
 
 from ._lib import PAGE_TOKENS, KernelError, _check, _dev, _dt, _fn, _i32, _p, _stream, set_bounds
 
-DECAY_STEP, DECAY_SIGMOID, DECAY_GIVEN = 1, 2, 3
+DECAY_STEP, DECAY_SIGMOID, DECAY_GIVEN, DECAY_CONST = 1, 2, 3, 4
 
 
 def _cols(t: torch.Tensor, name: str) -> int:
@@ -60,9 +60,10 @@ def causal_conv(u: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tens
     return out
 
 
-def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, raw: torch.Tensor, mode: int, p0: torch.Tensor,
+def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, raw: Optional[torch.Tensor], mode: int, p0: torch.Tensor,
                 p1: Optional[torch.Tensor], skip: Optional[torch.Tensor], q_scale: float, power: float,
-                state: torch.Tensor, step, heads: int, key_dim: int, value_dim: int, heads_per_group: int = 1) -> torch.Tensor:
+                state: torch.Tensor, step, heads: int, key_dim: int, value_dim: int, heads_per_group: int = 1,
+                activation: Optional[str] = None) -> torch.Tensor:
     """The recurrence S_t = diag(d_t) S_(t-1) + k_t v_t^T, y_t = S_t^T (q_scale q_t) (+ skip[h] v_t) over each
     sequence's tokens, per head, everything in float32; returns y [T, heads * value_dim] float32.
 
@@ -71,8 +72,14 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, raw: torch.Te
       DECAY_STEP     raw [T, heads]: dt = softplus(raw + p0[h]), d = exp(-exp(p1[h]) dt) for the whole head, and
                      v_t enters the state times dt (the skip term takes it unscaled)
       DECAY_SIGMOID  raw [T, heads * key_dim]: d[n] = sigmoid(raw + p0[h, n]) ** power
+      DECAY_CONST    raw None: d = p0[h] for the whole head and every token; with `activation="silu"` q, k and v pass
+                     SiLU on their way in (float32, from the rows as they are)
     `state` float32 [slots, >= heads * key_dim * value_dim] with contiguous rows holds S of every sequence as
     [heads, key_dim, value_dim] and is carried on."""
+    if raw is None and mode == DECAY_CONST:
+        raw = v                                              # (not read)
+    if activation not in (None, "silu") or (activation and mode != DECAY_CONST):
+        raise KernelError(f"linear_scan: activation {activation!r} is not known in this decay mode")
     ldq, ldk, ldv, ldr = _cols(q, "q"), _cols(k, "k"), _cols(v, "v"), _cols(raw, "raw")
     T = v.shape[0]
     H, N, P = heads, key_dim, value_dim
@@ -91,6 +98,8 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, raw: torch.Te
         if raw.shape != (T, H * N):
             raise KernelError("linear_scan: a decay per key channel wants raw [T, heads * key_dim]")
         _f32(p0, "p0", H * N)
+    elif mode == DECAY_CONST:
+        _f32(p0, "p0", H)
     else:
         raise KernelError(f"linear_scan: unknown decay mode {mode}")
     _f32(skip, "skip", H)
@@ -119,7 +128,7 @@ def linear_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, raw: torch.Te
     _check(_fn("recurrent", "plm_linear_scan")(
         _p(q), _p(k), _p(v), _p(raw), _dt(v, "v"), ldq, ldk, ldv, ldr, run_mode, _p(p0), _p(p1), _p(skip), float(q_scale),
         float(power), _p(state), lds, _p(y), H * P, _p(step.seq_start), _p(step.seq_slot), step.n_seqs, H, N, P,
-        heads_per_group, seg_len, n_segs, _p(seg_state), _p(seg_decay), _stream()),
+        heads_per_group, seg_len, n_segs, _p(seg_state), _p(seg_decay), 1 if activation == "silu" else 0, _stream()),
         f"linear_scan T={T} H={H} N={N} P={P}" + (f" in {n_segs} segments" if n_segs > 1 else ""),
         kernels=kernels,
         nbytes=T * (2 * G * N + H * P) * v.element_size() + T * H * P * 4 + 2 * step.n_seqs * H * N * P * 4,

@@ -29,7 +29,9 @@ def route_topk(logits: torch.Tensor, n_experts: int, top: int, correction: Optio
                gate_col: Optional[int] = None, scores: str = "sigmoid", group_score: str = "top2",
                normalize: bool = True) -> Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]:
     """The choice of `top` experts per token from router logits [T, >= n_experts] (float32): scores are
-    `sigmoid(logit)` (`scores="softmax"`: the softmax over the n_experts logits); the choice goes by score +
+    `sigmoid(logit)` (`scores="softmax"`: the softmax over the n_experts logits; `scores="logits"`: the logits plus
+    `correction`, which is then a bias of the router, and the weights are the softmax over the chosen ones alone, times
+    `scale`); the choice goes by score +
     `correction` (float32 [n_experts]), among the experts of the
     `keep_groups` best of `n_groups` equal groups of neighbours (a group's score: the sum of its two largest choice
     scores, or with `group_score="max"` its largest); the weights are the chosen scores without the correction,
@@ -46,14 +48,14 @@ def route_topk(logits: torch.Tensor, n_experts: int, top: int, correction: Optio
         _dev(correction, "correction")
         if correction.dtype != torch.float32 or correction.shape != (E,):
             raise KernelError("route_topk: correction must be float32 [experts]")
-    if scores not in ("sigmoid", "softmax") or group_score not in ("top2", "max"):
-        raise KernelError(f"route_topk: scores {scores!r} (sigmoid, softmax) or group_score {group_score!r} (top2, max) is not known")
+    if scores not in ("sigmoid", "softmax", "logits") or group_score not in ("top2", "max"):
+        raise KernelError(f"route_topk: scores {scores!r} (sigmoid, softmax, logits) or group_score {group_score!r} (top2, max) is not known")
     ids = torch.empty((T, top), dtype=torch.int32, device=logits.device)
     weights = torch.empty((T, top), dtype=torch.float32, device=logits.device)
     gate = torch.empty((T,), dtype=torch.float32, device=logits.device) if gate_col is not None else None
     _check(_fn("routed", "plm_route_topk")(
         _p(logits), ld, _p(correction), E, int(top), int(n_groups), int(keep_groups), float(scale), _p(ids), _p(weights),
-        _p(gate), int(gate_col or 0), T, 1 if scores == "softmax" else 0, 1 if group_score == "max" else 0,
+        _p(gate), int(gate_col or 0), T, ("sigmoid", "softmax", "logits").index(scores), 1 if group_score == "max" else 0,
         1 if normalize else 0, _stream()), f"route_topk T={T} E={E}")
     return ids, weights, gate
 

@@ -17,7 +17,8 @@ Families and what `forward` takes and returns (T = tokens of the step):
                 mixers (see `parts/position.py`).
   arrangement   forward(stream, step, cache): one block, i.e. how the layer's
                 norms, mixer and feed-forward are wired around the stream.
-  embedding     forward(step) -> stream x [T, d] fp32.
+  embedding     forward(step) -> stream x [T, d] fp32; one that keeps something per sequence says what in `cache_specs()`
+                and is called forward(step, caches).
   head          forward(h_rows) -> logits [rows, vocab] fp32.
   token_input   forward(x, step, rows=None) -> delta fp32 from the stream's rows x (in the run's dtype) and the
                 tokens they belong to (`rows`: the step's row numbers of x's rows where the stream was narrowed).

@@ -24,7 +24,7 @@ from .. import ops
 from ..cache.spec import CacheSpec
 from ..config.spec import LayerSpec, PartSpec
 from .base import Part, WeightSpec, build_part, register_part
-from .stream import PostNormed, settle
+from .stream import JoinedNorms, PostNormed, settle
 
 
 class Arrangement(Part):
@@ -137,6 +137,8 @@ class SandwichNormBlock(Arrangement):
 
     @staticmethod
     def _rows(delta):
+        if isinstance(delta, JoinedNorms):              # the closing norm joins the halves on its way
+            return delta
         return delta.compute() if hasattr(delta, "compute") else delta
 
     def forward(self, stream, step, caches, keep_rows=None):

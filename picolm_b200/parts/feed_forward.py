@@ -66,6 +66,37 @@ class GatedMLP(Part):
         return ops.linear(act, self.w_down, torch.float32, defer=True)
 
 
+@register_part("feed_forward", "mlp")
+class PlainMLP(Part):
+    """Two maps with an activation between them, `W_down act(W_up h)`, no gate and no biases.  params: hidden_size,
+    intermediate_size, activation ("gelu_erf": 0.5 z (1 + erf(z / sqrt 2))), up_name/down_name (relative tensor names)."""
+
+    def __init__(self, params, runtime):
+        super().__init__(params, runtime)
+        if self.params["activation"] not in ops.PLAIN_ACTIVATIONS:
+            raise ValueError(f"activation {self.params['activation']!r} without a gate has no kernel; known: "
+                             + ", ".join(ops.PLAIN_ACTIVATIONS))
+
+    def weight_specs(self):
+        p = self.params
+        d, F = p["hidden_size"], p["intermediate_size"]
+        return {p["up_name"]: WeightSpec((F, d)), p["down_name"]: WeightSpec((d, F))}
+
+    def load(self, tensors):
+        self.w_up, self.w_down = tensors[self.params["up_name"]], tensors[self.params["down_name"]]
+
+    def weight_bytes(self):
+        return sum(t.numel() * t.element_size() for t in (self.w_up, self.w_down))
+
+    takes_scaled_rows = True          # h goes into a product and nowhere else
+    graph_safe = True
+    graph_safe_prompts = True
+
+    def forward(self, h, step):
+        act = ops.linear_act(h, self.w_up, self.runtime.dtype, self.params["activation"])
+        return ops.linear(act, self.w_down, torch.float32, defer=True)
+
+
 @register_part("feed_forward", "routed_mlp")
 class RoutedMLP(Part):
     """A mixture of experts: every token uses `top` of `experts` small gated MLPs (`W_down(silu(W_gate h) * W_up h)`,
@@ -79,7 +110,8 @@ class RoutedMLP(Part):
     {"size", "prefix", "gate"}: the shared expert's inner width, its tensors' prefix, and the name under that prefix of
     the [1, hidden] row whose sigmoid multiplies the shared expert's result per token; None: no such gate).
 
-    Optional: scores ("sigmoid", or "softmax": over all router outputs), group_score ("top2", or "max": a group's
+    Optional: scores ("sigmoid", or "softmax": over all router outputs, or "logits": the choice goes by the logits plus the
+    tensor `correction_name`, a bias of the router, and the weights are the softmax over the chosen ones), group_score ("top2", or "max": a group's
     score is its best choice score), normalize (False: the weights are the chosen scores as they are, times
     `route_scale`), identity (a number: the router has that many outputs more, behind the experts', for experts
     without tensors whose output is their input; they take part in scores, groups and choice like the others).
@@ -106,8 +138,8 @@ class RoutedMLP(Part):
         self.n_out = self.E + self.identity                  # the router's outputs: experts, then identity experts
         self.scores, self.group_score = p.get("scores", "sigmoid"), p.get("group_score", "top2")
         self.normalize = bool(p.get("normalize", True))
-        if self.scores not in ("sigmoid", "softmax") or self.group_score not in ("top2", "max"):
-            raise ValueError(f"routed_mlp: scores={self.scores!r} (sigmoid, softmax) or group_score={self.group_score!r} "
+        if self.scores not in ("sigmoid", "softmax", "logits") or self.group_score not in ("top2", "max"):
+            raise ValueError(f"routed_mlp: scores={self.scores!r} (sigmoid, softmax, logits) or group_score={self.group_score!r} "
                              f"(top2, max) is not known")
         if not 0 < self.top <= self.n_out or self.n_out % self.n_groups or not 0 < self.keep <= self.n_groups or self.identity < 0:
             raise ValueError(f"routed_mlp: top={self.top}, router outputs={self.n_out}, groups={self.n_groups}, "

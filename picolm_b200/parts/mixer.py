@@ -20,7 +20,7 @@ from .. import ops
 from ..cache.spec import CacheSpec
 from ..config.spec import PartSpec
 from .base import Part, WeightSpec, build_part, register_part
-from .stream import BiasedDelta
+from .stream import BiasedDelta, JoinedNorms
 
 
 def _stack_rows(tensors):
@@ -60,6 +60,8 @@ class Attention(Part):
                     `<q_name|k_name|v_name><suffix>` [channels, taps], the last tap the token's own.  The last taps - 1
                     projected rows of a sequence are kept beside the keys and values (a cache of the layer's own
                     even where keys and values are borrowed)
+      keep_first    beside the window's keys a query sees the sequence's first keep_first positions
+      slopes        numbers, one per head: a score of head h loses slopes[h] times its key's distance, outside the scale
       head_scale_name  a tensor [num_heads]: head h's scores are multiplied by it (its queries are, after the rotation)
     With any of value_dim, bias, qk_norm or own_kv=False, what stands between the QKV product and attention is one
     kernel (`ops.qk_norm_rope_store`: bias, norm and rotation in float32 on the product's float32 result) and the
@@ -85,6 +87,12 @@ class Attention(Part):
         self.scale = float(p["scale"]) if p.get("scale") is not None else 1.0 / math.sqrt(self.hd)
         self.window = p.get("window")
         self.chunk = p.get("chunk")
+        self.keep_first = int(p.get("keep_first") or 0)
+        if self.keep_first and self.window is None:
+            raise ValueError("attention: keep_first goes with a sliding window")
+        self.slope_values = p.get("slopes")
+        if self.slope_values is not None and len(self.slope_values) != self.H:
+            raise ValueError(f"attention: {len(self.slope_values)} slopes for {self.H} heads")
         if self.chunk is not None and (self.window is not None or int(self.chunk) <= 0):
             raise ValueError("a mask of chunks needs a positive size and excludes a sliding window")
         self.vd = int(p.get("value_dim") or self.hd)
@@ -106,13 +114,19 @@ class Attention(Part):
         # the general form: its own kernel between the product and attention, a cache of padded heads
         self.general = (self.vd != self.hd or self.bias or self.qk_norm is not None or not self.own_kv or self.v_from_k
                         or self.sink_name is not None or self.sink_value is not None or self.gate_name is not None
-                        or self.conv is not None or self.head_scale_name is not None)
+                        or self.conv is not None or self.head_scale_name is not None or self.slope_values is not None
+                        or self.keep_first > 0)
         self.hd_c = -(-max(self.hd, self.vd) // 16) * 16 if self.general else self.hd
         pos = p.get("position") or PartSpec("none")
         self.position = build_part("position", pos, runtime)
         if self.general and not hasattr(self.position, "rotation") and pos.kind != "none":
             raise ValueError(f"attention with a bias, a norm of q and k or values of another width needs a position "
                              f"encoding that is a rotation (or none), not {pos.kind!r}")
+
+        # where nothing is computed from the projections' float32 sums (no norm, rotation, convolution, bias, factor or gate),
+        # the product's result is stored in the run's type at once: it is rounded to it before attention in any case
+        self.plain_rows = (pos.kind == "none" and not self.bias and self.qk_norm is None and self.conv is None
+                           and self.gate_name is None and self.head_scale_name is None)
 
     def _names(self):
         """(tensor names of the projections that feed attention, in the order of their rows in the one product)."""
@@ -160,6 +174,9 @@ class Attention(Part):
                 g = wide.view(self.H * self.hd_c, self.d)
             rows.append(g)
         self.w_qkv = _stack_rows(rows)
+        self.w_qkv_bytes = self.w_qkv.numel() * self.w_qkv.element_size()
+        self.slopes = (None if self.slope_values is None else
+                       torch.tensor([float(s) for s in self.slope_values], dtype=torch.float32, device=self.w_qkv.device))
         self.w_o = tensors[p["o_name"]]
         self.b_qkv = self.b_o = self.w_qn = self.w_kn = None
         self.sink = None if self.sink_name is None else tensors[self.sink_name].to(torch.float32).contiguous()
@@ -187,11 +204,21 @@ class Attention(Part):
             self.w_o = w.view(self.d, self.H * self.hd_c).contiguous()
 
     def weight_bytes(self):
-        return sum(t.numel() * t.element_size() for t in (self.w_qkv, self.w_o))
+        return self.w_qkv_bytes + self.w_o.numel() * self.w_o.element_size()
+
+    def projection_type(self):
+        """The stored type of the matrix `take_projection` would give, or None if the part needs its own product."""
+        return self.w_qkv.dtype if self.general and self.plain_rows else None
+
+    def take_projection(self):
+        """The matrix that makes everything this part reads of h, for an owner that makes one product of several parts'
+        (`forward(..., proj=)` then takes its columns, in the run's type); the part no longer holds it."""
+        w, self.w_qkv = self.w_qkv, None
+        return w
 
     def cache_spec(self):
         # (chunks: pages are kept; a layer that borrows this cache may cut its chunks elsewhere)
-        return CacheSpec.kv(self.G, self.hd_c, self.window)
+        return CacheSpec.kv(self.G, self.hd_c, self.window, keep_first=self.keep_first)
 
     def cache_specs(self):
         """The keys and values, and for a convolution the last taps - 1 projected rows of every sequence (the layer's
@@ -207,34 +234,35 @@ class Attention(Part):
 
     takes_scaled_rows = True          # h goes into a product and nowhere else
 
-    def _forward_general(self, h, step, cache, conv_state=None):
+    def _forward_general(self, h, step, cache, conv_state=None, proj=None):
         dt = self.runtime.dtype
         if self.own_kv and not cache.writable:
             raise RuntimeError("a layer that reads another layer's cache must be built with own_kv=False")
-        proj = ops.linear(h, self.w_qkv, torch.float32)      # bias, norm and rotation work on the float32 sums
+        if proj is None:                                     # bias, norm and rotation work on the float32 sums
+            proj = ops.linear(h, self.w_qkv, dt if self.plain_rows else torch.float32)
         qkv = proj[:, :self.n_qkv] if self.gate_name is not None else proj
         if self.w_conv is not None and self.w_conv.shape[0] > 1 and conv_state is None:
             raise RuntimeError("attention with a convolution was handed no state for it")
-        q = torch.empty((h.shape[0], self.H, self.hd_c), dtype=dt, device=h.device)
+        q = torch.empty((qkv.shape[0], self.H, self.hd_c), dtype=dt, device=qkv.device)
         rotation = self.position.rotation() if hasattr(self.position, "rotation") else None
         ops.qk_norm_rope_store(qkv, self.b_qkv, self.w_qn, self.w_kn, self.qk_norm["eps"] if self.qk_norm else 0.0, q,
                                cache, rotation, step, self.H, self.G, self.hd, self.vd, own_kv=self.own_kv,
                                per_head=self.per_head_norm, values_from_keys=self.v_from_k, q_scale=self.head_scale,
                                conv=self.w_conv, conv_state=conv_state.state if conv_state is not None else None)
-        ctx = ops.attention(q, cache, step, self.G, self.scale, chunk=self.chunk, sink=self.sink)
+        ctx = ops.attention(q, cache, step, self.G, self.scale, chunk=self.chunk, sink=self.sink, slopes=self.slopes)
         if self.gate_name is not None:
             ctx = ops.gated_norm(ctx, dt, group=self.hd_c, gate=proj[:, self.n_qkv:], gate_mode=ops.GATE_AFTER_NORM,
                                  activation="sigmoid", norm=False)
         delta = ops.linear(ctx, self.w_o, torch.float32, defer=True)
         return BiasedDelta(delta, self.b_o) if self.b_o is not None else delta
 
-    def forward(self, h, step, cache):
+    def forward(self, h, step, cache, proj=None):
         conv_state = None
         if isinstance(cache, (list, tuple)):                 # all of `cache_specs()`, in their order
             conv_state = cache[1] if len(cache) > 1 else None
             cache = cache[0]
         if self.general:
-            return self._forward_general(h, step, cache, conv_state)
+            return self._forward_general(h, step, cache, conv_state, proj)
         dt = self.runtime.dtype
         qkv = ops.linear(h, self.w_qkv, dt)
         # a position encoding that can describe itself as a rotation (`rotation()`) may be applied, and the
@@ -265,12 +293,25 @@ class ParallelMixers(Part):
     """Two mixers side by side that read the same normed rows; the result is `left_scale * left + right_scale *
     right`.  params: left, right (`PartSpec`s of the mixer family; their `prefix` is where their tensors live below
     this part's), left_scale, right_scale.  Each half keeps what it keeps in the cache: the layer's caches are the
-    left's, then the right's (`cache_specs`), and `forward` takes them as a list."""
+    left's, then the right's (`cache_specs`), and `forward` takes them as a list.
+
+    Optional: left_norm, right_norm (`PartSpec`s of the norm family, RMS norms over the model's width): each half's result
+    passes its own norm before the two are added; left_scale and right_scale are then equal, and the result comes
+    back as `JoinedNorms`, so that a norm behind it can do both norms and the sum in its own pass.
+
+    Where both halves can be handed their projections (`take_projection`), everything they read of h is one product."""
 
     def __init__(self, params, runtime):
         super().__init__(params, runtime)
         self.halves = [(self.params[side].prefix, build_part("mixer", self.params[side], runtime)) for side in ("left", "right")]
         self.scales = (float(self.params["left_scale"]), float(self.params["right_scale"]))
+        self.norms = None
+        if self.params.get("left_norm") is not None or self.params.get("right_norm") is not None:
+            if self.scales[0] != self.scales[1]:
+                raise ValueError("parallel mixers with a norm each need one scale for both")
+            self.norms = [(self.params[f"{side}_norm"].prefix, build_part("norm", self.params[f"{side}_norm"], runtime))
+                          for side in ("left", "right")]
+        self.w_in = None
 
     @property
     def graph_safe(self) -> bool:
@@ -281,15 +322,26 @@ class ParallelMixers(Part):
         return all(bool(getattr(part, "graph_safe_prompts", False)) for _, part in self.halves)
 
     def weight_specs(self):
-        return {(f"{prefix}.{name}" if prefix else name): ws for prefix, part in self.halves
+        return {self._join(prefix, name): ws for prefix, part in self.halves + (self.norms or [])
                 for name, ws in part.weight_specs().items()}
 
+    @staticmethod
+    def _join(prefix, name):
+        return ".".join(n for n in (prefix, name) if n)
+
     def load(self, tensors):
-        for prefix, part in self.halves:
-            part.load({name: tensors[f"{prefix}.{name}" if prefix else name] for name in part.weight_specs()})
+        for prefix, part in self.halves + (self.norms or []):
+            part.load({name: tensors[self._join(prefix, name)] for name in part.weight_specs()})
+        parts = [part for _, part in self.halves]
+        self.w_in = None
+        if all(hasattr(part, "take_projection") and part.projection_type() is not None for part in parts) \
+                and parts[0].projection_type() == parts[1].projection_type():
+            rows = [part.take_projection() for part in parts]
+            self.n_left = rows[0].shape[0]
+            self.w_in = torch.cat(rows, dim=0).contiguous()
 
     def weight_bytes(self):
-        return sum(part.weight_bytes() for _, part in self.halves)
+        return sum(part.weight_bytes() for _, part in self.halves + (self.norms or []))
 
     def cache_specs(self):
         return [s for _, part in self.halves for s in ([part.cache_spec()] if part.cache_spec() is not None else [])]
@@ -306,10 +358,19 @@ class ParallelMixers(Part):
 
     def forward(self, h, step, caches):
         caches = list(caches)
-        results = []
-        for _, part in self.halves:
+        results, proj = [], (None, None)
+        if self.w_in is not None:
+            both = ops.linear(h, self.w_in, self.runtime.dtype)
+            proj = (both[:, :self.n_left], both[:, self.n_left:])
+        for (_, part), rows in zip(self.halves, proj):
             cache = caches.pop(0) if part.cache_spec() is not None else None
-            results.append(_rows(part.forward(h, step, cache)))
+            results.append(part.forward(h, step, cache) if rows is None else part.forward(h, step, cache, proj=rows))
+        if self.norms is not None and not any(isinstance(r, BiasedDelta) for r in results):
+            return JoinedNorms(results[0], self.norms[0][1], results[1], self.norms[1][1], self.scales[0])
+        results = [_rows(r) for r in results]
+        if self.norms is not None:
+            rows = [ops.add_bias(r, bias) if bias is not None else r for r, bias in results]
+            return JoinedNorms(rows[0], self.norms[0][1], rows[1], self.norms[1][1], self.scales[0])
         (left, left_bias), (right, right_bias) = results
         if right_bias is not None:
             right = ops.add_bias(right, right_bias)

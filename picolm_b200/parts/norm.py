@@ -10,14 +10,16 @@ import torch
 
 from .. import ops
 from .base import Part, WeightSpec, register_part
-from .stream import BiasedDelta, PostNormed, ResidualStream, pending_addends
+from .stream import BiasedDelta, JoinedNorms, PostNormed, ResidualStream, pending_addends
 
 
 @register_part("norm", "rmsnorm")
 class RMSNorm(Part):
     """params: size, eps, name (the weight's tensor name relative to the part's prefix; default "weight", ""
     for a tensor that is called by the prefix alone), one_plus (True: the weight is stored around zero and the row
-    is multiplied by 1 + w; the sum is made once, in float32, when the weights are loaded).  Weight: [size]."""
+    is multiplied by 1 + w; the sum is made once, in float32, when the weights are loaded), scale (a constant that
+    multiplies the weight, likewise once and in float32: a factor on what a closing norm adds to the stream).
+    Weight: [size]."""
 
     @property
     def _name(self) -> str:
@@ -35,6 +37,8 @@ class RMSNorm(Part):
         if self.one_plus:
             # 1 + w has more digits than the stored type holds: kept in float32 (the norm kernels take either)
             self.weight = (1.0 + self.weight.to(torch.float32)).contiguous()
+        if float(self.params.get("scale", 1.0)) != 1.0:
+            self.weight = (float(self.params["scale"]) * self.weight.to(torch.float32)).contiguous()
 
     def weight_bytes(self):
         return self.weight.numel() * self.weight.element_size()
@@ -50,7 +54,7 @@ class RMSNorm(Part):
     def can_defer_scale(self) -> bool:
         """Whether the scale may be left to the products that take the result (their epilogues apply a weight of the
         run's type, which 1 + w is not)."""
-        return not self.one_plus
+        return not self.one_plus and float(self.params.get("scale", 1.0)) == 1.0
 
     graph_safe = True
     graph_safe_prompts = True
@@ -66,9 +70,21 @@ class RMSNorm(Part):
         p = stream.pending
         if isinstance(p, PostNormed):
             # a sublayer's result that wants a norm of its own before the add: both norms and the add in one kernel
-            if rows is None and ops.post_pre_norm_supported(stream.x, p.delta, p.norm.weight, self.weight):
+            if rows is None and isinstance(p.delta, JoinedNorms):
+                j = p.delta
+                a, b = j.rows()
+                w = [n.weight_f32() for n in (j.norm_a, j.norm_b, p.norm, self)]
+                if ops.joined_post_pre_norm_supported(stream.x, a, b, *w):
+                    stream.pending = None
+                    return ops.joined_post_pre_norm(stream.x, a, w[0], j.norm_a.params["eps"], b, w[1], j.norm_b.params["eps"],
+                                                    j.factor, w[2], p.norm.params["eps"], w[3], self.params["eps"],
+                                                    self.runtime.dtype)
+            w_post, w_pre = p.norm.weight, self.weight
+            if w_post.dtype != w_pre.dtype:
+                w_post, w_pre = p.norm.weight_f32(), self.weight_f32()
+            if rows is None and ops.post_pre_norm_supported(stream.x, p.delta, w_post, w_pre):
                 stream.pending = None
-                return ops.post_pre_norm(stream.x, p.delta, p.norm.weight, p.norm.params["eps"], self.weight,
+                return ops.post_pre_norm(stream.x, p.delta, w_post, p.norm.params["eps"], w_pre,
                                          self.params["eps"], self.runtime.dtype)
             stream.pending = p.compute()
         if isinstance(stream.pending, BiasedDelta):

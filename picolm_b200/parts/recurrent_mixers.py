@@ -151,6 +151,61 @@ class GatedLinearAttention(_StateMixer):
         return ops.linear(gated, self.w_o, torch.float32, defer=True)
 
 
+@register_part("mixer", "lightning")
+class LightningAttention(_StateMixer):
+    """Linear attention with one constant decay a head.  params: hidden_size, heads, dim (key size of a head), vdim,
+    decay (a number per head), eps.  `q = silu(W_q h)`, `k = silu(W_k h)`, `v = silu(W_v h)`; per head
+    `S_t = decay_h S_(t-1) + k_t v_t^T`, `o_t = S_t^T q_t`; the concatenated heads are RMS-normed together, multiplied by
+    `sigmoid(W_g h)` and projected.
+
+    Tensors: q, k [heads dim, hidden], v, g [heads vdim, hidden], norm [heads vdim], o [hidden, heads vdim]."""
+
+    def __init__(self, params, runtime):
+        super().__init__(params, runtime)
+        p = self.params
+        self.d, self.H, self.N, self.P, self.eps = p["hidden_size"], p["heads"], p["dim"], p["vdim"], float(p["eps"])
+        if len(p["decay"]) != self.H:
+            raise ValueError(f"lightning: {len(p['decay'])} decays for {self.H} heads")
+
+    def weight_specs(self):
+        HN, HP, d = self.H * self.N, self.H * self.P, self.d
+        return {"q": WeightSpec((HN, d)), "k": WeightSpec((HN, d)), "v": WeightSpec((HP, d)), "g": WeightSpec((HP, d)),
+                "norm": WeightSpec((HP,), init="ones_normal"), "o": WeightSpec((d, HP))}
+
+    def load(self, tensors):
+        self.w_h = _stack_rows([tensors[n] for n in ("q", "k", "v", "g")])       # one product for everything that reads h
+        self.w_o, self.norm_w = tensors["o"], self._f32(tensors["norm"])
+        self.w_h_bytes = self.w_h.numel() * self.w_h.element_size()
+        self.decay = torch.tensor([float(x) for x in self.params["decay"]], dtype=torch.float32, device=self.w_o.device)
+
+    def weight_bytes(self):
+        return self.w_h_bytes + self.w_o.numel() * self.w_o.element_size()
+
+    def projection_type(self):
+        return self.w_h.dtype
+
+    def take_projection(self):
+        """The matrix of the one product, for an owner that makes it together with other parts' (see `forward`)."""
+        w, self.w_h = self.w_h, None
+        return w
+
+    def cache_spec(self):
+        return CacheSpec.state((self.H * self.N * self.P,))
+
+    def forward(self, h, step, cache, proj=None):
+        dt = self.runtime.dtype
+        HN, HP = self.H * self.N, self.H * self.P
+        if proj is None:
+            proj = ops.linear(h, self.w_h, dt)
+        q, k, v, g = proj[:, :HN], proj[:, HN:2 * HN], proj[:, 2 * HN:2 * HN + HP], proj[:, 2 * HN + HP:]
+        o = ops.linear_scan(q=q, k=k, v=v, raw=None, mode=ops.DECAY_CONST, p0=self.decay, p1=None, skip=None, q_scale=1.0,
+                            power=1.0, state=cache.state, step=step, heads=self.H, key_dim=self.N, value_dim=self.P,
+                            activation="silu")
+        gated = ops.gated_norm(o, dt, weight=self.norm_w, eps=self.eps, gate=g, gate_mode=ops.GATE_AFTER_NORM,
+                               activation="sigmoid")
+        return ops.linear(gated, self.w_o, torch.float32, defer=True)
+
+
 @register_part("mixer", "rglru")
 class GatedDiagonalRecurrence(_StateMixer):
     """A recurrent block around a real-gated diagonal linear recurrence.  params: hidden_size, width (channels of the

@@ -10,7 +10,7 @@ import torch
 
 
 class PostNormed:
-    """A sublayer's float32 result that is still to be normalised (by `norm`, an RMSNorm part) before it is added to
+    """A sublayer's float32 result (rows, or `JoinedNorms`) that is still to be normalised (by `norm`, an RMSNorm part) before it is added to
     the stream: the next norm over the stream may do both in one kernel; anything else calls `compute()`."""
     __slots__ = ("delta", "norm")
 
@@ -22,7 +22,35 @@ class PostNormed:
         return self.delta.shape
 
     def compute(self) -> torch.Tensor:
-        return self.norm.normalize(self.delta)
+        return self.norm.normalize(self.delta.compute() if hasattr(self.delta, "compute") else self.delta)
+
+    def adds_in_place(self, x: torch.Tensor) -> bool:
+        return False
+
+
+class JoinedNorms:
+    """A sublayer's result that is `factor * (norm_a(a) + norm_b(b))`: two float32 results `a`, `b` (rows, or products
+    that have not run), each behind an RMSNorm part of its own.  The norm that closes the sublayer may do all of it in
+    its own pass (`PostNormed` around it); anything else calls `compute()`."""
+    __slots__ = ("a", "norm_a", "b", "norm_b", "factor")
+
+    def __init__(self, a, norm_a, b, norm_b, factor: float):
+        self.a, self.norm_a, self.b, self.norm_b, self.factor = a, norm_a, b, norm_b, float(factor)
+
+    @property
+    def shape(self):
+        return self.a.shape
+
+    def rows(self):
+        """(a, b) as float32 rows; products that have not run do so now, once."""
+        self.a = self.a.compute() if hasattr(self.a, "compute") else self.a
+        self.b = self.b.compute() if hasattr(self.b, "compute") else self.b
+        return self.a, self.b
+
+    def compute(self) -> torch.Tensor:
+        from .. import ops
+        a, b = self.rows()
+        return ops.scaled_sum(self.norm_a.normalize(a), self.factor, self.norm_b.normalize(b), self.factor)
 
     def adds_in_place(self, x: torch.Tensor) -> bool:
         return False
@@ -95,7 +123,9 @@ def _narrowed(p, rows):
     """The pending delta `p` at the rows `rows` only."""
     from .. import ops
     if isinstance(p, PostNormed):
-        return PostNormed(ops.gather_rows(p.delta, rows), p.norm)
+        return PostNormed(_narrowed(p.delta, rows), p.norm)
+    if isinstance(p, JoinedNorms):
+        return JoinedNorms(_narrowed(p.a, rows), p.norm_a, _narrowed(p.b, rows), p.norm_b, p.factor)
     if isinstance(p, BiasedDelta):
         return BiasedDelta(_narrowed(p.delta, rows), p.bias)
     if isinstance(p, ops.PendingLinear):
