@@ -1,9 +1,9 @@
-"""Throughput of another design (Potuzen, Kunulorn, Tebasun, Fupapel) beside the Llama decoder (Tebasun: beside Potuzen, the
+"""Throughput of another design (Potuzen, Kunulorn, Tebasun, Fupapel, Dobepel) beside the Llama decoder (Tebasun: beside Potuzen, the
 other design whose layers are recurrences and attention in turn; Fupapel: beside Kunulorn, the other design of chunked
-attention and routed feed-forwards) at equal layer sizes (random weights): prefill
+attention and routed feed-forwards; Dobepel: beside Tebasun, the other design of attention and a recurrence side by side) at equal layer sizes (random weights): prefill
 tokens/s of one prompt and decode tokens/s of a batch, at a few sizes that resemble a real model's layers,
 and, with `kernels=True`, the device time of every kind of launch with the fraction of the memory's or the
-tensor cores' measured rate that it reaches.  `bench.py --design potuzen|kunulorn|tebasun|fupapel` calls this."""
+tensor cores' measured rate that it reaches.  `bench.py --design potuzen|kunulorn|tebasun|fupapel|dobepel` calls this."""
 from __future__ import annotations
 
 import json
@@ -101,6 +101,24 @@ def fupapel_config(width: int, ff: int, layers: int, vocab: int, heads) -> dict:
     return {"architecture": "Fupapel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "layers": out}
 
 
+def dobepel_config(width: int, ff: int, layers: int, vocab: int) -> dict:
+    """Every layer attention (the heads of Tebasun's: width / 128 of 128 over a quarter as many key heads) with slopes
+    under a window of 4,096 positions that keeps the first 64, beside linear attention (width / 256 heads of 128 x 256);
+    feed-forwards in turn dense (two maps of 1.5 times the gated width, so the same weights) and routed (3 of 32 experts
+    a quarter as wide, 16 at the larger size, and one shared, so that a token's arithmetic equals the dense layer's)."""
+    experts = 32 if width <= 2048 else 16
+    left = {"heads": width // 128, "kv_heads": width // 512, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+            "mask": {"size": 4096, "keep_first": 64}}
+    H = width // 256
+    right = {"heads": H, "dim": 128, "vdim": 256, "decay": [1.0 - 2.0 ** (-1.0 - 10.0 * h / max(1, H - 1)) for h in range(H)]}
+    dense = {"kind": "dense", "ff": 3 * ff // 2}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4}, "shared": {"ff": ff // 4}, "router": {"experts": experts, "top": 3}}
+    return {"architecture": "Dobepel", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "embedding": {"bigram": {"buckets": 4 * vocab + 1, "mul_prev": 31, "mul_cur": 17}},
+            "layers": [{"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": moe if i % 2 else dense}
+                       for i in range(layers)]}
+
+
 def llama_config(width: int, ff: int, layers: int, vocab: int, heads) -> dict:
     H, G, hd = heads
     return {"architectures": ["LlamaForCausalLM"], "model_type": "llama", "num_hidden_layers": layers, "hidden_size": width,
@@ -174,7 +192,7 @@ def _measure(cfg_dict: dict, prompt_tokens: int, batch: int, steps: int, warmup:
     return out
 
 
-def _table(rows, top=14):
+def _table(rows, top=20):
     """The rows of `ops.trace_report` as dictionaries: share of the time, and the larger of the two roofline fractions."""
     from picolm_b200.ops import _lib
     total = sum(r[1] for _, r in rows) or 1.0
@@ -188,10 +206,10 @@ def _table(rows, top=14):
 
 
 def run(design: str, sizes, prompt_tokens: int, batch: int, steps: int, warmup: int, kernels: bool) -> dict:
-    if design not in ("potuzen", "kunulorn", "tebasun", "fupapel"):
-        raise ValueError(f"no design {design!r} to compare (known: potuzen, kunulorn, tebasun, fupapel)")
-    beside = {"tebasun": "potuzen", "fupapel": "kunulorn"}.get(design, "llama")
-    result = {"design": design, "beside": {"potuzen": "Potuzen", "kunulorn": "Kunulorn"}.get(beside, "LlamaForCausalLM"), "dtype": "bf16",
+    if design not in ("potuzen", "kunulorn", "tebasun", "fupapel", "dobepel"):
+        raise ValueError(f"no design {design!r} to compare (known: potuzen, kunulorn, tebasun, fupapel, dobepel)")
+    beside = {"tebasun": "potuzen", "fupapel": "kunulorn", "dobepel": "tebasun"}.get(design, "llama")
+    result = {"design": design, "beside": {"potuzen": "Potuzen", "kunulorn": "Kunulorn", "tebasun": "Tebasun"}.get(beside, "LlamaForCausalLM"), "dtype": "bf16",
               "data": "synthetic (random weights and tokens)",
               "prompt_tokens": prompt_tokens, "decode_batch": batch, "steps": steps, "warmup": warmup, "sizes": {}}
     for name in sizes:
@@ -200,10 +218,12 @@ def run(design: str, sizes, prompt_tokens: int, batch: int, steps: int, warmup: 
         config = {"potuzen": lambda: potuzen_config(width, ff, layers, vocab),
                   "kunulorn": lambda: kunulorn_config(width, ff, layers, vocab, heads),
                   "tebasun": lambda: tebasun_config(width, ff, layers, vocab),
-                  "fupapel": lambda: fupapel_config(width, ff, layers, vocab, heads)}[design]()
+                  "fupapel": lambda: fupapel_config(width, ff, layers, vocab, heads),
+                  "dobepel": lambda: dobepel_config(width, ff, layers, vocab)}[design]()
         ours = _measure(config, prompt_tokens, batch, steps, warmup, kernels)
         twin_config = {"potuzen": lambda: potuzen_config(width, ff, layers, vocab),
                        "kunulorn": lambda: kunulorn_config(width, ff, layers, vocab, heads),
+                       "tebasun": lambda: tebasun_config(width, ff, layers, vocab),
                        "llama": lambda: llama_config(width, ff, layers, vocab, heads)}[beside]()
         twin = _measure(twin_config, prompt_tokens, batch, steps, warmup, kernels)
         result["sizes"][name] = {

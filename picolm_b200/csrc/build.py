@@ -43,6 +43,7 @@ LIBRARIES: Dict[str, List[str]] = {
     "sampling": ["sampling.cu"],
     "recurrent": ["recurrent.cu"],
     "routed": ["routed.cu"],
+    "decay_chunk": ["decay_chunk.cu"],
 }
 HEADERS = ["common.cuh", "tc_common.cuh", "gemm_tc_static.h"]
 
@@ -59,6 +60,9 @@ MORE_BUILDS: List = [("gemm_tc_wide@stream", ["-DPLM_WIDE_STREAM"]),
                      # the gated epilogue with the tanh form of GELU in place of SiLU
                      ("gemm_tc_skinny@gelu", ["-DPLM_GATE_GELU"]), ("gemm_tc_wide@gelu", ["-DPLM_GATE_GELU"]),
                      ("gemm_tc_wide@stream_gelu", ["-DPLM_WIDE_STREAM", "-DPLM_GATE_GELU"]),
+                     # the bf16 store epilogue with the exact GELU (products with an activation and no gate)
+                     ("gemm_tc_skinny@gelu_erf", ["-DPLM_STORE_GELU_ERF"]), ("gemm_tc_wide@gelu_erf", ["-DPLM_STORE_GELU_ERF"]),
+                     ("gemm_tc_wide@stream_gelu_erf", ["-DPLM_WIDE_STREAM", "-DPLM_STORE_GELU_ERF"]),
                      # the gated epilogue with clamped branches and a sloped sigmoid (its constants come with the launch)
                      ("gemm_tc_skinny@clamped", ["-DPLM_GATE_CLAMPED"]), ("gemm_tc_wide@clamped", ["-DPLM_GATE_CLAMPED"]),
                      ("gemm_tc_wide@stream_clamped", ["-DPLM_WIDE_STREAM", "-DPLM_GATE_CLAMPED"])]

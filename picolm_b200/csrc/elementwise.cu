@@ -1451,6 +1451,47 @@ extern "C" int plm_joined_post_pre_norm(float* x, const float* a, const float* b
     return PLM_ERR_DTYPE;
 }
 
+// ------------------------------------------- a QKV product's rows to attention, nothing done to them on the way
+// qkv [T, H*D | G*D | G*Dv] (row stride ld) -> q_out [T, H, hd_c], keys and values into the pages of the cache (head size
+// hd_c); what lies beyond a head's own width is written as zero.  Sizes are counted in pieces of 16 bytes.
+__global__ void heads_store_kernel(const uint4* __restrict__ qkv, long ld, uint4* __restrict__ q_out, uint4* __restrict__ kc,
+                                   uint4* __restrict__ vc, const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
+                                   const int* __restrict__ block_table, int max_pages, int H, int G, int D, int Dv, int hc) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const uint4* row = qkv + (size_t)t * ld;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    uint4* qo = q_out + (size_t)t * H * hc;
+    for (int i = threadIdx.x; i < H * hc; i += blockDim.x) {
+        const int h = i / hc, c = i - h * hc;
+        qo[i] = c < D ? row[h * D + c] : zero;
+    }
+    if (!kc) return;
+    const int pos = PLM_POSITION(tok_pos[t]);
+    const int page = PLM_PAGE_NO(block_table[(size_t)PLM_SEQ_NO(tok_seq[t]) * max_pages + pos / PLM_PAGE]);
+    for (int i = threadIdx.x; i < G * hc; i += blockDim.x) {
+        const int g = i / hc, c = i - g * hc;
+        const size_t at = (((size_t)page * G + g) * PLM_PAGE + pos % PLM_PAGE) * hc + c;
+        kc[at] = c < D ? row[(H + g) * D + c] : zero;
+        vc[at] = c < Dv ? row[(H + G) * D + g * Dv + c] : zero;
+    }
+}
+
+extern "C" int plm_heads_store(const void* qkv, int dtype, long ld, void* q_out, void* kc, void* vc, const int* tok_pos,
+                               const int* tok_seq, const int* block_table, int max_pages, int n_tokens, int H, int G, int D,
+                               int Dv, int hd_c, cudaStream_t stream) {
+    if (n_tokens <= 0) return PLM_OK;
+    const int per = dtype == PLM_F32 ? 4 : 8;          // elements of a piece
+    if (H <= 0 || G <= 0 || D % per || Dv % per || hd_c % per || hd_c < D || hd_c < Dv) return PLM_ERR_SHAPE;
+    if (ld % per || (((uintptr_t)qkv | (uintptr_t)q_out | (uintptr_t)kc | (uintptr_t)vc) & 15)) return PLM_ERR_ALIGN;
+    const int pieces = H * hd_c / per;
+    const int nt = pieces >= 256 ? 256 : 128;
+    return plm_status_of(launch_pdl(heads_store_kernel, dim3(n_tokens), dim3(nt), 0, stream, (const uint4*)qkv, ld / per,
+                                    (uint4*)q_out, (uint4*)kc, (uint4*)vc, tok_pos, tok_seq, block_table, max_pages, H, G, D / per,
+                                    Dv / per, hd_c / per));
+}
+
 // ------------------------------------------------------------------------- an activation without a gate
 // y = 0.5 x (1 + erf(x / sqrt 2)), the exact GELU
 template <typename T>

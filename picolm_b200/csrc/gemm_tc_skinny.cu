@@ -324,6 +324,10 @@ gemm_tc_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
                     v[0] = swiglu_bf16(v[0], u.x, fz.gate_limit, fz.gate_slope); v[1] = swiglu_bf16(v[1], u.y, fz.gate_limit, fz.gate_slope);
                     v[2] = swiglu_bf16(v[2], u.z, fz.gate_limit, fz.gate_slope); v[3] = swiglu_bf16(v[3], u.w, fz.gate_limit, fz.gate_slope);
                 }
+                if (EPI == EPI_STORE) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) v[e] = store_act<OutT>(v[e]);
+                }
                 __nv_bfloat162 o01 = __floats2bfloat162_rn(v[0], v[1]), o23 = __floats2bfloat162_rn(v[2], v[3]);
                 uint2 o;
                 o.x = *reinterpret_cast<uint32_t*>(&o01);
@@ -355,7 +359,7 @@ gemm_tc_skinny_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_co
             if (f >= F) continue;
             float v = received(c, 0, pr);
             if (SCALE) v *= s_scale[c];
-            out[(size_t)t * ldo + f] = from_f32<OutT>(v);
+            out[(size_t)t * ldo + f] = from_f32<OutT>(store_act<OutT>(v));
         } else {
             const int fo = p0 / 2 + row;
             if (fo >= F / 2) continue;
@@ -529,7 +533,7 @@ gemm_tc_skinny_walk_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
                 if (f < F) {
 #pragma unroll
                     for (int j = 0; j < CHUNK; ++j)
-                        if (c + j < T) out[(size_t)(c + j) * ldo + f] = from_f32<OutT>(__uint_as_float(r[j]));
+                        if (c + j < T) out[(size_t)(c + j) * ldo + f] = from_f32<OutT>(store_act<OutT>(__uint_as_float(r[j])));
                 }
             }
             tc_fence_before();

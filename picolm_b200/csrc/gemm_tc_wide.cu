@@ -653,6 +653,12 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
                         get_part(c + 32);
                     }
                     add_parts(r, c, part);
+#ifdef PLM_STORE_GELU_ERF
+                    if (EPI == EPI_STORE && !F32_OUT) {
+#pragma unroll
+                        for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(store_act<OutT>(__uint_as_float(r[i])));
+                    }
+#endif
                     if (EPI == EPI_RESIDUAL && out_by_copies) {
                         // the piece goes to shared memory as the copy engine wants it (a row's eight 16-byte chunks
                         // at places turned by the row's number), and one thread hands it over; two pieces in turn
@@ -905,7 +911,8 @@ __global__ void reduce_splits_kernel(const float* __restrict__ scratch, OutT* __
         if (sizeof(OutT) == 4) {
             *reinterpret_cast<float4*>(reinterpret_cast<float*>(out) + 4 * i) = a;
         } else {
-            __nv_bfloat162 lo = __floats2bfloat162_rn(a.x, a.y), hi = __floats2bfloat162_rn(a.z, a.w);
+            __nv_bfloat162 lo = __floats2bfloat162_rn(store_act<OutT>(a.x), store_act<OutT>(a.y));
+            __nv_bfloat162 hi = __floats2bfloat162_rn(store_act<OutT>(a.z), store_act<OutT>(a.w));
             uint2 o;
             o.x = *reinterpret_cast<uint32_t*>(&lo);
             o.y = *reinterpret_cast<uint32_t*>(&hi);

@@ -235,7 +235,7 @@ struct ScanArgs {
     int n_seqs, H, N, P, heads_per_group;
     int seg_len, max_segs;                // tokens per segment; segments of the longest sequence
     float *seg_state, *seg_decay;         // [seq][segment][H][N][P] and [seq][segment][H][N]
-    int silu;                             // q, k and v pass SiLU as they are read
+    int silu;                             // q, k and v pass SiLU as they are read, rounded to their own type
     int vec8;                             // bf16 rows may be read eight channels at a time (sizes and addresses allow it)
 };
 
@@ -303,10 +303,10 @@ __global__ void __launch_bounds__(SCAN_THREADS, NS <= 8 ? 4 : 1) linear_scan_ker
     auto act8 = [&](float* f) {
         if (silu) {
 #pragma unroll
-            for (int e = 0; e < 8; ++e) f[e] = silu_f(f[e]);
+            for (int e = 0; e < 8; ++e) f[e] = to_f32<T>(from_f32<T>(silu_f(f[e])));
         }
     };
-    auto act = [&](float x) { return silu ? silu_f(x) : x; };
+    auto act = [&](float x) { return silu ? to_f32<T>(from_f32<T>(silu_f(x))) : x; };
     if (vec8) {
         for (int idx = threadIdx.x; idx < TC * 16 * NS; idx += SCAN_THREADS) {
             const int tt = idx / (16 * NS), n = idx % (16 * NS);
@@ -690,11 +690,79 @@ __global__ void gated_norm_kernel(const TI* __restrict__ x, long ldx, const TG* 
     }
 }
 
+// The same for wide groups: a block per (row, group), four columns at a time, the row and its gate in registers between
+// the sum of squares and the results (VPT times four values a thread).
+__device__ __forceinline__ float4 gn_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 gn_load4(const bf16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const __nv_bfloat162 a = *reinterpret_cast<const __nv_bfloat162*>(&u.x), b = *reinterpret_cast<const __nv_bfloat162*>(&u.y);
+    return make_float4(__low2float(a), __high2float(a), __low2float(b), __high2float(b));
+}
+__device__ __forceinline__ void gn_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void gn_store4(bf16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+template <typename TI, typename TG, typename TO, int NT, int VPT>
+__global__ void __launch_bounds__(NT)
+gated_norm_wide_kernel(const TI* __restrict__ x, long ldx, const TG* __restrict__ gate, long ldg, const float* __restrict__ w,
+                       int w_per_group, TO* __restrict__ out, long ldo, int groups, int group, float eps, int gate_mode, int act) {
+    __shared__ float red[33];
+    pdl_launch_dependents();
+    pdl_wait();
+    const long t = blockIdx.x / groups;
+    const int c0 = (int)(blockIdx.x % groups) * group;
+    const TI* xr = x + t * ldx + c0;
+    const TG* gr = gate ? gate + t * ldg + c0 : nullptr;
+    float4 v[VPT], ga[VPT];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        const int c = (threadIdx.x + k * NT) * 4;
+        if (c >= group) continue;
+        v[k] = gn_load4(xr + c);
+        ga[k] = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (gate_mode) {
+            const float4 g = gn_load4(gr + c);
+            ga[k] = act ? make_float4(sigmoid_f(g.x), sigmoid_f(g.y), sigmoid_f(g.z), sigmoid_f(g.w))
+                        : make_float4(silu_f(g.x), silu_f(g.y), silu_f(g.z), silu_f(g.w));
+            if (gate_mode == 1) v[k] = make_float4(v[k].x * ga[k].x, v[k].y * ga[k].y, v[k].z * ga[k].z, v[k].w * ga[k].w);
+        }
+        ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    }
+    const float r = 1.f / sqrtf(block_sum<NT>(ss, red) / (float)group + eps);
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+        const int c = (threadIdx.x + k * NT) * 4;
+        if (c >= group) continue;
+        float4 o = make_float4(v[k].x * r, v[k].y * r, v[k].z * r, v[k].w * r);
+        if (w) {
+            const float4 wv = gn_load4(w + (w_per_group ? c : c0 + c));
+            o = make_float4(o.x * wv.x, o.y * wv.y, o.z * wv.z, o.w * wv.w);
+        }
+        if (gate_mode == 2) o = make_float4(o.x * ga[k].x, o.y * ga[k].y, o.z * ga[k].z, o.w * ga[k].w);
+        gn_store4(out + t * ldo + c0 + c, o);
+    }
+}
+
 template <typename TI, typename TG, typename TO>
 static int gated_norm_launch(const void* x, long ldx, const void* gate, long ldg, const float* w, int w_per_group, void* out,
                              long ldo, int n_rows, int C, int group, float eps, int gate_mode, int act, int do_norm,
                              cudaStream_t stream) {
     const long warps = (long)n_rows * (C / group);
+    // (which kernel runs, and with it the order of the sums, depends on the group's width and on alignments that a model fixes)
+    const auto fits = [](const void* p, long ld, int size) { return (uintptr_t)p % (4 * size) == 0 && ld % 4 == 0; };
+    if (do_norm && group >= 1024 && group <= 16384 && group % 4 == 0 && fits(x, ldx, sizeof(TI)) && fits(out, ldo, sizeof(TO)) &&
+        (!gate || fits(gate, ldg, sizeof(TG))) && (uintptr_t)w % 16 == 0) {
+#define GN_WIDE(NT_, VPT_)                                                                                                   \
+    return plm_status_of(launch_pdl(gated_norm_wide_kernel<TI, TG, TO, NT_, VPT_>, dim3((unsigned)warps), dim3(NT_), 0, stream, \
+                                    (const TI*)x, ldx, (const TG*)gate, ldg, w, w_per_group, (TO*)out, ldo, C / group, group, eps, \
+                                    gate_mode, act))
+        if (group <= 4 * 512) GN_WIDE(512, 1);
+        if (group <= 4 * 1024) GN_WIDE(1024, 1);
+        GN_WIDE(1024, 4);
+#undef GN_WIDE
+    }
     const unsigned grid = (unsigned)((warps * 32 + 255) / 256);
     return plm_status_of(launch_pdl(gated_norm_kernel<TI, TG, TO>, dim3(grid), dim3(256), 0, stream, (const TI*)x, ldx,
                                     (const TG*)gate, ldg, w, w_per_group, (TO*)out, ldo, n_rows, C, group, eps, gate_mode, act,

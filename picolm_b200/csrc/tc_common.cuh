@@ -134,6 +134,15 @@ __device__ __forceinline__ float swiglu_bf16(float g, float u, float limit = 0.f
     return __fdividef(g, 1.0f + e) * u;
 }
 
+// What the bf16 store epilogue applies to a result before it is rounded: nothing, or with -DPLM_STORE_GELU_ERF (a build
+// variant for products with an activation that has no gate behind them) the exact GELU, 0.5 z (1 + erf(z / sqrt 2)).
+template <typename OutT> __device__ __forceinline__ float store_act(float z) {
+#ifdef PLM_STORE_GELU_ERF
+    if (sizeof(OutT) == 2) return 0.5f * z * (1.0f + erff(z * 0.70710678118654752f));
+#endif
+    return z;
+}
+
 template <typename T> __device__ __forceinline__ void store_vec8(T* p, const uint32_t* r);
 template <> __device__ __forceinline__ void store_vec8<float>(float* p, const uint32_t* r) {
     reinterpret_cast<uint4*>(p)[0] = make_uint4(r[0], r[1], r[2], r[3]);

@@ -17,7 +17,7 @@ from .gemm import (PLAIN_ACTIVATIONS, PendingLinear, ScaledRows, gemm_simt, gemm
                    gemm_tc_wide, interleave_gate_up, linear, linear_act, linear_residual_norm, linear_swiglu, pair_pays,
                    residual_norm_supported)
 from .recurrent import (DECAY_CONST, DECAY_SIGMOID, DECAY_STEP, GATE_AFTER_NORM, GATE_BEFORE_NORM, GATE_NONE, causal_conv,  # noqa: F401
-                        delta_prep, delta_scan, diag_scan, gated_norm, head_linear, linear_scan, rglru_gates,
+                        decay_chunk_supported, decay_powers, decay_scan, delta_prep, delta_scan, diag_scan, gated_norm, head_linear, linear_scan, rglru_gates,
                         store_rows_paged, latent_store)
 from .routed import (SortedPairs, moe_align, moe_combine, moe_down, moe_down_tc, moe_gate_up, moe_gate_up_tc,  # noqa: F401
                      moe_gather, moe_max_tiles, moe_tc_supported, route_topk, router_logits)

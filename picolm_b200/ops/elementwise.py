@@ -319,6 +319,18 @@ def qk_norm_rope_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], q_norm: 
     for wn, n, size in ((q_norm, "q_norm", D if per_head else H * D), (k_norm if own_kv else None, "k_norm", D if per_head else G * D)):
         if wn is not None and (wn.dtype != q_out.dtype or wn.shape != (size,) or not wn.is_cuda):
             raise KernelError(f"qk_norm_rope_store: {n} must be [{size}] of {q_out.dtype}")
+    if (rotation is None or rotation.cos is None) and bias is None and q_norm is None and k_norm is None and q_scale is None \
+            and conv is None and own_kv and not values_from_keys and qkv.dtype == q_out.dtype:
+        per = 16 // qkv.element_size()
+        if not (D % per or Dv % per or hd_c % per or qkv.stride(0) % per or qkv.data_ptr() % 16):
+            # nothing is done to the rows on their way: 16 bytes at a time
+            set_bounds("elementwise", n_pages=kv.k.shape[0], n_seqs=kv.block_table.shape[0],
+                       n_positions=kv.block_table.shape[1] * PAGE_TOKENS, device=qkv.device)
+            _check(_fn("elementwise", "plm_heads_store")(
+                _p(qkv), _dt(qkv, "qkv"), qkv.stride(0), _p(q_out), _p(kv.k), _p(kv.v), _p(step.tok_pos), _p(step.tok_seq),
+                _p(kv.block_table), kv.block_table.shape[1], T, H, G, D, Dv, hd_c, _stream()), f"heads_store T={T}",
+                nbytes=(qkv.numel() + T * (H + 2 * G) * hd_c) * qkv.element_size())
+            return
     cos = sin = None
     rot, pairing = 0, "half"
     if rotation is not None and rotation.cos is not None:

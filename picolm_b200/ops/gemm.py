@@ -13,6 +13,10 @@ from .chain import LazyRows
 from .elementwise import gelu_erf
 
 
+# activations without a gate that a product can apply to its own results
+PLAIN_ACTIVATIONS = ("gelu_erf",)
+
+
 def _work(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, extra: int = 0) -> dict:
     """What a product has to move and compute: both operands and the result once, 2 M N K flops."""
     return {"nbytes": a.numel() * a.element_size() + w.numel() * w.element_size() + out.numel() * out.element_size() + extra,
@@ -65,7 +69,9 @@ def _gated_library(name: str, flags: tuple, activation: str):
 
 
 # activation -> (the variant's name, its compile flag)
-_GATE_VARIANTS = {"gelu_tanh": ("gelu", "-DPLM_GATE_GELU"), "swish_clamped": ("clamped", "-DPLM_GATE_CLAMPED")}
+_GATE_VARIANTS = {"gelu_tanh": ("gelu", "-DPLM_GATE_GELU"), "swish_clamped": ("clamped", "-DPLM_GATE_CLAMPED"),
+                  # (not a gate: what the store epilogue applies, see `linear_act`)
+                  "gelu_erf": ("gelu_erf", "-DPLM_STORE_GELU_ERF")}
 
 
 def _set_gate_constants(lib, flags, activation: str, limit: float, slope: float) -> None:
@@ -76,12 +82,14 @@ def _set_gate_constants(lib, flags, activation: str, limit: float, slope: float)
 
 def gemm_tc_skinny(a, w: torch.Tensor, out_dtype: torch.dtype, swiglu: bool = False,
                    out: Optional[torch.Tensor] = None, activation: str = "silu", limit: float = 0.0,
-                   slope: float = 1.0) -> torch.Tensor:
+                   slope: float = 1.0, store_act: Optional[str] = None) -> torch.Tensor:
     """The decode-shaped tensor-core product: a [M <= 64, K] @ w [N, K]^T with the weights on the MMA's 128
     rows and K split over a thread-block cluster whose CTAs add their partial tiles up through distributed
     shared memory.  With `swiglu`, w holds tiles of 64 gate rows followed by their 64 up rows (see
     `interleave_gate_up`) and the result is silu(gate) * up, [M, N/2] in bfloat16.  `a` may be `ScaledRows`
-    (an RMSNorm whose scale is still due): the epilogue then scales each row of the result, in bfloat16."""
+    (an RMSNorm whose scale is still due): the epilogue then scales each row of the result, in bfloat16.  `store_act`
+    (an activation of `PLAIN_ACTIVATIONS`, bfloat16 results): applied to the sums before they are rounded."""
+    _store_act_check(store_act, swiglu, out_dtype)
     scaled = a if isinstance(a, ScaledRows) else None
     if scaled is not None:
         scaled.ready()
@@ -100,7 +108,7 @@ def gemm_tc_skinny(a, w: torch.Tensor, out_dtype: torch.dtype, swiglu: bool = Fa
     n_out = N // 2 if swiglu else N
     if out is None:
         out = torch.empty((M, n_out), dtype=out_dtype, device=a.device)
-    lib, lib_flags = _gated_library("gemm_tc_skinny", (), activation if swiglu else "silu")
+    lib, lib_flags = _gated_library("gemm_tc_skinny", (), activation if swiglu else store_act or "silu")
     if swiglu:
         _set_gate_constants(lib, lib_flags, activation, limit, slope)
     if scaled is not None:
@@ -111,8 +119,13 @@ def gemm_tc_skinny(a, w: torch.Tensor, out_dtype: torch.dtype, swiglu: bool = Fa
         return out
     _check(_fn(lib, "plm_gemm_tc_skinny", lib_flags)(
         _p(a), _p(w), _p(out), _dt(out, "out"), 1 if swiglu else 0, M, N, K, K, K, n_out,
-        _p(status_word(a.device)), _stream()), f"gemm_tc_skinny{'_swiglu' if swiglu else ''} {M}x{N}x{K}", **_work(a, w, out))
+        _p(status_word(a.device)), _stream()), f"gemm_tc_skinny{'_swiglu' if swiglu else '_' + store_act if store_act else ''} {M}x{N}x{K}", **_work(a, w, out))
     return out
+
+
+def _store_act_check(store_act: Optional[str], swiglu: bool, out_dtype: torch.dtype, add: bool = False) -> None:
+    if store_act is not None and (store_act not in PLAIN_ACTIVATIONS or swiglu or add or out_dtype != torch.bfloat16):
+        raise KernelError(f"a product's store epilogue applies {', '.join(PLAIN_ACTIVATIONS)} to bfloat16 results, not {store_act!r} here")
 
 
 class PendingLinear:
@@ -232,14 +245,16 @@ def linear_residual_norm(pending: PendingLinear, x: torch.Tensor, norm_weight: t
 
 def gemm_tc_wide(a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype, swiglu: bool = False,
                  out: Optional[torch.Tensor] = None, pair: bool = False, add: bool = False,
-                 activation: str = "silu", limit: float = 0.0, slope: float = 1.0) -> torch.Tensor:
+                 activation: str = "silu", limit: float = 0.0, slope: float = 1.0,
+                 store_act: Optional[str] = None) -> torch.Tensor:
     """The prompt-shaped tensor-core product: a [M > 64, K] @ w [N, K]^T by a persistent tcgen05 kernel
     (one CTA per SM, two accumulators in tensor memory so that a tile's epilogue overlaps the next
     tile's main loop; where the tiles do not fill one round over the SMs and K is long, the K blocks of all
     tiles are handed out as one stream, cut into equal ranges).  With `swiglu`, w comes from `interleave_gate_up`
     and the result is silu(gate) * up, [M, N/2] in bfloat16.  With `add`, `out` (float32) += the product.
     `pair`: the same by pairs of CTAs on tiles of 256 x 256 (`tcgen05.mma.cta_group::2`: each CTA of a pair
-    loads half of the weight tile)."""
+    loads half of the weight tile).  `store_act`: as `gemm_tc_skinny`'s."""
+    _store_act_check(store_act, swiglu, out_dtype, add)
     _dev(a, "a"), _dev(w, "w")
     M, K = a.shape
     N = w.shape[0]
@@ -256,11 +271,11 @@ def gemm_tc_wide(a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype, swigl
     if out is None:
         out = torch.empty((M, n_out), dtype=out_dtype, device=a.device)
     epilogue = 2 if add else 1 if swiglu else 0
-    name = f"{'_swiglu' if swiglu else '_residual' if add else ''} {M}x{N}x{K}"
+    name = f"{'_swiglu' if swiglu else '_residual' if add else '_' + store_act if store_act else ''} {M}x{N}x{K}"
     work = _work(a, w, out, extra=out.numel() * 4 if add else 0)
     # Shapes whose tiles leave most SMs idle walk K as one stream: that code is in a build variant of the library
     # (compiled when the first such shape comes), with a workspace; everything else runs the plain build.
-    act = activation if swiglu else "silu"
+    act = activation if swiglu else store_act or "silu"
     STREAM_LIB = _gated_library("gemm_tc_wide@stream", ("-DPLM_WIDE_STREAM",), act)
     PLAIN_LIB = _gated_library("gemm_tc_wide", (), act)
     if pair:
@@ -376,14 +391,17 @@ def linear_swiglu(a, w_gate_up: torch.Tensor, defer: bool = False, activation: s
                         limit=limit, slope=slope)
 
 
-PLAIN_ACTIVATIONS = ("gelu_erf",)
-
-
 def linear_act(a, w: torch.Tensor, out_dtype: torch.dtype, activation: str):
-    """act(a [M, K] times w [N, K]^T) -> [M, N]: a product with an activation that has no gate behind it."""
+    """act(a [M, K] times w [N, K]^T) -> [M, N]: a product with an activation that has no gate behind it.  On the
+    tensor cores the activation is applied in the product's epilogue; elsewhere it is a kernel of its own."""
     if activation not in PLAIN_ACTIVATIONS:
         raise KernelError(f"activation {activation!r} without a gate has no kernel; known: {', '.join(PLAIN_ACTIVATIONS)}")
-    return gelu_erf(linear(a, w, out_dtype))
+    x = a.materialize() if isinstance(a, (ScaledRows, LazyRows)) else a
+    if out_dtype == torch.bfloat16 and gemm_tc_supported(x, w):
+        if x.shape[0] <= 64:
+            return gemm_tc_skinny(x, w, out_dtype, store_act=activation)
+        return gemm_tc_wide(x, w, out_dtype, pair=pair_pays(x.shape[0], w.shape[0], x.shape[1], 0), store_act=activation)
+    return gelu_erf(linear(x, w, out_dtype))
 
 
 def linear(a, w: torch.Tensor, out_dtype: torch.dtype, defer: bool = False):

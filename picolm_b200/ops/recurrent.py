@@ -155,6 +155,72 @@ def scan_plan(n_seqs: int, heads: int, key_dim: int, value_dim: int, max_new: in
     return plan
 
 
+DECAY_CHUNK_FROM = 32      # tokens of a step's longest sequence from which a constant decay's recurrence runs chunk by chunk
+DECAY_CHUNK = 64           # tokens of a chunk
+
+
+def decay_powers(decay) -> torch.Tensor:
+    """The table a constant decay's chunks need: d^0 .. d^64 per head, float32 [heads, 65], from the decays as float32
+    in double precision."""
+    d = torch.as_tensor(decay, dtype=torch.float32).to(torch.float64)
+    return torch.stack([d ** i for i in range(DECAY_CHUNK + 1)], dim=1).to(torch.float32).contiguous()
+
+
+def decay_chunk_supported(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, key_dim: int, value_dim: int) -> bool:
+    """Whether `decay_scan` can run these rows chunk by chunk on the tensor cores: bfloat16, a key size that is a multiple
+    of 16 up to 128, a value size that is a multiple of 8, rows on 16-byte boundaries."""
+    return (q.dtype == k.dtype == v.dtype == torch.bfloat16 and key_dim % 16 == 0 and key_dim <= 128 and value_dim % 8 == 0
+            and all(t.data_ptr() % 16 == 0 and t.stride(0) % 8 == 0 for t in (q, k, v)))
+
+
+def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, powers: torch.Tensor,
+               state: torch.Tensor, step, heads: int, key_dim: int, value_dim: int,
+               activation: Optional[str] = None) -> torch.Tensor:
+    """S_t = d_h S_(t-1) + k_t v_t^T, y_t = S_t^T q_t over each sequence's tokens, with one constant decay a head; float32
+    [T, heads * value_dim].  q, k [T, heads * key_dim], v [T, heads * value_dim] (column slices will do); with
+    `activation="silu"` they pass SiLU on their way in.  `decay` float32 [heads], `powers` its table (`decay_powers`);
+    `state` float32 [slots, >= heads * key_dim * value_dim] is carried on.  Steps with prompts in bfloat16 run 64 tokens
+    at a time on the tensor cores where the sizes allow it, everything else token by token (`linear_scan`)."""
+    H, N, P = heads, key_dim, value_dim
+    T = v.shape[0]
+    if step.max_new < DECAY_CHUNK_FROM or not decay_chunk_supported(q, k, v, N, P) or state.stride(0) % 4:
+        return linear_scan(q, k, v, None, DECAY_CONST, decay, None, None, 1.0, 1.0, state, step, H, N, P, activation=activation)
+    ldq, ldk, ldv, lds = _cols(q, "q"), _cols(k, "k"), _cols(v, "v"), _cols(state, "state")
+    if q.shape != (T, H * N) or k.shape != (T, H * N) or v.shape != (T, H * P) or activation not in (None, "silu"):
+        raise KernelError("decay_scan: q, k, v do not have the shapes the head counts imply, or the activation is not known (silu)")
+    _f32(powers, "powers", H * (DECAY_CHUNK + 1))
+    if state.dtype != torch.float32 or state.shape[1] < H * N * P:
+        raise KernelError("decay_scan: the state must be float32 with heads * key_dim * value_dim values a row")
+    y = torch.empty((T, H * P), dtype=torch.float32, device=v.device)
+    seg_len, n_segs = _decay_chunk_plan(step.n_seqs, H, N, P, step.max_new, T)
+    seg_state = torch.empty((step.n_seqs, n_segs, H * N * P), dtype=torch.float32, device=v.device) if n_segs > 1 else None
+    _check(_fn("decay_chunk", "plm_decay_chunk_scan")(
+        _p(q), _p(k), _p(v), ldq, ldk, ldv, _p(powers), _p(state), lds, _p(y), H * P, _p(step.seq_start), _p(step.seq_slot),
+        step.n_seqs, H, N, P, seg_len, n_segs, _p(seg_state), 1 if activation == "silu" else 0, _stream()),
+        f"decay_chunk_scan T={T} H={H} N={N} P={P}" + (f" in {n_segs} segments" if n_segs > 1 else ""),
+        kernels=3 if n_segs > 1 else 1,
+        nbytes=T * (2 * H * N + H * P) * v.element_size() + T * H * P * 4 + 2 * step.n_seqs * H * N * P * 4,
+        flops=2 * T * H * (DECAY_CHUNK // 2 * (N + P) + 2 * N * P))
+    return y
+
+
+_chunk_plans = {}
+
+
+def _decay_chunk_plan(n_seqs: int, heads: int, key_dim: int, value_dim: int, max_new: int, n_tokens: int):
+    key = (n_seqs, heads, key_dim, value_dim, max_new, n_tokens)
+    plan = _chunk_plans.get(key)
+    if plan is None:
+        import ctypes
+        out = (ctypes.c_int * 2)()
+        _fn("decay_chunk", "plm_decay_chunk_plan")(n_seqs, heads, key_dim, value_dim, int(max_new), int(n_tokens),
+                                                   ctypes.cast(out, ctypes.c_void_p))
+        if len(_chunk_plans) > 4096:
+            _chunk_plans.clear()
+        plan = _chunk_plans[key] = (out[0], out[1])
+    return plan
+
+
 GATE_NONE, GATE_BEFORE_NORM, GATE_AFTER_NORM = 0, 1, 2
 _ACTS = {"silu": 0, "sigmoid": 1}
 

@@ -177,6 +177,7 @@ class LightningAttention(_StateMixer):
         self.w_o, self.norm_w = tensors["o"], self._f32(tensors["norm"])
         self.w_h_bytes = self.w_h.numel() * self.w_h.element_size()
         self.decay = torch.tensor([float(x) for x in self.params["decay"]], dtype=torch.float32, device=self.w_o.device)
+        self.powers = ops.decay_powers([float(x) for x in self.params["decay"]]).to(self.w_o.device)
 
     def weight_bytes(self):
         return self.w_h_bytes + self.w_o.numel() * self.w_o.element_size()
@@ -198,9 +199,7 @@ class LightningAttention(_StateMixer):
         if proj is None:
             proj = ops.linear(h, self.w_h, dt)
         q, k, v, g = proj[:, :HN], proj[:, HN:2 * HN], proj[:, 2 * HN:2 * HN + HP], proj[:, 2 * HN + HP:]
-        o = ops.linear_scan(q=q, k=k, v=v, raw=None, mode=ops.DECAY_CONST, p0=self.decay, p1=None, skip=None, q_scale=1.0,
-                            power=1.0, state=cache.state, step=step, heads=self.H, key_dim=self.N, value_dim=self.P,
-                            activation="silu")
+        o = ops.decay_scan(q, k, v, self.decay, self.powers, cache.state, step, self.H, self.N, self.P, activation="silu")
         gated = ops.gated_norm(o, dt, weight=self.norm_w, eps=self.eps, gate=g, gate_mode=ops.GATE_AFTER_NORM,
                                activation="sigmoid")
         return ops.linear(gated, self.w_o, torch.float32, defer=True)
