@@ -12,15 +12,18 @@
 // decayed values) goes in as two bf16 terms, x = hi + lo with hi = bf16(x) and lo = bf16(x - hi), so that it keeps 16
 // bits; the state itself is fp32 in registers from chunk to chunk and in the cache.
 //
-// One block per (sequence, head, 64 value columns, segment): 4 warps, each with a quarter of the state's rows and 16 of
-// the chunk's tokens.  Long prompts are cut into segments that run side by side, in three passes as in recurrent.cu: each
-// segment's own contribution from zero (LOCAL), the state at every segment's start (decay_combine_kernel), and the walk
-// that writes o (FINAL; WHOLE where there is one segment).
+// One block per (sequence, head, 128 value columns, segment), 8 warps.  For o a warp has 16 of the chunk's tokens and half
+// of the columns, for the state 16 of its rows.  A chunk's rows arrive through cp.async while the chunk before is worked
+// on.  Long prompts are cut into segments that run side by side, in three passes as in recurrent.cu: each segment's own
+// contribution from zero (LOCAL), the state at every segment's start (decay_combine_kernel), and the walk that writes o
+// (FINAL; WHOLE where there is one segment).
+//
+// Steps of single tokens take decay_step_kernel, which streams the state through once.
 #include "common.cuh"
 
 namespace {
 
-constexpr int NT = 128, C = 64, PT = 64;
+constexpr int NT = 256, C = 64, PT = 128;
 constexpr int LDV = PT + 8;                            // padded rows: ldmatrix without bank conflicts
 constexpr int POW_N = C + 1;
 constexpr int PASS_WHOLE = 0, PASS_LOCAL = 1, PASS_FINAL = 2;
@@ -59,7 +62,11 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
     hi = bits(h);
     lo = bits(__floats2bfloat162_rn(a - __low2float(h), b - __high2float(h)));
 }
-__device__ __forceinline__ float silu_f(float x) { return x / (1.f + __expf(-x)); }
+__device__ __forceinline__ float silu_f(float x) { return __fdividef(x, 1.f + __expf(-x)); }      // (rounded to bf16 right away)
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool full) {        // 16 bytes, or zeros
+    const int n = full ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
+}
 
 // eight activations of a row: SiLU where asked for, rounded to bf16
 __device__ __forceinline__ uint4 act8(uint4 raw, bool silu) {
@@ -74,12 +81,15 @@ __device__ __forceinline__ uint4 act8(uint4 raw, bool silu) {
 }
 
 template <int NP> constexpr size_t smem_bytes() {
-    return (size_t)(2 * C * (NP + 8) + 3 * C * LDV + 2 * NP * LDV) * sizeof(bf16) + (POW_N + 3) / 4 * 4 * sizeof(float);
+    // activations of q, k, v and the decayed v in two terms; the state in two terms; rows as they arrive; the powers
+    return (size_t)(2 * C * (NP + 8) + 3 * C * LDV + 2 * NP * LDV + C * (2 * NP + PT)) * sizeof(bf16) + (POW_N + 3) / 4 * 4 * sizeof(float);
 }
 
 template <int NP, int PASS>
-__global__ void __launch_bounds__(NT, 2) decay_chunk_kernel(const Args a) {
-    constexpr int LDK = NP + 8, MT = NP / 64, KS = NP / 16;
+__global__ void __launch_bounds__(NT, 1) decay_chunk_kernel(const Args a) {
+    constexpr int LDK = NP + 8, KS = NP / 16;
+    constexpr int ROW_GROUPS = NP / 16, COL_GROUPS = 8 / ROW_GROUPS, SJ = PT / COL_GROUPS / 8;    // a warp's share of the state
+    constexpr int OJ = PT / 2 / 8;                     // a warp's column tiles of o
     extern __shared__ __align__(16) uint8_t smem_raw[];
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);      // [C][LDK]
     bf16* Ks = Qs + C * LDK;                           // [C][LDK]
@@ -88,7 +98,10 @@ __global__ void __launch_bounds__(NT, 2) decay_chunk_kernel(const Args a) {
     bf16* Vlo = Vhi + C * LDV;
     bf16* Shi = Vlo + C * LDV;                         // [NP][LDV]: the state in two terms
     bf16* Slo = Shi + NP * LDV;
-    float* pw = reinterpret_cast<float*>(Slo + NP * LDV);      // [65]
+    bf16* Rq = Slo + NP * LDV;                         // rows as they arrive: q [C][NP], k [C][NP], v [C][PT]
+    bf16* Rk = Rq + C * NP;
+    bf16* Rv = Rk + C * NP;
+    float* pw = reinterpret_cast<float*>(Rv + C * PT); // [65]
     pdl_launch_dependents();
     const int ptiles = (a.P + PT - 1) / PT;
     int bid = blockIdx.x;
@@ -108,45 +121,61 @@ __global__ void __launch_bounds__(NT, 2) decay_chunk_kernel(const Args a) {
     float* sg = PASS == PASS_WHOLE ? nullptr : a.seg_state + (((long)b * a.max_segs + seg) * a.H + h) * N * P;
     const float* init = PASS == PASS_WHOLE ? st : PASS == PASS_FINAL ? sg : nullptr;
 
-    // this warp's rows of the state: n = warp * NP / 4 + 16 mt + lane / 4 (+ 8), columns p0 + 8 j + 2 (lane % 4) (+ 1)
-    const int nr = warp * (NP / 4) + (lane >> 2), pc = (lane & 3) * 2;
-    float S[MT][PT / 8][4];
+    auto request = [&](int base) {                     // the rows of the chunk that starts at token `base`
+        const int n = min(C, t1 - base);
 #pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-        for (int j = 0; j < PT / 8; ++j)
-#pragma unroll
-            for (int hi = 0; hi < 2; ++hi) {
-                const int n = nr + mt * 16 + hi * 8, p = p0 + j * 8 + pc;
-                float2 x = make_float2(0.f, 0.f);
-                if (init && n < N && p < P) x = *reinterpret_cast<const float2*>(init + (long)n * P + p);
-                S[mt][j][2 * hi] = x.x;
-                S[mt][j][2 * hi + 1] = x.y;
-            }
-
-    const bool silu = a.silu;
-    const int l7 = lane & 7, b3 = (lane >> 3) & 1, b4 = lane >> 4;
-    for (int base = t0; base < t1; base += C) {
-        const int n = min(C, t1 - base);               // tokens of this chunk
-        __syncthreads();                               // the chunk before has been read
-        const uint4 zero = make_uint4(0, 0, 0, 0);
-#pragma unroll 4
         for (int idx = threadIdx.x; idx < C * (NP / 8); idx += NT) {
             const int r = idx / (NP / 8), c = (idx % (NP / 8)) * 8;
             const bool in = r < n && c < N;
-            const uint4 kr = in ? *reinterpret_cast<const uint4*>(a.k + (long)(base + r) * a.ldk + (long)h * N + c) : zero;
-            if (PASS != PASS_LOCAL) {
-                const uint4 qr = in ? *reinterpret_cast<const uint4*>(a.q + (long)(base + r) * a.ldq + (long)h * N + c) : zero;
-                *reinterpret_cast<uint4*>(Qs + r * LDK + c) = act8(qr, silu);
-            }
-            *reinterpret_cast<uint4*>(Ks + r * LDK + c) = act8(kr, silu);
+            const long row = in ? base + r : base;
+            const int col = in ? c : 0;
+            cp_async16(smem_u32(Rk + r * NP + c), a.k + row * a.ldk + (long)h * N + col, in);
+            if (PASS != PASS_LOCAL) cp_async16(smem_u32(Rq + r * NP + c), a.q + row * a.ldq + (long)h * N + col, in);
         }
 #pragma unroll
         for (int idx = threadIdx.x; idx < C * (PT / 8); idx += NT) {
             const int r = idx / (PT / 8), c = (idx % (PT / 8)) * 8;
             const bool in = r < n && p0 + c < P;
-            uint4 vr = in ? *reinterpret_cast<const uint4*>(a.v + (long)(base + r) * a.ldv + (long)h * P + p0 + c) : zero;
-            vr = act8(vr, silu);
+            cp_async16(smem_u32(Rv + r * PT + c), a.v + (long)(in ? base + r : base) * a.ldv + (long)h * P + (in ? p0 + c : p0), in);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    request(t0);
+
+    // this warp's piece of the state: rows sr + lane / 4 (+ 8), columns p0 + sc + 8 j + 2 (lane % 4) (+ 1)
+    const int sr = (warp % ROW_GROUPS) * 16, sc = (warp / ROW_GROUPS) * (PT / COL_GROUPS);
+    const int pc = (lane & 3) * 2;
+    float S[SJ][4];
+#pragma unroll
+    for (int j = 0; j < SJ; ++j)
+#pragma unroll
+        for (int hi = 0; hi < 2; ++hi) {
+            const int n = sr + (lane >> 2) + hi * 8, p = p0 + sc + j * 8 + pc;
+            float2 x = make_float2(0.f, 0.f);
+            if (init && n < N && p < P) x = *reinterpret_cast<const float2*>(init + (long)n * P + p);
+            S[j][2 * hi] = x.x;
+            S[j][2 * hi + 1] = x.y;
+        }
+
+    // this warp's piece of o: tokens 16 tg .. 16 tg + 15 of the chunk, columns oc .. oc + 63 (later tokens meet more keys:
+    // the two warps of a scheduler take a late and an early group)
+    const int tg = warp < 4 ? warp : 7 - warp, oc = (warp >> 2) * (PT / 2);
+    const bool silu = a.silu;
+    const int l7 = lane & 7, b3 = (lane >> 3) & 1, b4 = lane >> 4;
+    for (int base = t0; base < t1; base += C) {
+        const int n = min(C, t1 - base);               // tokens of this chunk
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();                               // this chunk's rows are there, the chunk before has been read
+#pragma unroll
+        for (int idx = threadIdx.x; idx < C * (NP / 8); idx += NT) {
+            const int r = idx / (NP / 8), c = (idx % (NP / 8)) * 8;
+            if (PASS != PASS_LOCAL) *reinterpret_cast<uint4*>(Qs + r * LDK + c) = act8(*reinterpret_cast<const uint4*>(Rq + r * NP + c), silu);
+            *reinterpret_cast<uint4*>(Ks + r * LDK + c) = act8(*reinterpret_cast<const uint4*>(Rk + r * NP + c), silu);
+        }
+#pragma unroll
+        for (int idx = threadIdx.x; idx < C * (PT / 8); idx += NT) {
+            const int r = idx / (PT / 8), c = (idx % (PT / 8)) * 8;
+            const uint4 vr = act8(*reinterpret_cast<const uint4*>(Rv + r * PT + c), silu);
             if (PASS != PASS_LOCAL) *reinterpret_cast<uint4*>(Vs + r * LDV + c) = vr;
             const float g = r < n ? pw[n - 1 - r] : 0.f;
             uint32_t hi[4], lo[4];
@@ -160,119 +189,121 @@ __global__ void __launch_bounds__(NT, 2) decay_chunk_kernel(const Args a) {
         }
         if (PASS != PASS_LOCAL) {
 #pragma unroll
-            for (int mt = 0; mt < MT; ++mt)
+            for (int j = 0; j < SJ; ++j)
 #pragma unroll
-                for (int j = 0; j < PT / 8; ++j)
-#pragma unroll
-                    for (int hi = 0; hi < 2; ++hi) {
-                        uint32_t xh, xl;
-                        split2(S[mt][j][2 * hi], S[mt][j][2 * hi + 1], xh, xl);
-                        const int at = (nr + mt * 16 + hi * 8) * LDV + j * 8 + pc;
-                        *reinterpret_cast<uint32_t*>(Shi + at) = xh;
-                        *reinterpret_cast<uint32_t*>(Slo + at) = xl;
-                    }
+                for (int hi = 0; hi < 2; ++hi) {
+                    uint32_t xh, xl;
+                    split2(S[j][2 * hi], S[j][2 * hi + 1], xh, xl);
+                    const int at = (sr + (lane >> 2) + hi * 8) * LDV + sc + j * 8 + pc;
+                    *reinterpret_cast<uint32_t*>(Shi + at) = xh;
+                    *reinterpret_cast<uint32_t*>(Slo + at) = xl;
+                }
         }
         __syncthreads();
-        if (PASS != PASS_LOCAL && warp * 16 < n) {
-            // this warp's 16 tokens: rows warp * 16 + lane / 4 (+ 8)
-            const int tl = warp * 16 + (lane >> 2);
+        if (base + C < t1) request(base + C);
+        if (PASS != PASS_LOCAL && tg * 16 < n && p0 + oc < P) {
+            const int tl = tg * 16 + (lane >> 2);      // this lane's first token; the other is tl + 8
             uint32_t qa[KS][4];
 #pragma unroll
-            for (int ks = 0; ks < KS; ++ks) ldsm_x4(qa[ks], smem_u32(Qs + (warp * 16 + (lane & 15)) * LDK + ks * 16 + b4 * 8));
-            float o[PT / 8][4];
+            for (int ks = 0; ks < KS; ++ks) ldsm_x4(qa[ks], smem_u32(Qs + (tg * 16 + (lane & 15)) * LDK + ks * 16 + b4 * 8));
+            float o[OJ][4];
 #pragma unroll
-            for (int j = 0; j < PT / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+            for (int j = 0; j < OJ; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
 #pragma unroll
             for (int ks = 0; ks < KS; ++ks) {          // S^T q: what comes from the chunks before
 #pragma unroll
-                for (int j = 0; j < PT / 8; j += 2) {
-                    uint32_t bh[4], bl[4];
-                    const int at = (ks * 16 + l7 + b3 * 8) * LDV + j * 8 + b4 * 8;
-                    ldsm_x4_t(bh, smem_u32(Shi + at));
-                    ldsm_x4_t(bl, smem_u32(Slo + at));
-                    mma_bf16(o[j], qa[ks], bh[0], bh[1]);
-                    mma_bf16(o[j + 1], qa[ks], bh[2], bh[3]);
-                    mma_bf16(o[j], qa[ks], bl[0], bl[1]);
-                    mma_bf16(o[j + 1], qa[ks], bl[2], bl[3]);
+                for (int term = 0; term < 2; ++term) {
+                    const bf16* Sx = term ? Slo : Shi;
+                    uint32_t f[OJ / 2][4];
+#pragma unroll
+                    for (int j = 0; j < OJ / 2; ++j)
+                        ldsm_x4_t(f[j], smem_u32(Sx + (ks * 16 + l7 + b3 * 8) * LDV + oc + j * 16 + b4 * 8));
+#pragma unroll
+                    for (int j = 0; j < OJ / 2; ++j) {
+                        mma_bf16(o[2 * j], qa[ks], f[j][0], f[j][1]);
+                        mma_bf16(o[2 * j + 1], qa[ks], f[j][2], f[j][3]);
+                    }
                 }
             }
             const float dlo = pw[tl + 1], dhi = pw[tl + 9];
 #pragma unroll
-            for (int j = 0; j < PT / 8; ++j) {
+            for (int j = 0; j < OJ; ++j) {
                 o[j][0] *= dlo; o[j][1] *= dlo;
                 o[j][2] *= dhi; o[j][3] *= dhi;
             }
 #pragma unroll 1
-            for (int kb = 0; kb <= warp; ++kb) {       // the chunk's own keys, 16 at a time
-                float w[2][4];
+            for (int kb = 0; kb <= tg; ++kb) {         // the chunk's own keys, 16 at a time
+                float w[2][2][4];                      // two sums a tile: even and odd steps of the key size
 #pragma unroll
-                for (int i = 0; i < 2; ++i) w[i][0] = w[i][1] = w[i][2] = w[i][3] = 0.f;
+                for (int i = 0; i < 2; ++i)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) w[0][i][e] = w[1][i][e] = 0.f;
 #pragma unroll
                 for (int ks = 0; ks < KS; ++ks) {
                     uint32_t kf[4];
                     ldsm_x4(kf, smem_u32(Ks + (kb * 16 + l7 + b4 * 8) * LDK + ks * 16 + b3 * 8));
-                    mma_bf16(w[0], qa[ks], kf[0], kf[1]);
-                    mma_bf16(w[1], qa[ks], kf[2], kf[3]);
+                    mma_bf16(w[ks & 1][0], qa[ks], kf[0], kf[1]);
+                    mma_bf16(w[ks & 1][1], qa[ks], kf[2], kf[3]);
                 }
 #pragma unroll
                 for (int i = 0; i < 2; ++i)
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
                         const int dist = tl + (e >> 1) * 8 - (kb * 16 + i * 8 + pc + (e & 1));
-                        w[i][e] = dist >= 0 ? w[i][e] * pw[dist] : 0.f;
+                        w[0][i][e] = dist >= 0 ? (w[0][i][e] + w[1][i][e]) * pw[dist] : 0.f;
                     }
                 uint32_t ah[4], al[4];
-                split2(w[0][0], w[0][1], ah[0], al[0]);
-                split2(w[0][2], w[0][3], ah[1], al[1]);
-                split2(w[1][0], w[1][1], ah[2], al[2]);
-                split2(w[1][2], w[1][3], ah[3], al[3]);
+                split2(w[0][0][0], w[0][0][1], ah[0], al[0]);
+                split2(w[0][0][2], w[0][0][3], ah[1], al[1]);
+                split2(w[0][1][0], w[0][1][1], ah[2], al[2]);
+                split2(w[0][1][2], w[0][1][3], ah[3], al[3]);
+                uint32_t vf[OJ / 2][4];
 #pragma unroll
-                for (int j = 0; j < PT / 8; j += 2) {
-                    uint32_t vf[4];
-                    ldsm_x4_t(vf, smem_u32(Vs + (kb * 16 + l7 + b3 * 8) * LDV + j * 8 + b4 * 8));
-                    mma_bf16(o[j], ah, vf[0], vf[1]);
-                    mma_bf16(o[j + 1], ah, vf[2], vf[3]);
-                    mma_bf16(o[j], al, vf[0], vf[1]);
-                    mma_bf16(o[j + 1], al, vf[2], vf[3]);
+                for (int j = 0; j < OJ / 2; ++j)
+                    ldsm_x4_t(vf[j], smem_u32(Vs + (kb * 16 + l7 + b3 * 8) * LDV + oc + j * 16 + b4 * 8));
+#pragma unroll
+                for (int j = 0; j < OJ / 2; ++j) {
+                    mma_bf16(o[2 * j], ah, vf[j][0], vf[j][1]);
+                    mma_bf16(o[2 * j + 1], ah, vf[j][2], vf[j][3]);
+                }
+#pragma unroll
+                for (int j = 0; j < OJ / 2; ++j) {
+                    mma_bf16(o[2 * j], al, vf[j][0], vf[j][1]);
+                    mma_bf16(o[2 * j + 1], al, vf[j][2], vf[j][3]);
                 }
             }
 #pragma unroll
             for (int hi = 0; hi < 2; ++hi) {
                 const int t = tl + hi * 8;
                 if (t >= n) continue;
-                float* yr = a.y + (long)(base + t) * a.ldy + (long)h * P + p0 + pc;
+                float* yr = a.y + (long)(base + t) * a.ldy + (long)h * P + p0 + oc + pc;
 #pragma unroll
-                for (int j = 0; j < PT / 8; ++j)
-                    if (p0 + j * 8 < P) *reinterpret_cast<float2*>(yr + j * 8) = make_float2(o[j][2 * hi], o[j][2 * hi + 1]);
+                for (int j = 0; j < OJ; ++j)
+                    if (p0 + oc + j * 8 < P) *reinterpret_cast<float2*>(yr + j * 8) = make_float2(o[j][2 * hi], o[j][2 * hi + 1]);
             }
         }
         // the state: d^n S + K^T (decayed V)
         const float dn = pw[n];
 #pragma unroll
-        for (int mt = 0; mt < MT; ++mt)
+        for (int j = 0; j < SJ; ++j)
 #pragma unroll
-            for (int j = 0; j < PT / 8; ++j)
+            for (int e = 0; e < 4; ++e) S[j][e] *= dn;
+        if (p0 + sc < P) {
 #pragma unroll
-                for (int e = 0; e < 4; ++e) S[mt][j][e] *= dn;
+            for (int sb = 0; sb < C / 16; ++sb) {
+                if (sb * 16 >= n) break;
+                uint32_t ka[4];
+                ldsm_x4_t(ka, smem_u32(Ks + (sb * 16 + b4 * 8 + l7) * LDK + sr + b3 * 8));
 #pragma unroll
-        for (int sb = 0; sb < C / 16; ++sb) {
-            if (sb * 16 >= n) break;
-            uint32_t ka[MT][4];
+                for (int term = 0; term < 2; ++term) {
+                    const bf16* Vx = term ? Vlo : Vhi;
 #pragma unroll
-            for (int mt = 0; mt < MT; ++mt)
-                ldsm_x4_t(ka[mt], smem_u32(Ks + (sb * 16 + b4 * 8 + l7) * LDK + warp * (NP / 4) + mt * 16 + b3 * 8));
-#pragma unroll
-            for (int j = 0; j < PT / 8; j += 2) {
-                uint32_t vh[4], vl[4];
-                const int at = (sb * 16 + l7 + b3 * 8) * LDV + j * 8 + b4 * 8;
-                ldsm_x4_t(vh, smem_u32(Vhi + at));
-                ldsm_x4_t(vl, smem_u32(Vlo + at));
-#pragma unroll
-                for (int mt = 0; mt < MT; ++mt) {
-                    mma_bf16(S[mt][j], ka[mt], vh[0], vh[1]);
-                    mma_bf16(S[mt][j + 1], ka[mt], vh[2], vh[3]);
-                    mma_bf16(S[mt][j], ka[mt], vl[0], vl[1]);
-                    mma_bf16(S[mt][j + 1], ka[mt], vl[2], vl[3]);
+                    for (int j = 0; j < SJ / 2; ++j) {
+                        uint32_t f[4];
+                        ldsm_x4_t(f, smem_u32(Vx + (sb * 16 + l7 + b3 * 8) * LDV + sc + j * 16 + b4 * 8));
+                        mma_bf16(S[2 * j], ka, f[0], f[1]);
+                        mma_bf16(S[2 * j + 1], ka, f[2], f[3]);
+                    }
                 }
             }
         }
@@ -280,15 +311,74 @@ __global__ void __launch_bounds__(NT, 2) decay_chunk_kernel(const Args a) {
     float* dst = PASS == PASS_LOCAL ? sg : (PASS == PASS_WHOLE || seg == n_segs - 1) ? st : nullptr;
     if (dst) {
 #pragma unroll
-        for (int mt = 0; mt < MT; ++mt)
+        for (int j = 0; j < SJ; ++j)
 #pragma unroll
-            for (int j = 0; j < PT / 8; ++j)
+            for (int hi = 0; hi < 2; ++hi) {
+                const int n = sr + (lane >> 2) + hi * 8, p = p0 + sc + j * 8 + pc;
+                if (n < N && p < P) *reinterpret_cast<float2*>(dst + (long)n * P + p) = make_float2(S[j][2 * hi], S[j][2 * hi + 1]);
+            }
+    }
+}
+
+// One token for each sequence: S <- d S + k v^T and o = S^T q in one pass over the state.  A block per (64 value columns,
+// head, sequence); 16 threads hold four columns each of a row, 16 rows at a time; the rows' shares of o are added in
+// the order of the 16 row groups.  q, k and v are fp32 here, their activations rounded to the run's type.
+constexpr int STEP_NT = 256, STEP_COLS = 64;
+template <typename T>
+__global__ void __launch_bounds__(STEP_NT)
+decay_step_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, long ldq, long ldk, long ldv,
+                  const float* __restrict__ decay, float* __restrict__ state, long state_stride, float* __restrict__ y, long ldy,
+                  const int* __restrict__ seq_slot, int N, int P, int silu) {
+    extern __shared__ float step_sm[];                 // q [N], k [N], shares [16][64]
+    float* qs = step_sm;
+    float* ks = qs + N;
+    float4* share = reinterpret_cast<float4*>(step_sm + (2 * N + 3) / 4 * 4);
+    pdl_launch_dependents();
+    pdl_wait();
+    const int b = blockIdx.z, h = blockIdx.y;
+    auto act = [&](float x) { return silu ? to_f32<T>(from_f32<T>(x / (1.f + expf(-x)))) : x; };
+    for (int i = threadIdx.x; i < N; i += STEP_NT) {
+        qs[i] = act(to_f32<T>(q[b * ldq + (long)h * N + i]));
+        ks[i] = act(to_f32<T>(k[b * ldk + (long)h * N + i]));
+    }
+    const int cq = threadIdx.x & 15, rg = threadIdx.x >> 4;
+    const int p = blockIdx.x * STEP_COLS + cq * 4;
+    const float d = decay[h];
+    float4 vv = make_float4(0.f, 0.f, 0.f, 0.f);
+    const bool in = p < P;                             // P is a multiple of 4
+    if (in) {
+        const T* vr = v + b * ldv + (long)h * P + p;
+        vv = make_float4(act(to_f32<T>(vr[0])), act(to_f32<T>(vr[1])), act(to_f32<T>(vr[2])), act(to_f32<T>(vr[3])));
+    }
+    __syncthreads();
+    float* st = state + (long)seq_slot[b] * state_stride + (long)h * N * P + p;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (in) {
+        for (int n0 = rg; n0 < N; n0 += 128) {         // eight rows' values are asked for at once
+            float4 x[8];
 #pragma unroll
-                for (int hi = 0; hi < 2; ++hi) {
-                    const int n = nr + mt * 16 + hi * 8, p = p0 + j * 8 + pc;
-                    if (n < N && p < P)
-                        *reinterpret_cast<float2*>(dst + (long)n * P + p) = make_float2(S[mt][j][2 * hi], S[mt][j][2 * hi + 1]);
-                }
+            for (int i = 0; i < 8; ++i)
+                if (n0 + 16 * i < N) x[i] = *reinterpret_cast<const float4*>(st + (long)(n0 + 16 * i) * P);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const int n = n0 + 16 * i;
+                if (n >= N) break;
+                const float kn = ks[n], qn = qs[n];
+                x[i] = make_float4(fmaf(d, x[i].x, kn * vv.x), fmaf(d, x[i].y, kn * vv.y), fmaf(d, x[i].z, kn * vv.z), fmaf(d, x[i].w, kn * vv.w));
+                *reinterpret_cast<float4*>(st + (long)n * P) = x[i];
+                acc = make_float4(fmaf(x[i].x, qn, acc.x), fmaf(x[i].y, qn, acc.y), fmaf(x[i].z, qn, acc.z), fmaf(x[i].w, qn, acc.w));
+            }
+        }
+    }
+    share[rg * 16 + cq] = acc;
+    __syncthreads();
+    if (threadIdx.x < STEP_COLS) {
+        const int c = threadIdx.x, pp = blockIdx.x * STEP_COLS + c;
+        const float* sh = reinterpret_cast<const float*>(share) + c;
+        float sum = sh[0];
+#pragma unroll
+        for (int r = 1; r < 16; ++r) sum += sh[r * STEP_COLS];
+        if (pp < P) y[b * ldy + (long)h * P + pp] = sum;
     }
 }
 
@@ -351,7 +441,7 @@ int launch(const Args& a, cudaStream_t stream) {
 
 // How a step of `n_tokens` tokens whose longest sequence brings `max_new` of them is cut: out[0] tokens per segment (a
 // multiple of 64), out[1] segments of the longest sequence (1: one pass, no scratch memory): as many as make one wave of
-// blocks at two an SM, each of at least 128 tokens, and no more than keep the scratch memory under 1 GiB.
+// blocks at one an SM, each of at least 128 tokens, and no more than keep the scratch memory under 1 GiB.
 extern "C" int plm_decay_chunk_plan(int n_seqs, int H, int N, int P, int max_new, int n_tokens, int* out) {
     out[0] = max_new > 0 ? (max_new + C - 1) / C * C : C;
     out[1] = 1;
@@ -361,7 +451,7 @@ extern "C" int plm_decay_chunk_plan(int n_seqs, int H, int N, int P, int max_new
     if (busy > n_seqs) busy = n_seqs;
     if (busy < 1) busy = 1;
     const long blocks = busy * H * ((P + PT - 1) / PT);
-    long segs = 2L * PLM_SM_COUNT / blocks;
+    long segs = (long)PLM_SM_COUNT / blocks;
     if (segs > max_new / (2 * C)) segs = max_new / (2 * C);
     const long state_bytes = (long)n_seqs * H * N * P * 4;
     while (segs > 1 && segs * state_bytes > (1L << 30)) --segs;
@@ -391,4 +481,22 @@ extern "C" int plm_decay_chunk_scan(const void* q, const void* k, const void* v,
     a.n_seqs = n_seqs, a.H = H, a.N = N, a.P = P, a.seg_len = seg_len, a.max_segs = max_segs < 1 ? 1 : max_segs;
     a.silu = silu, a.seg_state = seg_state;
     return N <= 64 ? launch<64>(a, stream) : launch<128>(a, stream);
+}
+
+// One token for each of n_seqs sequences (token b of q, k, v is sequence b's): `decay` [H] fp32, the rest as above; any
+// element type, N and P (a multiple of 4; state rows and heads on 16-byte boundaries).
+extern "C" int plm_decay_step(const void* q, const void* k, const void* v, int dtype, long ldq, long ldk, long ldv,
+                              const float* decay, float* state, long state_stride, float* y, long ldy, const int* seq_slot,
+                              int n_seqs, int H, int N, int P, int silu, cudaStream_t stream) {
+    if (n_seqs <= 0 || H <= 0 || N <= 0 || N > 4096 || P <= 0 || P % 4 || n_seqs > 65535 || H > 65535) return PLM_ERR_SHAPE;
+    if (((uintptr_t)state & 15) || state_stride % 4) return PLM_ERR_ALIGN;
+    const dim3 grid((P + STEP_COLS - 1) / STEP_COLS, H, n_seqs);
+    const size_t smem = ((size_t)(2 * N + 3) / 4 * 4 + 16 * STEP_COLS) * sizeof(float);
+    if (dtype == PLM_F32)
+        return plm_status_of(launch_pdl(decay_step_kernel<float>, grid, dim3(STEP_NT), smem, stream, (const float*)q, (const float*)k,
+                                        (const float*)v, ldq, ldk, ldv, decay, state, state_stride, y, ldy, seq_slot, N, P, silu));
+    if (dtype == PLM_BF16)
+        return plm_status_of(launch_pdl(decay_step_kernel<bf16>, grid, dim3(STEP_NT), smem, stream, (const bf16*)q, (const bf16*)k,
+                                        (const bf16*)v, ldq, ldk, ldv, decay, state, state_stride, y, ldy, seq_slot, N, P, silu));
+    return PLM_ERR_DTYPE;
 }

@@ -21,6 +21,7 @@ _SIGNATURES = {
     "plm_embed_pair": [_vp, _vp, _vp, _i, _vp, _l, _vp, _vp, _vp, _vp, _i, _i, _i, _l, _l, _l, _f, _vp],
     "plm_joined_post_pre_norm": [_vp, _vp, _vp, _vp, _vp, _f, _vp, _vp, _vp, _i, _i, _i, _f, _f, _f, _f, _vp],
     "plm_heads_store": [_vp, _i, _l, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
+    "plm_decay_step": [_vp, _vp, _vp, _i, _l, _l, _l, _vp, _vp, _l, _vp, _l, _vp, _i, _i, _i, _i, _i, _vp],
     "plm_decay_chunk_plan": [_i, _i, _i, _i, _i, _i, _vp],
     "plm_decay_chunk_scan": [_vp, _vp, _vp, _l, _l, _l, _vp, _vp, _l, _vp, _l, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _i, _vp],
     "plm_gelu_erf": [_vp, _vp, _i, _l, _vp],

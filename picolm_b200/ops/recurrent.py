@@ -180,9 +180,12 @@ def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.T
     [T, heads * value_dim].  q, k [T, heads * key_dim], v [T, heads * value_dim] (column slices will do); with
     `activation="silu"` they pass SiLU on their way in.  `decay` float32 [heads], `powers` its table (`decay_powers`);
     `state` float32 [slots, >= heads * key_dim * value_dim] is carried on.  Steps with prompts in bfloat16 run 64 tokens
-    at a time on the tensor cores where the sizes allow it, everything else token by token (`linear_scan`)."""
+    at a time on the tensor cores where the sizes allow it, steps of single tokens stream the state through once,
+    everything else goes token by token (`linear_scan`)."""
     H, N, P = heads, key_dim, value_dim
     T = v.shape[0]
+    if step.is_decode and step.n_tokens == step.n_seqs and P % 4 == 0 and state.stride(0) % 4 == 0 and state.data_ptr() % 16 == 0:
+        return _decay_step(q, k, v, decay, state, step, H, N, P, activation)
     if step.max_new < DECAY_CHUNK_FROM or not decay_chunk_supported(q, k, v, N, P) or state.stride(0) % 4:
         return linear_scan(q, k, v, None, DECAY_CONST, decay, None, None, 1.0, 1.0, state, step, H, N, P, activation=activation)
     ldq, ldk, ldv, lds = _cols(q, "q"), _cols(k, "k"), _cols(v, "v"), _cols(state, "state")
@@ -201,6 +204,23 @@ def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.T
         kernels=3 if n_segs > 1 else 1,
         nbytes=T * (2 * H * N + H * P) * v.element_size() + T * H * P * 4 + 2 * step.n_seqs * H * N * P * 4,
         flops=2 * T * H * (DECAY_CHUNK // 2 * (N + P) + 2 * N * P))
+    return y
+
+
+def _decay_step(q, k, v, decay, state, step, H, N, P, activation):
+    ldq, ldk, ldv, lds = _cols(q, "q"), _cols(k, "k"), _cols(v, "v"), _cols(state, "state")
+    T = v.shape[0]
+    if (q.shape != (T, H * N) or k.shape != (T, H * N) or v.shape != (T, H * P) or not (q.dtype == k.dtype == v.dtype)
+            or activation not in (None, "silu")):
+        raise KernelError("decay_scan: q, k, v do not have the shapes the head counts imply, differ in type, or the activation is not known (silu)")
+    _f32(decay, "decay", H)
+    if state.dtype != torch.float32 or state.shape[1] < H * N * P:
+        raise KernelError("decay_scan: the state must be float32 with heads * key_dim * value_dim values a row")
+    y = torch.empty((T, H * P), dtype=torch.float32, device=v.device)
+    _check(_fn("decay_chunk", "plm_decay_step")(
+        _p(q), _p(k), _p(v), _dt(v, "v"), ldq, ldk, ldv, _p(decay), _p(state), lds, _p(y), H * P, _p(step.seq_slot), T, H, N, P,
+        1 if activation == "silu" else 0, _stream()), f"decay_step T={T} H={H} N={N} P={P}",
+        nbytes=T * H * (8 * N * P + (2 * N + P) * v.element_size() + 4 * P), flops=4 * T * H * N * P)
     return y
 
 
