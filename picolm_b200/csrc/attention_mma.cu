@@ -170,9 +170,9 @@ __device__ __forceinline__ void pv_tile_sw(float (&o)[HD / 8][4], const float (&
 // Scale, mask and fold one block of scores into the running softmax of the thread's two rows
 // (row_lo = lane/4, row_hi = lane/4 + 8).  Scores become probabilities in place.
 // key_base: position of the block's first key; pos_*: each row's own position (keys above it are
-// masked); lo_*: first key of each row's window; keys before `keep` are seen whatever the window.
-// BIAS: a score also loses slope_* (in log2 units) times the distance of its key.
-template <int NKT, bool BIAS>
+// masked); lo_*: first key of each row's window.  EXTRA: keys before `keep` are seen whatever the window, and a score
+// loses slope_* (in log2 units) times the distance of its key.
+template <int NKT, bool EXTRA>
 __device__ __forceinline__ void softmax_block(float (&s)[NKT][4], float (&o)[HD / 8][4], float (&m)[2], float (&l)[2],
                                               float scale_log2, int key_base, int pos_lo, int pos_hi, int lo_lo,
                                               int lo_hi, int lane, int keep, float slope_lo, float slope_hi) {
@@ -183,9 +183,10 @@ __device__ __forceinline__ void softmax_block(float (&s)[NKT][4], float (&o)[HD 
         for (int e = 0; e < 4; ++e) {
             const int key = key_base + j * 8 + (lane & 3) * 2 + (e & 1);
             const int hi = e >> 1;
-            const bool ok = hi ? (key <= pos_hi && (key >= lo_hi || key < keep)) : (key <= pos_lo && (key >= lo_lo || key < keep));
+            bool ok = hi ? (key <= pos_hi && key >= lo_hi) : (key <= pos_lo && key >= lo_lo);
+            if (EXTRA) ok = hi ? (key <= pos_hi && (key >= lo_hi || key < keep)) : (key <= pos_lo && (key >= lo_lo || key < keep));
             float raw = s[j][e] * scale_log2;
-            if (BIAS) raw = fmaf(s[j][e], scale_log2, (hi ? slope_hi : slope_lo) * (float)(key - (hi ? pos_hi : pos_lo)));
+            if (EXTRA) raw = fmaf(s[j][e], scale_log2, (hi ? slope_hi : slope_lo) * (float)(key - (hi ? pos_hi : pos_lo)));
             const float v = ok ? raw : -INFINITY;
             s[j][e] = v;
             mx[hi] = fmaxf(mx[hi], v);
@@ -239,6 +240,9 @@ __device__ __forceinline__ float sink_inverse(float m, float l, float sink) {
 constexpr int PF_STAGES = 2;
 constexpr size_t PF_SMEM = (size_t)(1 + 2 * PF_STAGES) * TILE_ELEMS * sizeof(bf16);
 
+// EXTRA (here and in the decode kernel): instances for kept first positions and slopes; without it `keep` and `slopes` are
+// not looked at.
+template <bool EXTRA>
 __global__ void __launch_bounds__(NT)
 attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const bf16* __restrict__ vc,
                     bf16* __restrict__ out, const int* __restrict__ seq_start, const int* __restrict__ seq_kv_len,
@@ -282,9 +286,9 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, con
     const int pos_min = pos0 + row0 / R, pos_max = pos0 + last_row / R;
     const int first_key = plm_first_key(pos_min, window);
     const int page_first = first_key / PLM_PAGE, page_last = pos_max / PLM_PAGE;
-    const int n_kept = plm_kept_pages(first_key, keep);     // pages of kept first positions in front of the window's
+    const int n_kept = EXTRA ? plm_kept_pages(first_key, keep) : 0;     // pages of kept first positions in front of the window's
     const int n_pages = n_kept + page_last - page_first + 1;
-    auto page_at = [&](int i) { return i < n_kept ? i : page_first + i - n_kept; };
+    auto page_at = [&](int i) { return EXTRA && i < n_kept ? i : page_first + i - n_kept; };
 
     auto issue = [&](int i) {                          // the i-th page of this tile's walk into stage i % PF_STAGES
         const size_t base = ((size_t)PLM_PAGE_NO(pages[page_at(i)]) * G + g) * PLM_PAGE * HD;
@@ -302,7 +306,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, con
     const int lo_lo = plm_first_key(pos_lo, window);
     const int lo_hi = plm_first_key(pos_hi, window);
     float slope_lo = 0.f, slope_hi = 0.f;
-    if (slopes) {
+    if (EXTRA && slopes) {
         if (r_lo < rows_total) slope_lo = slopes[g * R + r_lo % R] * LOG2E;
         if (r_hi < rows_total) slope_hi = slopes[g * R + r_hi % R] * LOG2E;
     }
@@ -327,10 +331,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, con
 #pragma unroll
             for (int j = 0; j < 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
             qk_tile<8>(s, q_s + warp * 16 * LDS, kt, 0, lane, lane & 15);
-            if (slopes)
-                softmax_block<8, true>(s, o, m, l, scale_log2, key_base, pos_lo, pos_hi, lo_lo, lo_hi, lane, keep, slope_lo, slope_hi);
-            else
-                softmax_block<8, false>(s, o, m, l, scale_log2, key_base, pos_lo, pos_hi, lo_lo, lo_hi, lane, keep, 0.f, 0.f);
+            softmax_block<8, EXTRA>(s, o, m, l, scale_log2, key_base, pos_lo, pos_hi, lo_lo, lo_hi, lane, keep, slope_lo, slope_hi);
             pv_tile<8>(o, s, vt, 0, lane);
         }
         __syncthreads();                               // the stage may be overwritten by the next issue
@@ -416,7 +417,7 @@ struct PageMaps {               // the TMA form: the caches as [pages * G * 64 r
     CUtensorMap k, v;
 };
 
-template <bool CLUSTER, bool ROPE, bool TMA>
+template <bool CLUSTER, bool ROPE, bool TMA, bool EXTRA>
 __global__ void __launch_bounds__(NT)
 attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const bf16* __restrict__ vc,
                    bf16* __restrict__ out, float* __restrict__ ws_o, float* __restrict__ ws_ml,
@@ -456,12 +457,12 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, cons
     const int page_first = lo / PLM_PAGE, page_last = pos / PLM_PAGE;
     // the walk: the pages of kept first positions that lie before the window's, then the window's; a split takes `per`
     // of them in a row, from the w_begin-th on
-    const int n_kept = plm_kept_pages(lo, keep);
+    const int n_kept = EXTRA ? plm_kept_pages(lo, keep) : 0;
     const int total_pages = n_kept + page_last - page_first + 1;
     const int per = (total_pages + n_splits - 1) / n_splits;
     const int w_begin = split * per;
     const int n_pages = min(total_pages, w_begin + per) - w_begin;
-    auto page_at = [&](int i) { return w_begin + i < n_kept ? w_begin + i : page_first + w_begin + i - n_kept; };
+    auto page_at = [&](int i) { return EXTRA && w_begin + i < n_kept ? w_begin + i : page_first + w_begin + i - n_kept; };
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int* pages = block_table + (size_t)PLM_SEQ_NO(tok_seq[t]) * max_pages;
 
@@ -530,15 +531,12 @@ attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, cons
     for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
     float slope_lo = 0.f, slope_hi = 0.f;               // of this lane's two rows (heads)
-    if (slopes) {
+    if (EXTRA && slopes) {
         if ((lane >> 2) < n_rows) slope_lo = slopes[h0 + (lane >> 2)] * LOG2E;
         if ((lane >> 2) + 8 < n_rows) slope_hi = slopes[h0 + (lane >> 2) + 8] * LOG2E;
     }
     auto fold = [&](float (&s)[2][4], int key_base) {
-        if (slopes)
-            softmax_block<2, true>(s, o, m, l, scale_log2, key_base, pos, pos, lo, lo, lane, keep, slope_lo, slope_hi);
-        else
-            softmax_block<2, false>(s, o, m, l, scale_log2, key_base, pos, pos, lo, lo, lane, keep, 0.f, 0.f);
+        softmax_block<2, EXTRA>(s, o, m, l, scale_log2, key_base, pos, pos, lo, lo, lane, keep, slope_lo, slope_hi);
     };
 
     for (int i = 0; i < n_pages; ++i) {
@@ -821,13 +819,14 @@ extern "C" int plm_attn_prefill(const void* q, const void* kc, const void* vc, v
     if (H <= 0 || G <= 0 || H % G || n_seqs > 65535 || G > 65535 || keep < 0) return PLM_ERR_SHAPE;
     static bool configured = false;
     if (!configured) {
-        int rc = set_smem(attn_prefill_kernel, PF_SMEM);
+        int rc = set_smem(attn_prefill_kernel<false>, PF_SMEM);
+        if (rc == PLM_OK) rc = set_smem(attn_prefill_kernel<true>, PF_SMEM);
         if (rc != PLM_OK) return rc;
         configured = true;
     }
     const int R = H / G;
     dim3 grid(((size_t)max_new * R + 63) / 64, G, n_seqs);
-    return plm_status_of(launch_pdl(attn_prefill_kernel, grid, dim3(NT), PF_SMEM, stream, (const bf16*)q, (const bf16*)kc,
+    return plm_status_of(launch_pdl(keep || slopes ? attn_prefill_kernel<true> : attn_prefill_kernel<false>, grid, dim3(NT), PF_SMEM, stream, (const bf16*)q, (const bf16*)kc,
                                     (const bf16*)vc, (bf16*)out, seq_start, seq_kv_len, block_table, max_pages, H, G,
                                     scale * LOG2E, window, sink, keep, slopes));
 }
@@ -849,10 +848,14 @@ extern "C" int plm_attn_decode(const void* q, const void* kc, const void* vc, vo
     if (n_tokens <= 0) return PLM_OK;
     if (H <= 0 || G <= 0 || H % G || n_splits < 1 || n_tokens > 65535 || keep < 0) return PLM_ERR_SHAPE;
     constexpr bool TMA = HAS_TMA;
+    const bool extra = keep > 0 || slopes != nullptr;
     static bool configured = false;
     if (!configured) {
-        int rc = set_smem(attn_decode_kernel<false, false, TMA>, TMA ? dc_smem_tma(16) : DC_SMEM);
-        if (rc == PLM_OK) rc = set_smem(attn_decode_kernel<true, false, TMA>, TMA ? dc_smem_tma(16) : DC_SMEM);
+        const size_t most = TMA ? dc_smem_tma(16) : DC_SMEM;
+        int rc = set_smem(attn_decode_kernel<false, false, TMA, false>, most);
+        if (rc == PLM_OK) rc = set_smem(attn_decode_kernel<true, false, TMA, false>, most);
+        if (rc == PLM_OK) rc = set_smem(attn_decode_kernel<false, false, TMA, true>, most);
+        if (rc == PLM_OK) rc = set_smem(attn_decode_kernel<true, false, TMA, true>, most);
         if (rc != PLM_OK) return rc;
         configured = true;
     }
@@ -870,14 +873,16 @@ extern "C" int plm_attn_decode(const void* q, const void* kc, const void* vc, vo
     if (n_splits > MERGE_MAX_SPLITS) return PLM_ERR_SHAPE;
     if (n_splits > 1 && !workspace) {                       // the splits merge inside their cluster
         if (n_splits > DC_MAX_CLUSTER) return PLM_ERR_SHAPE;
-        return plm_status_of(launch_pdl_cluster(attn_decode_kernel<true, false, TMA>, grid, dim3(NT), dim3(n_splits, 1, 1), smem,
+        return plm_status_of(launch_pdl_cluster(extra ? attn_decode_kernel<true, false, TMA, true>
+                                                      : attn_decode_kernel<true, false, TMA, false>, grid, dim3(NT), dim3(n_splits, 1, 1), smem,
                                                 stream, (const bf16*)q, (const bf16*)kc, (const bf16*)vc, (bf16*)out,
                                                 (float*)nullptr, (float*)nullptr, tok_pos, tok_seq, block_table,
                                                 max_pages, H, G, scale * LOG2E, window, row_groups, Rotary{}, q_rows, maps, status, sink, keep, slopes));
     }
     float* ws_o = workspace;
     float* ws_ml = workspace ? workspace + (size_t)n_tokens * H * n_splits * HD : nullptr;
-    int rc = plm_status_of(launch_pdl(attn_decode_kernel<false, false, TMA>, grid, dim3(NT), smem, stream, (const bf16*)q,
+    int rc = plm_status_of(launch_pdl(extra ? attn_decode_kernel<false, false, TMA, true>
+                                            : attn_decode_kernel<false, false, TMA, false>, grid, dim3(NT), smem, stream, (const bf16*)q,
                                       (const bf16*)kc, (const bf16*)vc, (bf16*)out, ws_o, ws_ml, tok_pos, tok_seq,
                                       block_table, max_pages, H, G, scale * LOG2E, window, row_groups, Rotary{}, q_rows, maps, status, sink, keep, slopes));
     if (rc != PLM_OK || n_splits == 1) return rc;
@@ -898,8 +903,8 @@ extern "C" int plm_attn_decode_rope(const void* qkv, void* kc, void* vc, void* o
     constexpr bool TMA = HAS_TMA;
     static bool configured = false;
     if (!configured) {
-        int rc = set_smem(attn_decode_kernel<false, true, TMA>, TMA ? dc_smem_tma(16) : DC_SMEM);
-        if (rc == PLM_OK) rc = set_smem(attn_decode_kernel<true, true, TMA>, TMA ? dc_smem_tma(16) : DC_SMEM);
+        int rc = set_smem(attn_decode_kernel<false, true, TMA, false>, TMA ? dc_smem_tma(16) : DC_SMEM);
+        if (rc == PLM_OK) rc = set_smem(attn_decode_kernel<true, true, TMA, false>, TMA ? dc_smem_tma(16) : DC_SMEM);
         if (rc != PLM_OK) return rc;
         configured = true;
     }
@@ -918,14 +923,14 @@ extern "C" int plm_attn_decode_rope(const void* qkv, void* kc, void* vc, void* o
     if (n_splits > MERGE_MAX_SPLITS) return PLM_ERR_SHAPE;
     if (n_splits > 1 && !workspace) {
         if (n_splits > DC_MAX_CLUSTER) return PLM_ERR_SHAPE;
-        return plm_status_of(launch_pdl_cluster(attn_decode_kernel<true, true, TMA>, grid, dim3(NT), dim3(n_splits, 1, 1), smem,
+        return plm_status_of(launch_pdl_cluster(attn_decode_kernel<true, true, TMA, false>, grid, dim3(NT), dim3(n_splits, 1, 1), smem,
                                                 stream, (const bf16*)qkv, (const bf16*)kc, (const bf16*)vc, (bf16*)out,
                                                 (float*)nullptr, (float*)nullptr, tok_pos, tok_seq, block_table,
                                                 max_pages, H, G, scale * LOG2E, window, row_groups, rot, q_rows, maps, status, (const float*)nullptr, 0, (const float*)nullptr));
     }
     float* ws_o = workspace;
     float* ws_ml = workspace ? workspace + (size_t)n_tokens * H * n_splits * HD : nullptr;
-    int rc = plm_status_of(launch_pdl(attn_decode_kernel<false, true, TMA>, grid, dim3(NT), smem, stream, (const bf16*)qkv,
+    int rc = plm_status_of(launch_pdl(attn_decode_kernel<false, true, TMA, false>, grid, dim3(NT), smem, stream, (const bf16*)qkv,
                                       (const bf16*)kc, (const bf16*)vc, (bf16*)out, ws_o, ws_ml, tok_pos, tok_seq,
                                       block_table, max_pages, H, G, scale * LOG2E, window, row_groups, rot, q_rows, maps, status, (const float*)nullptr, 0, (const float*)nullptr));
     if (rc != PLM_OK || n_splits == 1) return rc;

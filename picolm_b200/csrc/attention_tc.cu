@@ -20,10 +20,10 @@
 // barriers of their own.  Keys of a KV head are shared by its
 // query heads through L2 (consecutive CTAs work on the heads of one group).
 //
-// A sliding window may keep the sequence's first positions in sight: the walk then starts with their pages.  With
-// slopes (BIAS: a score loses its head's slope times the key's distance) the walk goes backwards, from the tile's own
-// page to the oldest: the scores' level falls along it, so that the reference maximum is found on the first pages and
-// O is hardly ever rescaled.
+// EXTRA instances: a sliding window may keep the sequence's first positions in sight (their pages, where they lie before
+// the window's, belong to the walk), and with slopes a score loses its head's slope times the key's distance.  The walk
+// then goes backwards, from the tile's own page to the oldest: the scores' level falls along it, so that the reference
+// maximum is found on the first pages and O is hardly ever rescaled.
 //
 // Waits on mbarriers are bounded as in gemm_tc.cu: a wait that runs out records where in
 // `status`, the CTA stops issuing work, lets what is in flight land, frees its TMEM and returns.
@@ -165,7 +165,7 @@ __device__ long long plm_attn_trace[5][TRACE_PAGES][8];
 #endif
 
 // grid = (query tiles of the longest sequence, heads, sequences)
-template <bool BIAS>
+template <bool EXTRA>
 __global__ void __launch_bounds__(NUM_THREADS, 2)
 attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out,
@@ -202,10 +202,11 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     const int pos_last = pos0 + rows - 1;
     const int first_key = plm_first_key(pos0, window);
     const int page_first = first_key / BKV, page_last = pos_last / BKV;
-    const int n_kept = plm_kept_pages(first_key, keep);                  // pages of kept first positions before the window's
+    const int n_kept = EXTRA ? plm_kept_pages(first_key, keep) : 0;      // pages of kept first positions before the window's
     const int n_pages = n_kept + page_last - page_first + 1;
     auto page_at = [&](int i) {                                          // the i-th page of the walk
-        const int w = BIAS ? n_pages - 1 - i : i;
+        if (!EXTRA) return page_first + i;
+        const int w = n_pages - 1 - i;
         return w < n_kept ? w : page_first + w - n_kept;
     };
     const int* pages = block_table + (size_t)b * max_pages;
@@ -339,7 +340,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         const int r = quarter * 32 + lane;                               // this thread's query row
         const int pos = r < rows ? pos0 + r : -1;                        // -1: no such row, everything masked
         const int lo = plm_first_key(pos, window);
-        const float slope2 = BIAS ? slopes[h] * LOG2E : 0.f;             // what a key loses per position of distance, log2 units
+        const float slope2 = EXTRA && slopes ? slopes[h] * LOG2E : 0.f;  // what a key loses per position of distance, log2 units
         const uint32_t lane_bits = (uint32_t)(quarter * 32) << 16;
         // O stays in tensor memory and the MMAs accumulate into it across pages.  Probabilities are
         // taken relative to a reference maximum m_ref that is raised (and O rescaled) only when a
@@ -352,14 +353,14 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             tc_fence_after();
             ATTN_TRACE(softmax_warp, i, 0);
             const int key0 = page_at(i) * BKV;
-            const bool need_mask = key0 + BKV - 1 > pos0 || (key0 < plm_first_key(pos_last, window) && key0 + BKV > keep);
+            const bool need_mask = key0 + BKV - 1 > pos0 || (key0 < plm_first_key(pos_last, window) && (!EXTRA || key0 + BKV > keep));
             float mx = -INFINITY;
             uint32_t s0[32], s1[32];
             tc_ld32(tmem + lane_bits + TM_S + (i % NSB) * 64, s0);
             tc_ld32(tmem + lane_bits + TM_S + (i % NSB) * 64 + 32, s1);
             tc_wait_ld();
             ATTN_TRACE(softmax_warp, i, 1);
-            if (BIAS) {                                                  // scores in log2 units, the distance's share taken off
+            if (EXTRA) {                                                 // scores in log2 units, the distance's share taken off
                 const uint64_t sc2 = pack2(__float_as_uint(scale_log2), __float_as_uint(scale_log2));
                 const uint64_t sl2 = pack2(__float_as_uint(slope2), __float_as_uint(slope2));
                 const float off = slope2 * (float)(key0 - pos), off_hi = slope2 * (float)(key0 + 32 - pos);
@@ -381,8 +382,8 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
 #pragma unroll
                 for (int j = 0; j < 32; ++j) {
                     const int ka = key0 + j, kc2 = key0 + 32 + j;
-                    if (ka > pos || (ka < lo && ka >= keep)) s0[j] = 0xff800000u;        // -inf
-                    if (kc2 > pos || (kc2 < lo && kc2 >= keep)) s1[j] = 0xff800000u;
+                    if (ka > pos || (ka < lo && (!EXTRA || ka >= keep))) s0[j] = 0xff800000u;        // -inf
+                    if (kc2 > pos || (kc2 < lo && (!EXTRA || kc2 >= keep))) s1[j] = 0xff800000u;
                 }
             } else if (pos < 0) {
 #pragma unroll
@@ -398,7 +399,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             }
             mx = fmaxf(fmaxf(mx, mx1), fmaxf(mx2, mx3));
             // the scale is positive, so the maximum of the scaled scores is the scaled maximum
-            const float m_cand = fmaxf(m_ref, BIAS ? mx : mx * scale_log2);
+            const float m_cand = fmaxf(m_ref, EXTRA ? mx : mx * scale_log2);
             const bool raise = m_cand > m_ref + RESCALE_LOG2 || (m_ref == -INFINITY && m_cand > -INFINITY);
             // P has two buffers: page i writes the one that page i - 2 used, whose P V must be done.  (Written over
             // the scores it is: S(i) was issued after P(i - 2) V(i - 2) by the same thread.)
@@ -430,7 +431,7 @@ attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
 #pragma unroll
             for (int j = 0; j < 16; ++j) {                              // p = 2^(s * scale - m_ref): half an FFMA2 and one EX2 each
                 float xa0, xa1, xc0, xc1;
-                if (BIAS) {
+                if (EXTRA) {
                     unpack2(add2(pack2(s0[2 * j], s0[2 * j + 1]), neg_m2), xa0, xa1);
                     unpack2(add2(pack2(s1[2 * j], s1[2 * j + 1]), neg_m2), xc0, xc1);
                 } else {
@@ -549,7 +550,7 @@ extern "C" int plm_attn_tc_prefill(const void* q, const void* kc, const void* vc
     if ((rc = make_map(&mk, kc, (long)n_pages * G * BKV, HD, HD, BKV)) != PLM_OK) return rc;
     if ((rc = make_map(&mv, vc, (long)n_pages * G * BKV, HD, HD, BKV)) != PLM_OK) return rc;
     dim3 grid((max_new + BQ - 1) / BQ, H, n_seqs);
-    if (slopes)
+    if (keep || slopes)
         return plm_status_of(launch_pdl(attn_tc_prefill_kernel<true>, grid, dim3(NUM_THREADS), SMEM, stream, mq, mk, mv,
                                         (bf16*)out, seq_start, seq_kv_len, block_table, max_pages, H, G, scale * LOG2E, window,
                                         status, sink, keep, slopes));
