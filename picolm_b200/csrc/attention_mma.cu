@@ -244,10 +244,10 @@ constexpr size_t PF_SMEM = (size_t)(1 + 2 * PF_STAGES) * TILE_ELEMS * sizeof(bf1
 // not looked at.
 template <bool EXTRA>
 __global__ void __launch_bounds__(NT)
-attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const bf16* __restrict__ vc,
-                    bf16* __restrict__ out, const int* __restrict__ seq_start, const int* __restrict__ seq_kv_len,
-                    const int* __restrict__ block_table, int max_pages, int H, int G, float scale_log2, int window,
-                    const float* __restrict__ sink, int keep, const float* __restrict__ slopes) {
+attn_prefill_kernel(const bf16* q, const bf16* kc, const bf16* vc,
+                    bf16* __restrict__ out, const int* seq_start, const int* seq_kv_len,
+                    const int* block_table, int max_pages, int H, int G, float scale_log2, int window,
+                    const float* sink, int keep, const float* slopes) {
     extern __shared__ __align__(16) uint8_t smem_raw[];
     bf16* q_s = reinterpret_cast<bf16*>(smem_raw);
     bf16* k_s = q_s + TILE_ELEMS;                     // [PF_STAGES][64][LDS]
@@ -397,8 +397,8 @@ struct Rotary {
 };
 
 // x[j..j+8) and x[HD/2+j..HD/2+j+8) of one head, rotated by the angles of `pos` (fp32, rounded once)
-__device__ __forceinline__ void rotate16(uint4& lo, uint4& hi, const float* __restrict__ cos_t,
-                                         const float* __restrict__ sin_t, int pos, int j) {
+__device__ __forceinline__ void rotate16(uint4& lo, uint4& hi, const float* cos_t,
+                                         const float* sin_t, int pos, int j) {
     const float* cp = cos_t + (size_t)pos * (HD / 2) + j;
     const float* sp = sin_t + (size_t)pos * (HD / 2) + j;
     __nv_bfloat162* l2 = reinterpret_cast<__nv_bfloat162*>(&lo);
@@ -419,12 +419,12 @@ struct PageMaps {               // the TMA form: the caches as [pages * G * 64 r
 
 template <bool CLUSTER, bool ROPE, bool TMA, bool EXTRA>
 __global__ void __launch_bounds__(NT)
-attn_decode_kernel(const bf16* __restrict__ q, const bf16* __restrict__ kc, const bf16* __restrict__ vc,
+attn_decode_kernel(const bf16* q, const bf16* kc, const bf16* vc,
                    bf16* __restrict__ out, float* __restrict__ ws_o, float* __restrict__ ws_ml,
-                   const int* __restrict__ tok_pos, const int* __restrict__ tok_seq, const int* __restrict__ block_table,
+                   const int* tok_pos, const int* tok_seq, const int* block_table,
                    int max_pages, int H, int G, float scale_log2, int window, int row_groups, const Rotary rot,
                    int q_rows, const __grid_constant__ PageMaps maps, int* __restrict__ status,
-                   const float* __restrict__ sink, int keep, const float* __restrict__ slopes) {
+                   const float* sink, int keep, const float* slopes) {
     extern __shared__ __align__(16) uint8_t smem_raw[];
     const size_t q_bytes = (size_t)q_rows * LDS * sizeof(bf16);          // q_rows: 16, or 9 (8 heads and a row of zeros)
     bf16* q_s = reinterpret_cast<bf16*>(smem_raw);
@@ -721,8 +721,8 @@ constexpr int MERGE_MAX_SPLITS = 8192;                   // the weights of all r
 constexpr int MERGE_LANES = HD <= 64 ? 64 : HD <= 128 ? 128 : 256;
 constexpr int MERGE_GROUPS = MERGE_THREADS / MERGE_LANES;
 __global__ void __launch_bounds__(MERGE_THREADS)
-attn_merge_kernel(const float* __restrict__ ws_o, const float* __restrict__ ws_ml, bf16* __restrict__ out, int n_splits,
-                  const float* __restrict__ sink, int H) {
+attn_merge_kernel(const float* ws_o, const float* ws_ml, bf16* __restrict__ out, int n_splits,
+                  const float* sink, int H) {
     extern __shared__ float merge_w[];                  // [n_splits] weights, then [MERGE_GROUPS][MERGE_LANES] sums
     __shared__ float red[MERGE_THREADS / 32];
     __shared__ float s_max, s_l;

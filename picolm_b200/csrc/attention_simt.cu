@@ -25,10 +25,10 @@ constexpr int MAX_HD = 1024;           // the largest head size; acc registers p
 // latent cache, whose keys are the latents themselves).
 template <typename Ta, typename Tc, int MAX_HD>
 __global__ void __launch_bounds__(WARPS * 32)
-attention_rows_kernel(const Ta* __restrict__ q, const Tc* __restrict__ kc, const Tc* __restrict__ vc,
-                      Ta* __restrict__ out, const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
-                      const int* __restrict__ block_table, int max_pages, int H, int G, int hd, float scale,
-                      int window, const float* __restrict__ sink, int keep, const float* __restrict__ slopes) {
+attention_rows_kernel(const Ta* q, const Tc* kc, const Tc* vc,
+                      Ta* __restrict__ out, const int* tok_pos, const int* tok_seq,
+                      const int* block_table, int max_pages, int H, int G, int hd, float scale,
+                      int window, const float* sink, int keep, const float* slopes) {
     extern __shared__ float q_sm[];                 // [WARPS][hd]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x;

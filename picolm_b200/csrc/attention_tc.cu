@@ -169,9 +169,9 @@ template <bool EXTRA>
 __global__ void __launch_bounds__(NUM_THREADS, 2)
 attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out,
-                       const int* __restrict__ seq_start, const int* __restrict__ seq_kv_len,
-                       const int* __restrict__ block_table, int max_pages, int H, int G, float scale_log2, int window,
-                       int* __restrict__ status, const float* __restrict__ sink, int keep, const float* __restrict__ slopes) {
+                       const int* seq_start, const int* seq_kv_len,
+                       const int* block_table, int max_pages, int H, int G, float scale_log2, int window,
+                       int* __restrict__ status, const float* sink, int keep, const float* slopes) {
     extern __shared__ uint8_t smem_raw[];
     const uint32_t raw = smem_u32(smem_raw);
     const uint32_t base = (raw + 1023u) & ~1023u;

@@ -95,6 +95,10 @@ __device__ __forceinline__ float rope_second(float a, float b, float c, float s)
 // set itself up and read what no earlier kernel of the step writes (weights); it must not write
 // global memory.  pdl_launch_dependents() lets the next kernel begin its own set-up.  Without the
 // launch attribute both are no-ops.
+// What a kernel only reads is declared `const T*`, not `const T* __restrict__`: a load through the latter counts as one of
+// an unchanging value, and the compiler may move it above pdl_wait(), where it reads what the kernel before has not
+// written yet.  (That happened: a grouped product took its tiles' group numbers before the sort had written them, at
+// sizes where neighbouring kernels overlap.)  What a kernel writes may be restrict; __ldg is for weights alone.
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 __device__ __forceinline__ void pdl_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 

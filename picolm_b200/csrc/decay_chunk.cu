@@ -326,9 +326,9 @@ __global__ void __launch_bounds__(NT, 1) decay_chunk_kernel(const Args a) {
 constexpr int STEP_NT = 256, STEP_COLS = 64;
 template <typename T>
 __global__ void __launch_bounds__(STEP_NT)
-decay_step_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, long ldq, long ldk, long ldv,
-                  const float* __restrict__ decay, float* __restrict__ state, long state_stride, float* __restrict__ y, long ldy,
-                  const int* __restrict__ seq_slot, int N, int P, int silu) {
+decay_step_kernel(const T* q, const T* k, const T* v, long ldq, long ldk, long ldv,
+                  const float* decay, float* __restrict__ state, long state_stride, float* __restrict__ y, long ldy,
+                  const int* seq_slot, int N, int P, int silu) {
     extern __shared__ float step_sm[];                 // q [N], k [N], shares [16][64]
     float* qs = step_sm;
     float* ks = qs + N;

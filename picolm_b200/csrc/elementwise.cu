@@ -13,7 +13,7 @@
 
 // ------------------------------------------------------------------ embedding
 template <typename Tw>
-__global__ void embed_kernel(const int* __restrict__ tok, const Tw* __restrict__ table, float* __restrict__ out,
+__global__ void embed_kernel(const int* tok, const Tw* table, float* __restrict__ out,
                              int d, int vocab, float scale) {
     pdl_launch_dependents();
     pdl_wait();
@@ -47,8 +47,8 @@ extern "C" int plm_embed(const int* tok, const void* table, int table_dtype, flo
 // else is in the batch.
 
 template <typename Tw, typename To, int NT>
-__global__ void rmsnorm_kernel(float* __restrict__ x, const float* __restrict__ delta, const Tw* __restrict__ w,
-                               To* __restrict__ out, const int* __restrict__ rows, int d, float eps, int write_back) {
+__global__ void rmsnorm_kernel(float* __restrict__ x, const float* delta, const Tw* w,
+                               To* __restrict__ out, const int* rows, int d, float eps, int write_back) {
     __shared__ float red[33];
     pdl_launch_dependents();
     pdl_wait();
@@ -94,8 +94,8 @@ __device__ __forceinline__ void store4(bf16* p, float4 v) {
 
 template <typename Tw, typename To, int NT>
 __global__ void __launch_bounds__(NT)
-rmsnorm_vec_kernel(float* __restrict__ x, const float* __restrict__ delta, const Tw* __restrict__ w,
-                   To* __restrict__ out, const int* __restrict__ rows, int d, float eps, int write_back) {
+rmsnorm_vec_kernel(float* __restrict__ x, const float* delta, const Tw* w,
+                   To* __restrict__ out, const int* rows, int d, float eps, int write_back) {
     __shared__ float red[33];
     pdl_launch_dependents();
     pdl_wait();
@@ -174,8 +174,8 @@ extern "C" int plm_rmsnorm(float* x, const float* delta, const void* w, int w_dt
 // Rows whose width is a multiple of 4 and at most 16 * NT stay in registers throughout.
 template <typename Tw, typename To, int NT>
 __global__ void __launch_bounds__(NT)
-post_pre_norm_kernel(float* __restrict__ x, const float* __restrict__ delta, const Tw* __restrict__ w_post,
-                     const Tw* __restrict__ w_pre, To* __restrict__ out, int d, float eps_post, float eps_pre) {
+post_pre_norm_kernel(float* __restrict__ x, const float* delta, const Tw* w_post,
+                     const Tw* w_pre, To* __restrict__ out, int d, float eps_post, float eps_pre) {
     __shared__ float red[33];
     pdl_launch_dependents();
     pdl_wait();
@@ -250,7 +250,7 @@ extern "C" int plm_post_pre_norm(float* x, const float* delta, const void* w_pos
 // out[t, :] = bf16(x[t, :] * r[t]) with r[t] = 1 / sqrt(sum_p parts[p, t] / size + eps): what is left of
 // an RMSNorm whose weight a product's epilogue has already applied (x) and whose sums of squares it has
 // left as partial sums (parts [n_parts, ld_parts]).  One block per row, sums in a fixed order.
-__global__ void scale_rows_kernel(const bf16* __restrict__ x, const float* __restrict__ parts, int n_parts, int ld_parts,
+__global__ void scale_rows_kernel(const bf16* x, const float* parts, int n_parts, int ld_parts,
                                   float inv_size, float eps, bf16* __restrict__ out, int d) {
     pdl_launch_dependents();
     pdl_wait();
@@ -290,7 +290,7 @@ __device__ __forceinline__ float gate_clamped(float g, float u, float limit, flo
 }
 
 template <typename T, int ACT>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int F, size_t total, float limit, float slope) {
+__global__ void swiglu_kernel(const T* gu, T* __restrict__ out, int F, size_t total, float limit, float slope) {
     pdl_launch_dependents();
     pdl_wait();
     size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -337,10 +337,10 @@ extern "C" int plm_swiglu(const void* gu, void* out, int dtype, int act, int n_r
 // and beyond rot_dim pass through.  store = 0 skips the cache (a layer that reads
 // another layer's cache).
 template <typename Ta, typename Tc>
-__global__ void rope_store_kernel(const Ta* __restrict__ qkv, Ta* __restrict__ q_out, Tc* __restrict__ kc,
-                                  Tc* __restrict__ vc, const float* __restrict__ cos_t,
-                                  const float* __restrict__ sin_t, const int* __restrict__ tok_pos,
-                                  const int* __restrict__ tok_seq, const int* __restrict__ block_table,
+__global__ void rope_store_kernel(const Ta* qkv, Ta* __restrict__ q_out, Tc* __restrict__ kc,
+                                  Tc* __restrict__ vc, const float* cos_t,
+                                  const float* sin_t, const int* tok_pos,
+                                  const int* tok_seq, const int* block_table,
                                   int max_pages, int H, int G, int hd, int rot_dim, int pairing, int store) {
     pdl_launch_dependents();
     pdl_wait();
@@ -402,10 +402,10 @@ __global__ void rope_store_kernel(const Ta* __restrict__ qkv, Ta* __restrict__ q
 // The common case eight pairs at a time: bf16, the whole head rotated (rot_dim == hd), half-split
 // pairing, head size a multiple of 16.  A thread takes x[j..j+8) and x[half+j..half+j+8) of one head
 // as two 16-byte loads and writes two 16-byte stores.
-__global__ void rope_store_vec_kernel(const bf16* __restrict__ qkv, bf16* __restrict__ q_out, bf16* __restrict__ kc,
-                                      bf16* __restrict__ vc, const float* __restrict__ cos_t,
-                                      const float* __restrict__ sin_t, const int* __restrict__ tok_pos,
-                                      const int* __restrict__ tok_seq, const int* __restrict__ block_table,
+__global__ void rope_store_vec_kernel(const bf16* qkv, bf16* __restrict__ q_out, bf16* __restrict__ kc,
+                                      bf16* __restrict__ vc, const float* cos_t,
+                                      const float* sin_t, const int* tok_pos,
+                                      const int* tok_seq, const int* block_table,
                                       int max_pages, int H, int G, int hd, int store) {
     pdl_launch_dependents();
     pdl_wait();
@@ -488,7 +488,7 @@ extern "C" int plm_rope_store(const void* qkv, void* q_out, void* kc, void* vc, 
 
 // dst[i, :] = src[rows[i], :] for rows of `row_bytes` bytes (a multiple of 4; 16 bytes at a time where the rows
 // and both pointers allow it).  Rows of a prompt step that are wanted further on, out of all of its rows.
-__global__ void gather_rows_kernel(const uint8_t* __restrict__ src, uint8_t* __restrict__ dst, const int* __restrict__ rows,
+__global__ void gather_rows_kernel(const uint8_t* src, uint8_t* __restrict__ dst, const int* rows,
                                    long row_bytes, long src_ld, int wide) {
     pdl_launch_dependents();
     pdl_wait();
@@ -521,8 +521,8 @@ extern "C" int plm_gather_rows(const void* src, void* dst, const int* rows, int 
 // stays in shared memory between the passes (mean, deviations, output), so x is read once.
 template <typename Tw, typename To, int NT>
 __global__ void __launch_bounds__(NT)
-layernorm_kernel(float* __restrict__ x, const float* __restrict__ delta, const float* __restrict__ bias,
-                 const Tw* __restrict__ w, To* __restrict__ out, const int* __restrict__ rows, int d, float eps,
+layernorm_kernel(float* __restrict__ x, const float* delta, const float* bias,
+                 const Tw* w, To* __restrict__ out, const int* rows, int d, float eps,
                  int write_back) {
     extern __shared__ float row_sm[];               // [d]
     __shared__ float red[33];
@@ -557,8 +557,8 @@ layernorm_kernel(float* __restrict__ x, const float* __restrict__ delta, const f
 // at most 16 * NT (and 16-byte aligned pointers).
 template <typename Tw, typename To, int NT>
 __global__ void __launch_bounds__(NT)
-layernorm_vec_kernel(float* __restrict__ x, const float* __restrict__ delta, const float* __restrict__ bias,
-                     const Tw* __restrict__ w, To* __restrict__ out, const int* __restrict__ rows, int d, float eps,
+layernorm_vec_kernel(float* __restrict__ x, const float* delta, const float* bias,
+                     const Tw* w, To* __restrict__ out, const int* rows, int d, float eps,
                      int write_back) {
     __shared__ float red[33];
     pdl_launch_dependents();
@@ -647,7 +647,7 @@ extern "C" int plm_layernorm(float* x, const float* delta, const float* bias, co
 }
 
 // x[t, :] += bias[:] in place on fp32 rows: a projection's bias, where nothing that follows can take it along.
-__global__ void add_bias_kernel(float* __restrict__ x, const float* __restrict__ bias, int d, size_t total) {
+__global__ void add_bias_kernel(float* __restrict__ x, const float* bias, int d, size_t total) {
     pdl_launch_dependents();
     pdl_wait();
     size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -685,15 +685,15 @@ __device__ __forceinline__ void store_pair(bf16* p, float a, float b) { *reinter
 
 template <typename Ta, typename Tw, typename Tc, int NT, bool CONV>
 __global__ void __launch_bounds__(NT)
-qk_norm_rope_store_kernel(const Ta* __restrict__ qkv, const float* __restrict__ bias, const Tw* __restrict__ wq,
-                          const Tw* __restrict__ wk, float eps, Tc* __restrict__ q_out, Tc* __restrict__ kc,
-                          Tc* __restrict__ vc, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
-                          const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
-                          const int* __restrict__ block_table, int max_pages, int H, int G, int D, int Dv, int hd_c,
+qk_norm_rope_store_kernel(const Ta* qkv, const float* bias, const Tw* wq,
+                          const Tw* wk, float eps, Tc* __restrict__ q_out, Tc* __restrict__ kc,
+                          Tc* __restrict__ vc, const float* cos_t, const float* sin_t,
+                          const int* tok_pos, const int* tok_seq,
+                          const int* block_table, int max_pages, int H, int G, int D, int Dv, int hd_c,
                           int rot_dim, int pairing, int own_kv, int per_head, int v_from_k, long ld,
-                          const float* __restrict__ q_scale, const float* __restrict__ conv_w, int taps,
-                          float* __restrict__ conv_state, long state_stride, const int* __restrict__ seq_start,
-                          const int* __restrict__ seq_slot, int conv_keeps_state) {
+                          const float* q_scale, const float* conv_w, int taps,
+                          float* __restrict__ conv_state, long state_stride, const int* seq_start,
+                          const int* seq_slot, int conv_keeps_state) {
     extern __shared__ float qk_sm[];                 // [nq + nk] (with a convolution: [nq + nk + nv])
     __shared__ float red[33];
     pdl_launch_dependents();
@@ -875,8 +875,8 @@ qk_norm_rope_store_kernel(const Ta* __restrict__ qkv, const float* __restrict__ 
 // oldest first (old tail rows move up where the step brought fewer).  One thread per (sequence, column); it reads what
 // it needs of the old tail before it writes (ascending s: slot s takes old slot s + n > s).
 template <typename Ta>
-__global__ void conv_tail_kernel(const Ta* __restrict__ qkv, long ld, float* __restrict__ state, long state_stride,
-                                 const int* __restrict__ seq_start, const int* __restrict__ seq_slot, int n_seqs, int C, int taps) {
+__global__ void conv_tail_kernel(const Ta* qkv, long ld, float* __restrict__ state, long state_stride,
+                                 const int* seq_start, const int* seq_slot, int n_seqs, int C, int taps) {
     pdl_launch_dependents();
     pdl_wait();
     const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -946,10 +946,10 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
 
 template <typename To, int NT>
 __global__ void __launch_bounds__(NT)
-dyt_norm_kernel(float* __restrict__ x, const float* __restrict__ delta, const float* __restrict__ dbias,
-                const float* __restrict__ post_w, float post_eps, const float* __restrict__ extra,
-                const float* __restrict__ alpha, const float* __restrict__ w, const float* __restrict__ b,
-                To* __restrict__ out, const int* __restrict__ rows, int d, int write_back) {
+dyt_norm_kernel(float* __restrict__ x, const float* delta, const float* dbias,
+                const float* post_w, float post_eps, const float* extra,
+                const float* alpha, const float* w, const float* b,
+                To* __restrict__ out, const int* rows, int d, int write_back) {
     __shared__ float red[33];
     pdl_launch_dependents();
     pdl_wait();
@@ -995,8 +995,8 @@ extern "C" int plm_dyt_norm(float* x, const float* delta, const float* dbias, co
 }
 
 // x[r, :] += a[r, :] + b[r, :] + vec[:], in that order; every addend may be null.
-__global__ void add_rows_kernel(float* __restrict__ x, const float* __restrict__ a, const float* __restrict__ b,
-                                const float* __restrict__ vec, long n, int d) {
+__global__ void add_rows_kernel(float* __restrict__ x, const float* a, const float* b,
+                                const float* vec, long n, int d) {
     pdl_launch_dependents();
     pdl_wait();
     const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -1015,8 +1015,8 @@ extern "C" int plm_add_rows(float* x, const float* a, const float* b, const floa
 }
 
 // out[r, :] = sa * (a[r, :] + bias_a[:]) + sb * b[r, :]: two float32 results added with two constants.
-__global__ void scaled_sum_kernel(const float* __restrict__ a, float sa, const float* __restrict__ bias_a,
-                                  const float* __restrict__ b, float sb, float* __restrict__ out, long n, int d) {
+__global__ void scaled_sum_kernel(const float* a, float sa, const float* bias_a,
+                                  const float* b, float sb, float* __restrict__ out, long n, int d) {
     pdl_launch_dependents();
     pdl_wait();
     const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -1036,8 +1036,8 @@ extern "C" int plm_scaled_sum(const float* a, float sa, const float* bias_a, con
 
 // out[r, j] = gelu_tanh(gate[r, j]) * table[tok[row r], col0 + j]: a gate times a row of a per-token table.
 template <typename T, typename Tw>
-__global__ void token_gate_kernel(const T* __restrict__ gate, const Tw* __restrict__ table, long ld_table, int col0,
-                                  const int* __restrict__ tok, const int* __restrict__ rows, T* __restrict__ out, int n_rows,
+__global__ void token_gate_kernel(const T* gate, const Tw* table, long ld_table, int col0,
+                                  const int* tok, const int* rows, T* __restrict__ out, int n_rows,
                                   int dim, int vocab) {
     pdl_launch_dependents();
     pdl_wait();
@@ -1069,8 +1069,8 @@ extern "C" int plm_token_gate(const void* gate, int dtype, const void* table, in
 // (pairing 0: (x[i], x[i + rot_dim/2]); pairing 1: (x[2i], x[2i+1])), in fp32, in place; the others stay.  For rows that
 // reach attention by another way than a QKV product (queries taken into a latent's space, for instance).
 template <typename T>
-__global__ void rope_rows_kernel(T* __restrict__ x, long ld, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
-                                 const int* __restrict__ tok_pos, int n_rows, int n_heads, int hd, int rot_dim, int pairing) {
+__global__ void rope_rows_kernel(T* __restrict__ x, long ld, const float* cos_t, const float* sin_t,
+                                 const int* tok_pos, int n_rows, int n_heads, int hd, int rot_dim, int pairing) {
     pdl_launch_dependents();
     pdl_wait();
     const int half = rot_dim / 2;
@@ -1133,7 +1133,7 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float* red) {    
 }
 
 template <int NT>
-__device__ __forceinline__ float row_sum_squares(const float* __restrict__ row, int d) {
+__device__ __forceinline__ float row_sum_squares(const float* row, int d) {
     float ss = 0.f;
     if ((d & 3) == 0) {
         for (int i = threadIdx.x * 4; i < d; i += NT * 4) {
@@ -1148,9 +1148,9 @@ __device__ __forceinline__ float row_sum_squares(const float* __restrict__ row, 
 
 template <typename To, int NT>
 __global__ void __launch_bounds__(NT)
-norm_pair_shift_kernel(const float* __restrict__ x, const float* __restrict__ w_a, const float* __restrict__ w_b,
-                       const float* __restrict__ mix, float* __restrict__ state, long state_stride,
-                       const int* __restrict__ tok_seq, const int* __restrict__ seq_start, const int* __restrict__ seq_slot,
+norm_pair_shift_kernel(const float* x, const float* w_a, const float* w_b,
+                       const float* mix, float* __restrict__ state, long state_stride,
+                       const int* tok_seq, const int* seq_start, const int* seq_slot,
                        To* __restrict__ out_a, To* __restrict__ out_b, int d, float eps) {
     __shared__ float red[33];
     pdl_launch_dependents();
@@ -1191,9 +1191,9 @@ norm_pair_shift_kernel(const float* __restrict__ x, const float* __restrict__ w_
 // registers between the sums of squares and the results (VPT float4 a thread and row), so that x is read once.
 template <typename To, int NT, int VPT>
 __global__ void __launch_bounds__(NT)
-norm_pair_shift_vec_kernel(const float* __restrict__ x, const float* __restrict__ w_a, const float* __restrict__ w_b,
-                           const float* __restrict__ mix, float* __restrict__ state, long state_stride,
-                           const int* __restrict__ tok_seq, const int* __restrict__ seq_start, const int* __restrict__ seq_slot,
+norm_pair_shift_vec_kernel(const float* x, const float* w_a, const float* w_b,
+                           const float* mix, float* __restrict__ state, long state_stride,
+                           const int* tok_seq, const int* seq_start, const int* seq_slot,
                            To* __restrict__ out_a, To* __restrict__ out_b, int d, float eps) {
     __shared__ float red[66];
     pdl_launch_dependents();
@@ -1298,9 +1298,9 @@ extern "C" int plm_norm_pair_shift(const float* x, const float* w_a, const float
 // a sequence that has none yet.  The block of a sequence's first token of the step reads the state and then writes the
 // sequence's last token of the step into it, so no block reads a state that is already new.
 template <typename Tw>
-__global__ void embed_pair_kernel(const int* __restrict__ tok, const Tw* __restrict__ table, const Tw* __restrict__ pairs,
-                                  int* __restrict__ state, long state_stride, const int* __restrict__ tok_seq,
-                                  const int* __restrict__ seq_start, const int* __restrict__ seq_slot, float* __restrict__ out,
+__global__ void embed_pair_kernel(const int* tok, const Tw* table, const Tw* pairs,
+                                  int* __restrict__ state, long state_stride, const int* tok_seq,
+                                  const int* seq_start, const int* seq_slot, float* __restrict__ out,
                                   int d, int vocab, long buckets, long mul_prev, long mul_cur, float scale) {
     pdl_launch_dependents();
     pdl_wait();
@@ -1360,9 +1360,9 @@ extern "C" int plm_embed_pair(const int* tok, const void* table, const void* pai
 __device__ __forceinline__ float dot4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
 template <typename To, int NT, int VPT>
 __global__ void __launch_bounds__(NT)
-joined_post_pre_norm_kernel(float* __restrict__ x, const float* __restrict__ a, const float* __restrict__ b,
-                            const float* __restrict__ w_a, const float* __restrict__ w_b, float factor,
-                            const float* __restrict__ w_post, const float* __restrict__ w_pre, To* __restrict__ out, int d,
+joined_post_pre_norm_kernel(float* __restrict__ x, const float* a, const float* b,
+                            const float* w_a, const float* w_b, float factor,
+                            const float* w_post, const float* w_pre, To* __restrict__ out, int d,
                             float eps_a, float eps_b, float eps_post, float eps_pre) {
     __shared__ float red[66];
     pdl_launch_dependents();
@@ -1454,13 +1454,16 @@ extern "C" int plm_joined_post_pre_norm(float* x, const float* a, const float* b
 // ------------------------------------------- a QKV product's rows to attention, nothing done to them on the way
 // qkv [T, H*D | G*D | G*Dv] (row stride ld) -> q_out [T, H, hd_c], keys and values into the pages of the cache (head size
 // hd_c); what lies beyond a head's own width is written as zero.  Sizes are counted in pieces of 16 bytes.
-__global__ void heads_store_kernel(const uint4* __restrict__ qkv, long ld, uint4* __restrict__ q_out, uint4* __restrict__ kc,
-                                   uint4* __restrict__ vc, const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
-                                   const int* __restrict__ block_table, int max_pages, int H, int G, int D, int Dv, int hc) {
+__global__ void heads_store_kernel(const uint4* qkv, long ld, uint4* __restrict__ q_out, uint4* __restrict__ kc,
+                                   uint4* __restrict__ vc, const int* tok_pos, const int* tok_seq,
+                                   const int* block_table, int max_pages, int H, int G, int D, int Dv, int hc) {
     pdl_launch_dependents();
-    pdl_wait();
     const int t = blockIdx.x;
     const uint4* row = qkv + (size_t)t * ld;
+    // what describes the step was written before it began: read while the product in front finishes
+    const int pos = PLM_POSITION(tok_pos[t]);
+    const int page = kc ? PLM_PAGE_NO(block_table[(size_t)PLM_SEQ_NO(tok_seq[t]) * max_pages + pos / PLM_PAGE]) : 0;
+    pdl_wait();
     const uint4 zero = make_uint4(0, 0, 0, 0);
     uint4* qo = q_out + (size_t)t * H * hc;
     for (int i = threadIdx.x; i < H * hc; i += blockDim.x) {
@@ -1468,8 +1471,6 @@ __global__ void heads_store_kernel(const uint4* __restrict__ qkv, long ld, uint4
         qo[i] = c < D ? row[h * D + c] : zero;
     }
     if (!kc) return;
-    const int pos = PLM_POSITION(tok_pos[t]);
-    const int page = PLM_PAGE_NO(block_table[(size_t)PLM_SEQ_NO(tok_seq[t]) * max_pages + pos / PLM_PAGE]);
     for (int i = threadIdx.x; i < G * hc; i += blockDim.x) {
         const int g = i / hc, c = i - g * hc;
         const size_t at = (((size_t)page * G + g) * PLM_PAGE + pos % PLM_PAGE) * hc + c;
@@ -1495,7 +1496,7 @@ extern "C" int plm_heads_store(const void* qkv, int dtype, long ld, void* q_out,
 // ------------------------------------------------------------------------- an activation without a gate
 // y = 0.5 x (1 + erf(x / sqrt 2)), the exact GELU
 template <typename T>
-__global__ void gelu_erf_kernel(const T* __restrict__ x, T* __restrict__ out, size_t total) {
+__global__ void gelu_erf_kernel(const T* x, T* __restrict__ out, size_t total) {
     pdl_launch_dependents();
     pdl_wait();
     for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {

@@ -21,7 +21,7 @@ constexpr int BM = 64, BN = 64, BK = 16, NT = 256;
 
 template <typename Ta, typename Tw, typename To>
 __global__ void __launch_bounds__(NT)
-gemm_simt_kernel(const Ta* __restrict__ A, const Tw* __restrict__ W, To* __restrict__ C, int M, int N, int K,
+gemm_simt_kernel(const Ta* A, const Tw* W, To* __restrict__ C, int M, int N, int K,
                  long lda, long ldw, long ldc) {
     __shared__ float As[BK][BM + 4];
     __shared__ float Ws[BK][BN + 4];

@@ -184,7 +184,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_p, const __grid_constant_
 // out[i] = sum over splits of partial[s][i], in ascending s.  VEC: total is a
 // multiple of 4, so every split's slice starts on a 16-byte boundary.
 template <typename OutT, bool VEC>
-__global__ void splitk_reduce_kernel(const float* __restrict__ partial, OutT* __restrict__ out, int splits, size_t total) {
+__global__ void splitk_reduce_kernel(const float* partial, OutT* __restrict__ out, int splits, size_t total) {
     pdl_launch_dependents();
     pdl_wait();
     if (VEC) {

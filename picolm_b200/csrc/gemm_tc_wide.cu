@@ -279,7 +279,7 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
                     OutT* __restrict__ out, int T, int F, int K, long ldo, int m_tiles, int n_tiles,
                     int* __restrict__ status, int k_splits, int kb_per_split, size_t split_stride,
                     float* parts, int* flags, const __grid_constant__ CUtensorMap map_out, int out_by_copies,
-                    const int* __restrict__ tile_group, int group_rows, float gate_limit, float gate_slope) {
+                    const int* tile_group, int group_rows, float gate_limit, float gate_slope) {
     // tile_group (grouped form, null otherwise): the weights are `groups` matrices of group_rows rows one below the
     // other, and the token rows of tile m (128 rows) meet matrix tile_group[m] (below 0: a tile without rows, which is passed by):
     // the weight rows that the producer asks for start group_rows * tile_group[m] further down.  An earlier kernel
@@ -312,6 +312,7 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
     // tile of tokens follow each other; the token tiles of one group are neighbours, so one wave of CTAs holds all tiles that
     // read a group's weights, each weight comes from memory once, and the token rows stay in the L2 (measured at 6,144 rows
     // over 32 groups of 4,096 x 2,048: the other order read 800 MB where the weights are 537 MB).
+    auto group_at = [&](int m) { return ((const volatile int*)tile_group)[m]; };     // (read behind pdl_wait(), never before)
     auto tile_m = [&](int tile) { return tile_group ? tile / n_tiles : tile % m_tiles; };
     auto tile_n = [&](int tile) { return tile_group ? tile % n_tiles : tile / m_tiles; };
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -374,7 +375,7 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
                 int f0 = tile_n(w.tile) * BN + (int)rank * W_ROWS;
                 if (tile_group) {
                     if (!waited) { pdl_wait(); waited = true; }
-                    const int grp = tile_group[tile_m(w.tile)];
+                    const int grp = group_at(tile_m(w.tile));
                     if (grp < 0) continue;                               // a tile without rows: every role passes it by
                     f0 += grp * group_rows;
                 }
@@ -446,7 +447,7 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
 #endif
             if (tile_group) pdl_wait();                                  // an earlier kernel of the step writes it
             for (; ok && walk.next(w); ++j) {
-                if (tile_group && tile_group[tile_m(w.tile)] < 0) { --j; continue; }
+                if (tile_group && group_at(tile_m(w.tile)) < 0) { --j; continue; }
                 const int acc = j & 1;
                 // the epilogue must have read this accumulator's previous piece out
                 if (!mbar_wait(acc_empty0 + 8 * acc, ((j >> 1) & 1) ^ 1, status, 2)) { s_abort = 1; ok = false; break; }
@@ -496,7 +497,7 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
         Walk walk = walk0;
         Piece w;
         for (; ok && walk.next(w); ++j) {
-            if (tile_group && tile_group[tile_m(w.tile)] < 0) { --j; continue; }
+            if (tile_group && group_at(tile_m(w.tile)) < 0) { --j; continue; }
             const int acc = j & 1;
             const int m0 = tile_m(w.tile) * TILE_M + (int)rank * BM, f0 = tile_n(w.tile) * BN;
             const int row0 = m0 + quarter * 32;                          // this warp's 32 token rows
@@ -898,7 +899,7 @@ int launch(const CUtensorMap& mx, const CUtensorMap& mw, OutT* out, int T, int F
 
 // out[i] = sum over the K splits of scratch[s * stride + i], in order; four at a time.
 template <typename OutT>
-__global__ void reduce_splits_kernel(const float* __restrict__ scratch, OutT* __restrict__ out, int k_splits, size_t n4,
+__global__ void reduce_splits_kernel(const float* scratch, OutT* __restrict__ out, int k_splits, size_t n4,
                                      size_t stride) {
     pdl_launch_dependents();
     pdl_wait();

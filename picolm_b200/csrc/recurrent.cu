@@ -53,10 +53,10 @@ __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
 #define CONV_ACT_SILU 0
 #define CONV_ACT_NONE 1
 template <typename T>
-__global__ void causal_conv_kernel(const T* __restrict__ u, long ldu, const float* __restrict__ w, const float* __restrict__ bias,
-                                   const float* __restrict__ state, long state_stride, const int* __restrict__ tok_seq,
-                                   const int* __restrict__ seq_start, const int* __restrict__ seq_slot, T* __restrict__ out,
-                                   int n_tokens, int C, int taps, const float* __restrict__ in_bias, int act) {
+__global__ void causal_conv_kernel(const T* u, long ldu, const float* w, const float* bias,
+                                   const float* state, long state_stride, const int* tok_seq,
+                                   const int* seq_start, const int* seq_slot, T* __restrict__ out,
+                                   int n_tokens, int C, int taps, const float* in_bias, int act) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x, c = blockIdx.y * blockDim.x + threadIdx.x;
@@ -76,10 +76,10 @@ __global__ void causal_conv_kernel(const T* __restrict__ u, long ldu, const floa
 
 // The same for bf16 rows whose channels come in eights on 16-byte boundaries: a thread takes 8 channels of a token
 // with one 16-byte load per tap.
-__global__ void causal_conv_vec8_kernel(const bf16* __restrict__ u, long ldu, const float* __restrict__ w,
-                                        const float* __restrict__ bias, const float* __restrict__ state, long state_stride,
-                                        const int* __restrict__ tok_seq, const int* __restrict__ seq_start,
-                                        const int* __restrict__ seq_slot, bf16* __restrict__ out, int n_tokens, int C, int taps) {
+__global__ void causal_conv_vec8_kernel(const bf16* u, long ldu, const float* w,
+                                        const float* bias, const float* state, long state_stride,
+                                        const int* tok_seq, const int* seq_start,
+                                        const int* seq_slot, bf16* __restrict__ out, int n_tokens, int C, int taps) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x, c = (blockIdx.y * blockDim.x + threadIdx.x) << 3;
@@ -120,9 +120,9 @@ __global__ void causal_conv_vec8_kernel(const bf16* __restrict__ u, long ldu, co
 // The state after the step: the last taps - 1 inputs of old state followed by the step's tokens.  One thread per
 // (sequence, channel); it reads what it needs of the old state before it writes.
 template <typename T>
-__global__ void causal_conv_state_kernel(const T* __restrict__ u, long ldu, float* __restrict__ state, long state_stride,
-                                         const int* __restrict__ seq_start, const int* __restrict__ seq_slot, int n_seqs,
-                                         int C, int taps, const float* __restrict__ in_bias) {
+__global__ void causal_conv_state_kernel(const T* u, long ldu, float* __restrict__ state, long state_stride,
+                                         const int* seq_start, const int* seq_slot, int n_seqs,
+                                         int C, int taps, const float* in_bias) {
     pdl_launch_dependents();
     pdl_wait();
     const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -139,10 +139,10 @@ __global__ void causal_conv_state_kernel(const T* __restrict__ u, long ldu, floa
 
 // A decode step (one token per sequence): output and new state by the same thread.
 template <typename T>
-__global__ void causal_conv_decode_kernel(const T* __restrict__ u, long ldu, const float* __restrict__ w,
-                                          const float* __restrict__ bias, float* __restrict__ state, long state_stride,
-                                          const int* __restrict__ seq_slot, T* __restrict__ out, int n_seqs, int C, int taps,
-                                          const float* __restrict__ in_bias, int act) {
+__global__ void causal_conv_decode_kernel(const T* u, long ldu, const float* w,
+                                          const float* bias, float* __restrict__ state, long state_stride,
+                                          const int* seq_slot, T* __restrict__ out, int n_seqs, int C, int taps,
+                                          const float* in_bias, int act) {
     pdl_launch_dependents();
     pdl_wait();
     const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -580,7 +580,7 @@ extern "C" int plm_linear_scan_plan(int n_seqs, int H, int N, int P, int max_new
 
 // out[t, c] = sigmoid(raw[t, c] + bias[c]) ^ power in fp32: the decays of DECAY_SIGMOID, worked out once.
 template <typename T>
-__global__ void sigmoid_decay_kernel(const T* __restrict__ raw, long ld, const float* __restrict__ bias, float power,
+__global__ void sigmoid_decay_kernel(const T* raw, long ld, const float* bias, float power,
                                      float* __restrict__ out, int n_rows, int C) {
     pdl_launch_dependents();
     pdl_wait();
@@ -644,8 +644,8 @@ extern "C" int plm_linear_scan(const void* q, const void* k, const void* v, cons
 //   val = val * act(gate)                     (gate_mode 2: the gate comes after the norm)
 // act: 0 SiLU, 1 sigmoid.  Statistics and products in fp32.
 template <typename TI, typename TG, typename TO>
-__global__ void gated_norm_kernel(const TI* __restrict__ x, long ldx, const TG* __restrict__ gate, long ldg,
-                                  const float* __restrict__ w, int w_per_group, TO* __restrict__ out, long ldo, int n_rows,
+__global__ void gated_norm_kernel(const TI* x, long ldx, const TG* gate, long ldg,
+                                  const float* w, int w_per_group, TO* __restrict__ out, long ldo, int n_rows,
                                   int C, int group, float eps, int gate_mode, int act, int do_norm) {
     pdl_launch_dependents();
     pdl_wait();
@@ -705,7 +705,7 @@ __device__ __forceinline__ void gn_store4(bf16* p, float4 v) {
 }
 template <typename TI, typename TG, typename TO, int NT, int VPT>
 __global__ void __launch_bounds__(NT)
-gated_norm_wide_kernel(const TI* __restrict__ x, long ldx, const TG* __restrict__ gate, long ldg, const float* __restrict__ w,
+gated_norm_wide_kernel(const TI* x, long ldx, const TG* gate, long ldg, const float* w,
                        int w_per_group, TO* __restrict__ out, long ldo, int groups, int group, float eps, int gate_mode, int act) {
     __shared__ float red[33];
     pdl_launch_dependents();
@@ -800,8 +800,8 @@ extern "C" int plm_gated_norm(const void* x, int x_dtype, long ldx, const void* 
 #define HL_TO 64
 #define HL_TI 32
 template <typename T, typename TG>
-__global__ void __launch_bounds__(256) head_linear_kernel(const T* __restrict__ x, long ldx, const T* __restrict__ W,
-                                                          const TG* __restrict__ gate, long ldg, T* __restrict__ out, long ldo,
+__global__ void __launch_bounds__(256) head_linear_kernel(const T* x, long ldx, const T* W,
+                                                          const TG* gate, long ldg, T* __restrict__ out, long ldo,
                                                           int n_tokens, int H, int O, int I, int gate_per_head) {
     __shared__ float xs[HL_TI][HL_TT + 4];                 // transposed: a thread reads its 4 tokens as one float4
     __shared__ float ws[HL_TI][HL_TO + 4];
@@ -856,8 +856,8 @@ __global__ void __launch_bounds__(256) head_linear_kernel(const T* __restrict__ 
 // token's x[t, h, :]; a lane's elements are I / 32 apart so that the warp's loads are contiguous.
 #define HLS_MAX_T 16
 template <typename T, typename TG>
-__global__ void __launch_bounds__(256) head_linear_small_kernel(const T* __restrict__ x, long ldx, const T* __restrict__ W,
-                                                                const TG* __restrict__ gate, long ldg, T* __restrict__ out,
+__global__ void __launch_bounds__(256) head_linear_small_kernel(const T* x, long ldx, const T* W,
+                                                                const TG* gate, long ldg, T* __restrict__ out,
                                                                 long ldo, int n_tokens, int H, int O, int I, int gate_per_head) {
     pdl_launch_dependents();
     const long row = ((long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;          // h * O + o
@@ -919,8 +919,8 @@ extern "C" int plm_head_linear(const void* x, int dtype, long ldx, const void* W
 // ------------------------------------------------------------------------------------------------ rows into pages
 // pages [n_pages][PLM_PAGE][R] (one kv head): row t goes to position tok_pos[t] of sequence tok_seq[t].
 template <typename T>
-__global__ void store_rows_paged_kernel(const T* __restrict__ rows, long ld, T* __restrict__ pages, const int* __restrict__ tok_pos,
-                                        const int* __restrict__ tok_seq, const int* __restrict__ block_table, int pages_per_seq,
+__global__ void store_rows_paged_kernel(const T* rows, long ld, T* __restrict__ pages, const int* tok_pos,
+                                        const int* tok_seq, const int* block_table, int pages_per_seq,
                                         int n_tokens, int R) {
     pdl_launch_dependents();
     pdl_wait();
@@ -957,11 +957,11 @@ extern "C" int plm_store_rows_paged(const void* rows, int dtype, long ld, void* 
 // ldq, divided by their root mean square and multiplied by wq [n_q], to q_out [T, n_q] (contiguous).
 template <typename Ti, typename To>
 __global__ void __launch_bounds__(128)
-latent_store_kernel(const Ti* __restrict__ rows, long ld, const float* __restrict__ w, float eps, const float* __restrict__ cos_t,
-                    const float* __restrict__ sin_t, To* __restrict__ pages, const int* __restrict__ tok_pos,
-                    const int* __restrict__ tok_seq, const int* __restrict__ block_table, int pages_per_seq, int n_tokens,
-                    int n_rot, int n_norm, int R, int pairing, int store, const Ti* __restrict__ q_rows, long ldq,
-                    const float* __restrict__ wq, To* __restrict__ q_out, int n_q) {
+latent_store_kernel(const Ti* rows, long ld, const float* w, float eps, const float* cos_t,
+                    const float* sin_t, To* __restrict__ pages, const int* tok_pos,
+                    const int* tok_seq, const int* block_table, int pages_per_seq, int n_tokens,
+                    int n_rot, int n_norm, int R, int pairing, int store, const Ti* q_rows, long ldq,
+                    const float* wq, To* __restrict__ q_out, int n_q) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -1037,8 +1037,8 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
 
 template <typename T, typename Tw>
 __global__ void __launch_bounds__(256)
-rglru_gates_kernel(const T* __restrict__ u, long ldu, const Tw* __restrict__ wr, const Tw* __restrict__ wi,
-                   const float* __restrict__ br, const float* __restrict__ bi, const float* __restrict__ rate,
+rglru_gates_kernel(const T* u, long ldu, const Tw* wr, const Tw* wi,
+                   const float* br, const float* bi, const float* rate,
                    float* __restrict__ a_out, float* __restrict__ x_out, int n_tokens, int W, int n) {
     __shared__ float us[32][33], wrs[32][33], wis[32][33];
     pdl_launch_dependents();
@@ -1121,9 +1121,9 @@ extern "C" int plm_rglru_gates(const void* u, int dtype, long ldu, const void* w
 // stretch's product of decays and its own sum, one warp chains them from the cache's state, a second walk writes.
 template <typename T>
 __global__ void __launch_bounds__(1024)
-diag_scan_kernel(const float* __restrict__ a, const float* __restrict__ x, const T* __restrict__ yraw, long ldy,
-                 const float* __restrict__ ybias, float* __restrict__ state, long state_stride, T* __restrict__ out,
-                 const int* __restrict__ seq_start, const int* __restrict__ seq_slot, int W) {
+diag_scan_kernel(const float* a, const float* x, const T* yraw, long ldy,
+                 const float* ybias, float* __restrict__ state, long state_stride, T* __restrict__ out,
+                 const int* seq_start, const int* seq_slot, int W) {
     __shared__ double As[32][33], Bs[32][33];
     pdl_launch_dependents();
     pdl_wait();
@@ -1165,9 +1165,9 @@ diag_scan_kernel(const float* __restrict__ a, const float* __restrict__ x, const
 
 // A decode step: one token per sequence, one thread per (sequence, channel).
 template <typename T>
-__global__ void diag_scan_decode_kernel(const float* __restrict__ a, const float* __restrict__ x, const T* __restrict__ yraw,
-                                        long ldy, const float* __restrict__ ybias, float* __restrict__ state, long state_stride,
-                                        T* __restrict__ out, const int* __restrict__ seq_slot, int n_seqs, int W) {
+__global__ void diag_scan_decode_kernel(const float* a, const float* x, const T* yraw,
+                                        long ldy, const float* ybias, float* __restrict__ state, long state_stride,
+                                        T* __restrict__ out, const int* seq_slot, int n_seqs, int W) {
     pdl_launch_dependents();
     pdl_wait();
     const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -1209,8 +1209,8 @@ extern "C" int plm_diag_scan(const float* a, const float* x, const void* yraw, i
 // long depends on; the recurrence takes S + expm1(dec) S.  One block per token; a warp per key head, then per head.
 template <typename T>
 __global__ void __launch_bounds__(128)
-delta_prep_kernel(const T* __restrict__ q, long ldq, const T* __restrict__ k, long ldk, const T* __restrict__ z, long ldz,
-                  const T* __restrict__ braw, long ldb, const float* __restrict__ a_log, const float* __restrict__ dt_bias,
+delta_prep_kernel(const T* q, long ldq, const T* k, long ldk, const T* z, long ldz,
+                  const T* braw, long ldb, const float* a_log, const float* dt_bias,
                   float l2_eps, float q_scale, float* __restrict__ qn, float* __restrict__ kn, float* __restrict__ qk,
                   float* __restrict__ dec, float* __restrict__ beta, int G, int H, int N) {
     pdl_launch_dependents();
@@ -1270,10 +1270,10 @@ extern "C" int plm_delta_prep(const void* q, long ldq, const void* k, long ldk, 
 #define DELTA_COLS 32
 template <typename T, int NR>
 __global__ void __launch_bounds__(128)
-delta_scan_kernel(const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ qk,
-                  const float* __restrict__ dec, const float* __restrict__ beta, const T* __restrict__ v, long ldv,
-                  float* __restrict__ state, long state_stride, float* __restrict__ y, const int* __restrict__ seq_start,
-                  const int* __restrict__ seq_slot, int H, int N, int P, int heads_per_group, int TC) {
+delta_scan_kernel(const float* qn, const float* kn, const float* qk,
+                  const float* dec, const float* beta, const T* v, long ldv,
+                  float* __restrict__ state, long state_stride, float* __restrict__ y, const int* seq_start,
+                  const int* seq_slot, int H, int N, int P, int heads_per_group, int TC) {
     constexpr int NP = NR * 4;
     extern __shared__ __align__(16) float smem[];
     float* qs = smem;                         // [TC][NP]
@@ -1408,8 +1408,8 @@ static inline int delta_chunk_np(int N) { return N <= 32 ? 32 : N <= 64 ? 64 : N
 // grid (chunk of the sequence, sequence, head).  ws per (slot, head): Kp [C][NP] | Qp [C][NP] | Ke [C][NP] | A^T [C][C] | M^T [C][C]
 // | e^{L_C} [NP], NP = delta_chunk_np(N), the padding zero.  A sequence's chunk c lives in slot seq_start / C + sequence + c.
 __global__ void __launch_bounds__(256)
-delta_chunk_prep_kernel(const float* __restrict__ qn, const float* __restrict__ kn, const float* __restrict__ lgd,
-                        float* __restrict__ ws, const int* __restrict__ seq_start, int H, int N, int NP, int heads_per_group) {
+delta_chunk_prep_kernel(const float* qn, const float* kn, const float* lgd,
+                        float* __restrict__ ws, const int* seq_start, int H, int N, int NP, int heads_per_group) {
     constexpr int C = DELTA_CHUNK;
     extern __shared__ __align__(16) float smem[];
     float* cum = smem;                  // [C][N]
@@ -1487,9 +1487,9 @@ __device__ __forceinline__ void cp_async16(float* dst, const float* src) {
 
 template <int NR, int STAGES>
 __global__ void __launch_bounds__(128)
-delta_chunk_scan_kernel(const float* __restrict__ ws, const float* __restrict__ beta, const void* __restrict__ v, int v_f32, long ldv,
-                        float* __restrict__ state, long state_stride, float* __restrict__ y, const int* __restrict__ seq_start,
-                        const int* __restrict__ seq_slot, int H, int N, int P) {
+delta_chunk_scan_kernel(const float* ws, const float* beta, const void* v, int v_f32, long ldv,
+                        float* __restrict__ state, long state_stride, float* __restrict__ y, const int* seq_start,
+                        const int* seq_slot, int H, int N, int P) {
     constexpr int C = DELTA_CHUNK, NP = NR * 8, SEG = NR + 4, RS = 8 * SEG;      // SEG: an eighth's floats in a row, padded
     constexpr int STAGE = 3 * C * RS + 2 * C * C + RS;                            // Kp | Qp | Ke [C][RS], A | M [C][C], e^{L_C} [RS]
     extern __shared__ __align__(16) float smem[];

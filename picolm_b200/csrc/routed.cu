@@ -30,7 +30,7 @@ constexpr int ROUTE_WARPS = 4;
 // One warp per token.  logits [T, ld] fp32: columns [0, E) the router's, column `gate_col` (if gate != null) the
 // logit of a shared expert's gate.  ids [T, top] int32, weights [T, top] fp32, gate [T] fp32 = sigmoid(that logit).
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
-route_topk_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ correction, int E, int top,
+route_topk_kernel(const float* logits, int ld, const float* correction, int E, int top,
                   int n_groups, int keep, float scale, int* __restrict__ ids, float* __restrict__ weights,
                   float* __restrict__ gate, int gate_col, int T, int score_mode, int group_by_max, int normalize) {
     extern __shared__ float route_sm[];             // per warp: s[E], c[E], group score[n_groups], group kept[n_groups]
@@ -157,7 +157,7 @@ __device__ __forceinline__ float4 rl_load4(const bf16* p) {
 }
 template <typename Th, typename Tw>
 __global__ void __launch_bounds__(RL_WARPS * 32)
-router_logits_kernel(const Th* __restrict__ h, const Tw* __restrict__ w, float* __restrict__ out, int T, int E, int K) {
+router_logits_kernel(const Th* h, const Tw* w, float* __restrict__ out, int T, int E, int K) {
     extern __shared__ float rl_sm[];                // [RL_TOKENS][K]
     pdl_launch_dependents();
     pdl_wait();
@@ -211,7 +211,7 @@ router_logits_kernel(const Th* __restrict__ h, const Tw* __restrict__ w, float* 
 // tensors) are left out: where = -1.
 constexpr int ALIGN_NT = 1024;
 __global__ void __launch_bounds__(ALIGN_NT)
-moe_align_kernel(const int* __restrict__ ids, int n_entries, int E, int BM, int* __restrict__ tile_expert,
+moe_align_kernel(const int* ids, int n_entries, int E, int BM, int* __restrict__ tile_expert,
                  int* __restrict__ sorted, int* __restrict__ where, int max_tiles, int n_skip) {
     extern __shared__ int align_sm[];               // cnt[E], off[E + 1], fill[E]
     pdl_launch_dependents();
@@ -276,8 +276,8 @@ __device__ __forceinline__ int up_row_of(int n, int N, int interleaved) { return
 
 template <typename Ta, typename Tw, typename To, int BM, int MODE>
 __global__ void __launch_bounds__(256)
-moe_gemm_kernel(const Ta* __restrict__ a, long lda, int top, const Tw* __restrict__ w, To* __restrict__ out, long ldo,
-                const int* __restrict__ tile_expert, const int* __restrict__ sorted, int N, int K, int interleaved) {
+moe_gemm_kernel(const Ta* a, long lda, int top, const Tw* w, To* __restrict__ out, long ldo,
+                const int* tile_expert, const int* sorted, int N, int K, int interleaved) {
     constexpr int TM = BM / 16;
     __shared__ float As[MG_BK][BM + 1];
     __shared__ float Bs[MODE == 0 ? 2 : 1][MG_BK][MG_BN + 1];
@@ -381,8 +381,8 @@ __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], uint32_t a0, uint3
 
 template <int MODE>
 __global__ void __launch_bounds__(MM_WARPS * 32)
-moe_gemm_mma_kernel(const bf16* __restrict__ a, long lda, int top, const bf16* __restrict__ w, void* __restrict__ out_, long ldo,
-                    const int* __restrict__ tile_expert, const int* __restrict__ sorted, int N, int K, int interleaved) {
+moe_gemm_mma_kernel(const bf16* a, long lda, int top, const bf16* w, void* __restrict__ out_, long ldo,
+                    const int* tile_expert, const int* sorted, int N, int K, int interleaved) {
     constexpr int BM = 16, NACC = MODE == 0 ? 2 : 1;
     extern __shared__ __align__(16) uint8_t mm_raw[];
     bf16* As = reinterpret_cast<bf16*>(mm_raw);                        // [16][MM_LD]
@@ -475,7 +475,7 @@ moe_gemm_mma_kernel(const bf16* __restrict__ a, long lda, int top, const bf16* _
 // ------------------------------------------------------------------ rows in sorted order
 // dst[p, :] = src[sorted[p] / top, :] (zero where sorted[p] < 0): the tokens' rows laid out as the sorted tiles want
 // them, for a product that takes whole tiles of its left operand.
-__global__ void moe_gather_kernel(const uint8_t* __restrict__ src, uint8_t* __restrict__ dst, const int* __restrict__ sorted,
+__global__ void moe_gather_kernel(const uint8_t* src, uint8_t* __restrict__ dst, const int* sorted,
                                   int top, long row_bytes) {
     pdl_launch_dependents();
     pdl_wait();
@@ -499,10 +499,10 @@ __global__ void moe_gather_kernel(const uint8_t* __restrict__ src, uint8_t* __re
 // [T, d] or null) is what a sublayer beside the feed-forward made of the same x, and with `accumulate` the result goes
 // straight into the residual stream.
 template <typename Th>
-__global__ void moe_combine_kernel(const float* __restrict__ y, long ldy, const int* __restrict__ where,
-                                   const float* __restrict__ weights, int top, const float* __restrict__ shared,
-                                   const float* __restrict__ gate, float* __restrict__ out, int d,
-                                   const Th* __restrict__ ident, const float* __restrict__ add, float out_scale, int accumulate) {
+__global__ void moe_combine_kernel(const float* y, long ldy, const int* where,
+                                   const float* weights, int top, const float* shared,
+                                   const float* gate, float* __restrict__ out, int d,
+                                   const Th* ident, const float* add, float out_scale, int accumulate) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;

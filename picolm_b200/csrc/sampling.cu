@@ -107,7 +107,7 @@ __device__ void slice_crossing(const unsigned long long* bins, unsigned long lon
 
 // The row's maximum and the first index that has it, over the whole cluster (strict > scan from
 // index 0, picolm/sampler.c:50-56).  Every CTA returns the same pair.
-__device__ void cluster_argmax(const float* __restrict__ row, int lo, int hi, Shared* sh, float* redf, int* redi,
+__device__ void cluster_argmax(const float* row, int lo, int hi, Shared* sh, float* redf, int* redi,
                                float& best_v, int& best_i) {
     float bv = -INFINITY;
     int bi = INT_MAX;
@@ -147,7 +147,7 @@ __device__ void cluster_argmax(const float* __restrict__ row, int lo, int hi, Sh
 }
 
 __global__ void __launch_bounds__(NT)
-argmax_kernel(const float* __restrict__ logits, long ld, int V, int chunk, int* __restrict__ out) {
+argmax_kernel(const float* logits, long ld, int V, int chunk, int* __restrict__ out) {
     __shared__ Shared sh;
     __shared__ float redf[33];
     __shared__ int redi[33];
@@ -165,7 +165,7 @@ argmax_kernel(const float* __restrict__ logits, long ld, int V, int chunk, int* 
 }
 
 __global__ void __launch_bounds__(NT, 2)
-sample_kernel(const float* __restrict__ logits, long ld, int V, int chunk, float temperature, int top_k, float top_p,
+sample_kernel(const float* logits, long ld, int V, int chunk, float temperature, int top_k, float top_p,
               float min_p, unsigned long long* __restrict__ rng, int* __restrict__ out) {
     extern __shared__ float prob[];                      // this CTA's eighth of the row's probabilities
     __shared__ Shared sh;

@@ -639,6 +639,29 @@ def test_bfloat16_at_sizes_the_tensor_cores_refuse(tmp_path, name):
         assert rel < 0.03, f"two cuts of the same request differ by {rel:.3f} of the spread"
 
 
+def test_overlapping_launches_see_what_the_ones_before_wrote(tmp_path):
+    """Steps whose kernels are queued far ahead of the GPU (a slow recurrence in front of routed layers whose prompts
+    take the grouped products): neighbouring launches then overlap, and a value read before the kernel in front has
+    written it shows as wrong logits.  The same step again and again, on memory that earlier steps used for other things."""
+    layers = [_layer(_left(heads=2, kv_heads=2, dim=48, vdim=8, size=17, keep=20, scale=0.07), _right(heads=1, dim=160, vdim=4, decay=[0.0]),
+                     mlp=_moe(experts=3, top=1, ff=128, shared=None)),
+              _layer(_left(heads=16, kv_heads=2, dim=64, vdim=16, size=100, keep=0, scale=0.2), _right(heads=3, dim=160, vdim=4),
+                     mlp=_moe(experts=3, top=2, ff=64, shared=64)),
+              _layer(_left(heads=4, kv_heads=1, dim=96, vdim=16, size=65, keep=100, scale=0.1), _right(heads=4, dim=48, vdim=4, decay=[0.999, 0.6, 0.9, 0.5]),
+                     mlp=_dense(100))]
+    d, tensors, config = _make(tmp_path, "overlap", _config(layers, width=160, mult=0.5), seed=315, std=0.08, bias=2.0)
+    reqs = [random_tokens(n, VOCAB, 70 + i) for i, n in enumerate([1, 160, 100])]
+    want = torch.cat([_plain(tensors, config, t) for t in reqs])
+    eng = _engine(d, dtype="bfloat16")
+    for turn in range(8):
+        slots = [eng.new_sequence() for _ in reqs]
+        got = eng.step(list(zip(slots, reqs)), [list(range(len(t))) for t in reqs]).float().cpu()
+        rel = (got - want).double().pow(2).mean(dim=1).sqrt() / want.double().std()
+        assert rel.median() < 0.02, f"turn {turn}: half of the rows are {rel.median().item():.3f} of the spread away"
+        for s in slots:
+            eng.end_sequence(s)
+
+
 # ---------------------------------------------------------------------------------------------- generation
 GEN = [_layer(_left(size=6, keep=2), mlp="dense"), _layer(_left(heads=2, kv_heads=1, dim=8, vdim=16, size=70, keep=0), mlp="moe"), _layer(mlp=None)]
 
