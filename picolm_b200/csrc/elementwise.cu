@@ -964,15 +964,17 @@ dyt_norm_kernel(float* __restrict__ x, const float* delta, const float* dbias,
         for (int i = threadIdx.x; i < d; i += NT) ss = fmaf(dr[i], dr[i], ss);
         post = 1.0f / sqrtf(block_sum<NT>(ss, red) / (float)d + post_eps);
     }
-    const float a = alpha ? alpha[0] : 0.f;
+    const float a = alpha ? __ldg(alpha) : 0.f;
     To* o = out ? out + (size_t)r * d : nullptr;
     for (int i = threadIdx.x; i < d; i += NT) {
+        // (weights alone go through __ldg: no kernel of the step writes them)
+        const float wi = alpha ? __ldg(w + i) : 0.f, bi = alpha ? __ldg(b + i) : 0.f;
         float v = xr[i];
-        if (dr) v += post_w ? dr[i] * post * post_w[i] : dr[i];
-        if (dbias) v += dbias[i];
+        if (dr) v += post_w ? dr[i] * post * __ldg(post_w + i) : dr[i];
+        if (dbias) v += __ldg(dbias + i);
         if (er) v += er[i];
         if (write_back) xr[i] = v;
-        if (o) o[i] = from_f32<To>(alpha ? fmaf(tanhf(a * v), w[i], b[i]) : v);
+        if (o) o[i] = from_f32<To>(alpha ? fmaf(tanhf(a * v), wi, bi) : v);
     }
 }
 

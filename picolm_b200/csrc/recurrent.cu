@@ -1221,6 +1221,7 @@ delta_prep_kernel(const T* q, long ldq, const T* k, long ldk, const T* z, long l
             const T* qr = q + (long)t * ldq + (long)job * N;
             const T* kr = k + (long)t * ldk + (long)job * N;
             float sq = 0.f, sk = 0.f, sqk = 0.f;
+#pragma unroll 4
             for (int i = lane; i < N; i += 32) {
                 const float a = to_f32<T>(qr[i]), b = to_f32<T>(kr[i]);
                 sq = fmaf(a, a, sq), sk = fmaf(b, b, sk), sqk = fmaf(a, b, sqk);
@@ -1236,10 +1237,10 @@ delta_prep_kernel(const T* q, long ldq, const T* k, long ldk, const T* z, long l
             if (lane == 0) qk[(long)t * G + job] = sqk * rq * rk;
         } else {
             const int h = job - G;
-            const float rate = expf(a_log[h]);
+            const float rate = expf(__ldg(a_log + h));
             const T* zr = z + (long)t * ldz + (long)h * N;
             float* d = dec + ((long)t * H + h) * N;
-            for (int i = lane; i < N; i += 32) d[i] = -rate * softplus_f(to_f32<T>(zr[i]) + dt_bias[(long)h * N + i]);
+            for (int i = lane; i < N; i += 32) d[i] = -rate * softplus_f(to_f32<T>(zr[i]) + __ldg(dt_bias + (long)h * N + i));
             if (lane == 0) beta[(long)t * H + h] = sigmoid_f(to_f32<T>(braw[(long)t * ldb + h]));
         }
     }
