@@ -63,6 +63,9 @@ MORE_BUILDS: List = [("gemm_tc_wide@stream", ["-DPLM_WIDE_STREAM"]),
                      # the bf16 store epilogue with the exact GELU (products with an activation and no gate)
                      ("gemm_tc_skinny@gelu_erf", ["-DPLM_STORE_GELU_ERF"]), ("gemm_tc_wide@gelu_erf", ["-DPLM_STORE_GELU_ERF"]),
                      ("gemm_tc_wide@stream_gelu_erf", ["-DPLM_WIDE_STREAM", "-DPLM_STORE_GELU_ERF"]),
+                     # the same with the square of ReLU
+                     ("gemm_tc_skinny@relu2", ["-DPLM_STORE_RELU2"]), ("gemm_tc_wide@relu2", ["-DPLM_STORE_RELU2"]),
+                     ("gemm_tc_wide@stream_relu2", ["-DPLM_WIDE_STREAM", "-DPLM_STORE_RELU2"]),
                      # the gated epilogue with clamped branches and a sloped sigmoid (its constants come with the launch)
                      ("gemm_tc_skinny@clamped", ["-DPLM_GATE_CLAMPED"]), ("gemm_tc_wide@clamped", ["-DPLM_GATE_CLAMPED"]),
                      ("gemm_tc_wide@stream_clamped", ["-DPLM_WIDE_STREAM", "-DPLM_GATE_CLAMPED"])]

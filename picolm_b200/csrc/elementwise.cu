@@ -40,6 +40,52 @@ extern "C" int plm_embed(const int* tok, const void* table, int table_dtype, flo
     return PLM_ERR_DTYPE;
 }
 
+// out[t, :] = RMSNorm of float(table[tok[t], :]) with weight w: a stream that begins normed.  One block per token, the row in
+// shared memory between the two passes.
+template <typename Tw, int NT>
+__global__ void __launch_bounds__(NT)
+embed_norm_kernel(const int* tok, const Tw* table, const Tw* w, float* __restrict__ out, int d, int vocab, float eps) {
+    extern __shared__ float embed_row[];            // [d]
+    __shared__ float red[33];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x;
+    int id = tok[t];
+    if (id < 0 || id >= vocab) id = 0;   // ids are checked on the host; never read outside the table
+    const Tw* row = table + (size_t)id * d;
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < d; i += NT) {
+        const float v = to_f32<Tw>(row[i]);
+        embed_row[i] = v;                           // (read back by the same thread)
+        ss += v * v;
+    }
+    ss = block_sum<NT>(ss, red);
+    const float scale = 1.0f / sqrtf(ss / (float)d + eps);
+    float* o = out + (size_t)t * d;
+    for (int i = threadIdx.x; i < d; i += NT) o[i] = embed_row[i] * scale * to_f32<Tw>(w[i]);
+}
+
+// table and w of one type, d at most 51,200 (a row in shared memory)
+extern "C" int plm_embed_norm(const int* tok, const void* table, const void* w, int dtype, float* out, int n_tokens, int d,
+                              int vocab, float eps, cudaStream_t stream) {
+    if (n_tokens <= 0) return PLM_OK;
+    const size_t smem = (size_t)d * sizeof(float);
+    if (d <= 0 || vocab <= 0 || smem > 200 * 1024) return PLM_ERR_SHAPE;
+    if (dtype == PLM_F32) {
+        if (smem > 48 * 1024)
+            cudaFuncSetAttribute(embed_norm_kernel<float, 256>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        return plm_status_of(launch_pdl(embed_norm_kernel<float, 256>, dim3(n_tokens), dim3(256), smem, stream, tok, (const float*)table,
+                                        (const float*)w, out, d, vocab, eps));
+    }
+    if (dtype == PLM_BF16) {
+        if (smem > 48 * 1024)
+            cudaFuncSetAttribute(embed_norm_kernel<bf16, 256>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        return plm_status_of(launch_pdl(embed_norm_kernel<bf16, 256>, dim3(n_tokens), dim3(256), smem, stream, tok, (const bf16*)table,
+                                        (const bf16*)w, out, d, vocab, eps));
+    }
+    return PLM_ERR_DTYPE;
+}
+
 // -------------------------------------------------------------------- RMSNorm
 // One block per output row.  Row r reads source row rows[r] (or r).  With a
 // delta the sum x + delta is normalised; it is written back to x unless rows are
@@ -1496,24 +1542,54 @@ extern "C" int plm_heads_store(const void* qkv, int dtype, long ld, void* q_out,
 }
 
 // ------------------------------------------------------------------------- an activation without a gate
-// y = 0.5 x (1 + erf(x / sqrt 2)), the exact GELU
-template <typename T>
-__global__ void gelu_erf_kernel(const T* x, T* __restrict__ out, size_t total) {
+// Activations without a gate, element by element: 0.5 x (1 + erf(x / sqrt 2)), the exact GELU, and relu(x)^2
+template <typename T, int ACT>
+__global__ void plain_act_kernel(const T* x, T* __restrict__ out, size_t total) {
     pdl_launch_dependents();
     pdl_wait();
-    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t stride = (size_t)gridDim.x * blockDim.x;
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += stride) {
         const float v = to_f32<T>(x[i]);
-        out[i] = from_f32<T>(0.5f * v * (1.f + erff(v * 0.70710678118654752f)));
+        const float r = fmaxf(v, 0.f);
+        out[i] = from_f32<T>(ACT == 0 ? 0.5f * v * (1.f + erff(v * 0.70710678118654752f)) : r * r);
     }
 }
 
-extern "C" int plm_gelu_erf(const void* x, void* out, int dtype, long total, cudaStream_t stream) {
+// act 0: exact GELU; 1: squared ReLU
+extern "C" int plm_plain_act(const void* x, void* out, int dtype, int act, long total, cudaStream_t stream) {
     if (total <= 0) return PLM_OK;
-    const long blocks = (total + 255) / 256;
-    const dim3 grid((unsigned)(blocks < 16 * PLM_SM_COUNT ? blocks : 16 * PLM_SM_COUNT));
-    if (dtype == PLM_F32)
-        return plm_status_of(launch_pdl(gelu_erf_kernel<float>, grid, dim3(256), 0, stream, (const float*)x, (float*)out, (size_t)total));
-    if (dtype == PLM_BF16)
-        return plm_status_of(launch_pdl(gelu_erf_kernel<bf16>, grid, dim3(256), 0, stream, (const bf16*)x, (bf16*)out, (size_t)total));
+    if (act != 0 && act != 1) return PLM_ERR_UNSUPPORTED;
+    const unsigned blocks = (unsigned)((total + 255) / 256);
+    const dim3 grid(blocks < 8u * PLM_SM_COUNT ? blocks : 8u * PLM_SM_COUNT);
+#define PA(T_, ACT_) return plm_status_of(launch_pdl(plain_act_kernel<T_, ACT_>, grid, dim3(256), 0, stream, (const T_*)x, (T_*)out, (size_t)total))
+    if (dtype == PLM_F32) { if (act == 0) PA(float, 0); PA(float, 1); }
+    if (dtype == PLM_BF16) { if (act == 0) PA(bf16, 0); PA(bf16, 1); }
+#undef PA
     return PLM_ERR_DTYPE;
+}
+
+// --------------------------------------------------------------------- logits
+// x = cap * tanh(x * scale / cap) in place (fp32): logits between -cap and cap, nearly scale * x near zero.
+__global__ void squash_kernel(float* __restrict__ x, long total, float scale, float cap) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long stride = (long)gridDim.x * blockDim.x * 4;
+    for (long i = ((long)blockIdx.x * blockDim.x + threadIdx.x) * 4; i < total; i += stride) {
+        if (i + 4 <= total && ((uintptr_t)x & 15) == 0) {
+            float4 v = *reinterpret_cast<const float4*>(x + i);
+            v.x = cap * tanhf(v.x * scale / cap), v.y = cap * tanhf(v.y * scale / cap);
+            v.z = cap * tanhf(v.z * scale / cap), v.w = cap * tanhf(v.w * scale / cap);
+            *reinterpret_cast<float4*>(x + i) = v;
+        } else {
+            for (long j = i; j < i + 4 && j < total; ++j) x[j] = cap * tanhf(x[j] * scale / cap);
+        }
+    }
+}
+
+extern "C" int plm_squash(float* x, long total, float scale, float cap, cudaStream_t stream) {
+    if (total <= 0) return PLM_OK;
+    if (!(cap > 0.f)) return PLM_ERR_SHAPE;
+    const long quads = (total + 3) / 4;
+    const unsigned blocks = (unsigned)((quads + 255) / 256 < 8L * PLM_SM_COUNT ? (quads + 255) / 256 : 8L * PLM_SM_COUNT);
+    return plm_status_of(launch_pdl(squash_kernel, dim3(blocks), dim3(256), 0, stream, x, total, scale, cap));
 }

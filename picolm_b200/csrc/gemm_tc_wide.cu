@@ -654,7 +654,7 @@ gemm_tc_wide_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
                         get_part(c + 32);
                     }
                     add_parts(r, c, part);
-#ifdef PLM_STORE_GELU_ERF
+#ifdef PLM_STORE_ACT
                     if (EPI == EPI_STORE && !F32_OUT) {
 #pragma unroll
                         for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(store_act<OutT>(__uint_as_float(r[i])));

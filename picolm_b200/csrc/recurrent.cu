@@ -1204,7 +1204,8 @@ extern "C" int plm_diag_scan(const float* a, const float* x, const void* yraw, i
 // ------------------------------------------------------------------------------------------------ gated delta rule
 // What the delta rule's recurrence takes, worked out per token in fp32 from the convolved projections:
 //   qn = q / sqrt(sum q^2 + l2_eps) * q_scale and kn = k / sqrt(sum k^2 + l2_eps) per key head, qk = qn . kn,
-//   dec[h, n] = -exp(A_log[h]) * softplus(z[h, n] + dt_bias[h, n]),  beta[h] = sigmoid(braw[h]).
+//   dec[h, n] = -exp(A_log[h]) * softplus(z[h, n] + dt_bias[h, n]),  beta[h] = sigmoid(braw[h]),
+// or, with ND = 1 in place of N, one decay a head: dec[h] from z[h] and dt_bias[h].
 // dec is the decay's logarithm: a float next to 1 has lost the digits of its distance from 1, which a state that lasts
 // long depends on; the recurrence takes S + expm1(dec) S.  One block per token; a warp per key head, then per head.
 template <typename T>
@@ -1212,7 +1213,7 @@ __global__ void __launch_bounds__(128)
 delta_prep_kernel(const T* q, long ldq, const T* k, long ldk, const T* z, long ldz,
                   const T* braw, long ldb, const float* a_log, const float* dt_bias,
                   float l2_eps, float q_scale, float* __restrict__ qn, float* __restrict__ kn, float* __restrict__ qk,
-                  float* __restrict__ dec, float* __restrict__ beta, int G, int H, int N) {
+                  float* __restrict__ dec, float* __restrict__ beta, int G, int H, int N, int ND) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -1238,9 +1239,9 @@ delta_prep_kernel(const T* q, long ldq, const T* k, long ldk, const T* z, long l
         } else {
             const int h = job - G;
             const float rate = expf(__ldg(a_log + h));
-            const T* zr = z + (long)t * ldz + (long)h * N;
-            float* d = dec + ((long)t * H + h) * N;
-            for (int i = lane; i < N; i += 32) d[i] = -rate * softplus_f(to_f32<T>(zr[i]) + __ldg(dt_bias + (long)h * N + i));
+            const T* zr = z + (long)t * ldz + (long)h * ND;
+            float* d = dec + ((long)t * H + h) * ND;
+            for (int i = lane; i < ND; i += 32) d[i] = -rate * softplus_f(to_f32<T>(zr[i]) + __ldg(dt_bias + (long)h * ND + i));
             if (lane == 0) beta[(long)t * H + h] = sigmoid_f(to_f32<T>(braw[(long)t * ldb + h]));
         }
     }
@@ -1248,23 +1249,25 @@ delta_prep_kernel(const T* q, long ldq, const T* k, long ldk, const T* z, long l
 
 extern "C" int plm_delta_prep(const void* q, long ldq, const void* k, long ldk, const void* z, long ldz, const void* braw, long ldb,
                               int dtype, const float* a_log, const float* dt_bias, float l2_eps, float q_scale, float* qn, float* kn,
-                              float* qk, float* dec, float* beta, int n_tokens, int G, int H, int N, cudaStream_t stream) {
+                              float* qk, float* dec, float* beta, int n_tokens, int G, int H, int N, int head_decay,
+                              cudaStream_t stream) {
     if (n_tokens <= 0) return PLM_OK;
     if (G <= 0 || H <= 0 || N <= 0) return PLM_ERR_SHAPE;
+    const int ND = head_decay ? 1 : N;
     if (dtype == PLM_F32)
         return plm_status_of(launch_pdl(delta_prep_kernel<float>, dim3(n_tokens), dim3(128), 0, stream, (const float*)q, ldq,
                                         (const float*)k, ldk, (const float*)z, ldz, (const float*)braw, ldb, a_log, dt_bias, l2_eps,
-                                        q_scale, qn, kn, qk, dec, beta, G, H, N));
+                                        q_scale, qn, kn, qk, dec, beta, G, H, N, ND));
     if (dtype == PLM_BF16)
         return plm_status_of(launch_pdl(delta_prep_kernel<bf16>, dim3(n_tokens), dim3(128), 0, stream, (const bf16*)q, ldq,
                                         (const bf16*)k, ldk, (const bf16*)z, ldz, (const bf16*)braw, ldb, a_log, dt_bias, l2_eps,
-                                        q_scale, qn, kn, qk, dec, beta, G, H, N));
+                                        q_scale, qn, kn, qk, dec, beta, G, H, N, ND));
     return PLM_ERR_DTYPE;
 }
 
 // The delta rule per head, token by token, state S [N, P] in fp32:
 //   S <- S + diag(expm1(dec_t)) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t  (the read-out sees the
-//   write; dec_t is the decay's logarithm).
+//   write; dec_t is the decay's logarithm, ND = N of them a head or one).
 // The columns of S do not meet, so a block takes 32 of them for one (sequence, head): a warp holds 8 columns, the N rows of
 // a column are dealt to 4 lanes (row n with lane n % 4), NR values of the state a thread.  Both sums over the rows,
 // k . (dec S) and q . (dec S), are taken in one pass before the write, and o = q . (dec S) + (q . k) u.
@@ -1274,7 +1277,7 @@ __global__ void __launch_bounds__(128)
 delta_scan_kernel(const float* qn, const float* kn, const float* qk,
                   const float* dec, const float* beta, const T* v, long ldv,
                   float* __restrict__ state, long state_stride, float* __restrict__ y, const int* seq_start,
-                  const int* seq_slot, int H, int N, int P, int heads_per_group, int TC) {
+                  const int* seq_slot, int H, int N, int P, int heads_per_group, int ND, int TC) {
     constexpr int NP = NR * 4;
     extern __shared__ __align__(16) float smem[];
     float* qs = smem;                         // [TC][NP]
@@ -1311,7 +1314,7 @@ delta_scan_kernel(const float* qn, const float* kn, const float* qk,
             const bool in = n < N;
             qs[idx] = in ? qn[(row * G + g) * N + n] : 0.f;
             ks[idx] = in ? kn[(row * G + g) * N + n] : 0.f;
-            gs[idx] = in ? expm1f(dec[(row * H + h) * N + n]) : 0.f;
+            gs[idx] = in ? expm1f(dec[(row * H + h) * ND + (ND > 1 ? n : 0)]) : 0.f;
         }
         for (int idx = threadIdx.x; idx < nt * DELTA_COLS; idx += 128) {
             const int tt = idx / DELTA_COLS, cc = idx - tt * DELTA_COLS;
@@ -1355,30 +1358,32 @@ delta_scan_kernel(const float* qn, const float* kn, const float* qk,
 template <typename T, int NR>
 static int delta_scan_launch(const float* qn, const float* kn, const float* qk, const float* dec, const float* beta, const void* v,
                              long ldv, float* state, long state_stride, float* y, const int* seq_start, const int* seq_slot,
-                             int n_seqs, int H, int N, int P, int heads_per_group, cudaStream_t stream) {
+                             int n_seqs, int H, int N, int P, int heads_per_group, int ND, cudaStream_t stream) {
     const int TC = NR <= 32 ? 16 : 8;
     const size_t smem = ((size_t)TC * NR * 4 * 3 + (size_t)TC * DELTA_COLS + 2 * TC) * sizeof(float);
     if (smem > 48 * 1024)
         cudaFuncSetAttribute(delta_scan_kernel<T, NR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     const unsigned grid = (unsigned)((long)n_seqs * H * ((P + DELTA_COLS - 1) / DELTA_COLS));
     return plm_status_of(launch_pdl(delta_scan_kernel<T, NR>, dim3(grid), dim3(128), smem, stream, qn, kn, qk, dec, beta,
-                                    (const T*)v, ldv, state, state_stride, y, seq_start, seq_slot, H, N, P, heads_per_group, TC));
+                                    (const T*)v, ldv, state, state_stride, y, seq_start, seq_slot, H, N, P, heads_per_group, ND, TC));
 }
 
 extern "C" int plm_delta_scan(const float* qn, const float* kn, const float* qk, const float* dec, const float* beta,
                               const void* v, int dtype, long ldv, float* state, long state_stride, float* y, const int* seq_start,
-                              const int* seq_slot, int n_seqs, int H, int N, int P, int heads_per_group, cudaStream_t stream) {
+                              const int* seq_slot, int n_seqs, int H, int N, int P, int heads_per_group, int head_decay,
+                              cudaStream_t stream) {
     if (n_seqs <= 0) return PLM_OK;
     if (H <= 0 || N <= 0 || P <= 0 || heads_per_group <= 0 || H % heads_per_group) return PLM_ERR_SHAPE;
     if (N > 256) return PLM_ERR_UNSUPPORTED;
+    const int ND = head_decay ? 1 : N;
     if (dtype != PLM_F32 && dtype != PLM_BF16) return PLM_ERR_DTYPE;
     const int nr = (N + 3) / 4;
 #define DS(NR_)                                                                                                                 \
     return dtype == PLM_F32                                                                                                     \
                ? delta_scan_launch<float, NR_>(qn, kn, qk, dec, beta, v, ldv, state, state_stride, y, seq_start, seq_slot, n_seqs, \
-                                               H, N, P, heads_per_group, stream)                                               \
+                                               H, N, P, heads_per_group, ND, stream)                                           \
                : delta_scan_launch<bf16, NR_>(qn, kn, qk, dec, beta, v, ldv, state, state_stride, y, seq_start, seq_slot, n_seqs, \
-                                              H, N, P, heads_per_group, stream)
+                                              H, N, P, heads_per_group, ND, stream)
     if (nr <= 4) DS(4);
     if (nr <= 8) DS(8);
     if (nr <= 16) DS(16);
@@ -1408,13 +1413,15 @@ static inline int delta_chunk_np(int N) { return N <= 32 ? 32 : N <= 64 ? 64 : N
 
 // grid (chunk of the sequence, sequence, head).  ws per (slot, head): Kp [C][NP] | Qp [C][NP] | Ke [C][NP] | A^T [C][C] | M^T [C][C]
 // | e^{L_C} [NP], NP = delta_chunk_np(N), the padding zero.  A sequence's chunk c lives in slot seq_start / C + sequence + c.
+// HEAD: one decay a head (lgd [T, H]): L is a number per token, so A and M are plain dot products times one exponential.
+template <bool HEAD>
 __global__ void __launch_bounds__(256)
 delta_chunk_prep_kernel(const float* qn, const float* kn, const float* lgd,
                         float* __restrict__ ws, const int* seq_start, int H, int N, int NP, int heads_per_group) {
     constexpr int C = DELTA_CHUNK;
     extern __shared__ __align__(16) float smem[];
     float* cum = smem;                  // [C][N]
-    float* ks = cum + (long)C * N;
+    float* ks = cum + (long)C * (HEAD ? 1 : N);
     float* qs = ks + (long)C * N;
     pdl_launch_dependents();
     pdl_wait();
@@ -1431,14 +1438,16 @@ delta_chunk_prep_kernel(const float* qn, const float* kn, const float* lgd,
         const long row = t0 + tt;
         ks[idx] = in ? kn[(row * G + g) * N + n] : 0.f;
         qs[idx] = in ? qn[(row * G + g) * N + n] : 0.f;
-        cum[idx] = in ? lgd[(row * H + h) * N + n] : 0.f;
+        if (!HEAD) cum[idx] = in ? lgd[(row * H + h) * N + n] : 0.f;
     }
+    if (HEAD && threadIdx.x < C) cum[threadIdx.x] = threadIdx.x < nt ? lgd[(long)(t0 + threadIdx.x) * H + h] : 0.f;
     __syncthreads();
-    for (int n = threadIdx.x; n < N; n += 256) {
+    const int nd = HEAD ? 1 : N;
+    for (int n = threadIdx.x; n < nd; n += 256) {
         float acc = 0.f;
         for (int tt = 0; tt < C; ++tt) {
-            acc += cum[tt * N + n];
-            cum[tt * N + n] = acc;
+            acc += cum[tt * nd + n];
+            cum[tt * nd + n] = acc;
         }
     }
     __syncthreads();
@@ -1453,14 +1462,15 @@ delta_chunk_prep_kernel(const float* qn, const float* kn, const float* lgd,
         const int tt = idx / NP, n = idx - tt * NP;
         float kp = 0.f, qp = 0.f, ke = 0.f;
         if (n < N) {
-            const float l = cum[tt * N + n], e = expf(l), kv = ks[tt * N + n];
+            const int dn = HEAD ? 0 : n;
+            const float l = cum[tt * nd + dn], e = expf(l), kv = ks[tt * N + n];
             kp = kv * e;
             qp = qs[tt * N + n] * e;
-            ke = kv * expf(cum[(C - 1) * N + n] - l);
+            ke = kv * expf(cum[(C - 1) * nd + dn] - l);
         }
         Kp[idx] = kp, Qp[idx] = qp, Ke[idx] = ke;
     }
-    for (int n = threadIdx.x; n < NP; n += 256) ge[n] = n < N ? expf(cum[(C - 1) * N + n]) : 0.f;
+    for (int n = threadIdx.x; n < NP; n += 256) ge[n] = n < N ? expf(cum[(C - 1) * nd + (HEAD ? 0 : n)]) : 0.f;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     // both stored transposed, [s][t], so that lanes that hold different t read different banks; zero where s > t (A: s >= t)
     for (int i = warp; i < C * C; i += 8) {
@@ -1468,11 +1478,15 @@ delta_chunk_prep_kernel(const float* qn, const float* kn, const float* lgd,
         float a = 0.f, m = 0.f;
         if (s <= t) {
             for (int n = lane; n < N; n += 32) {
-                const float kk = ks[s * N + n] * expf(cum[t * N + n] - cum[s * N + n]);
+                const float kk = HEAD ? ks[s * N + n] : ks[s * N + n] * expf(cum[t * N + n] - cum[s * N + n]);
                 a = fmaf(ks[t * N + n], kk, a);
                 m = fmaf(qs[t * N + n], kk, m);
             }
             a = warp_sum(a), m = warp_sum(m);
+            if (HEAD) {
+                const float e = expf(cum[t] - cum[s]);
+                a *= e, m *= e;
+            }
         }
         if (lane == 0) A[s * C + t] = s < t ? a : 0.f, M[s * C + t] = m;
     }
@@ -1657,18 +1671,17 @@ static int delta_chunk_launch(const float* ws, const float* beta, const void* v,
 extern "C" int plm_delta_chunk_scan(const float* qn, const float* kn, const float* dec, const float* beta, const void* v,
                                     int dtype, long ldv, float* state, long state_stride, float* y, float* ws,
                                     const int* seq_start, const int* seq_slot, int n_seqs, int max_new, int H, int N, int P,
-                                    int heads_per_group, cudaStream_t stream) {
+                                    int heads_per_group, int head_decay, cudaStream_t stream) {
     if (n_seqs <= 0 || max_new <= 0) return PLM_OK;
     if (H <= 0 || N <= 0 || P <= 0 || heads_per_group <= 0 || H % heads_per_group) return PLM_ERR_SHAPE;
     if (N > 256) return PLM_ERR_UNSUPPORTED;
     if (dtype != PLM_F32 && dtype != PLM_BF16) return PLM_ERR_DTYPE;
     const int NP = delta_chunk_np(N);
-    const size_t prep_smem = (size_t)3 * DELTA_CHUNK * N * sizeof(float);
-    if (prep_smem > 48 * 1024)
-        cudaFuncSetAttribute(delta_chunk_prep_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep_smem);
+    const size_t prep_smem = (size_t)DELTA_CHUNK * (head_decay ? 2 * N + 1 : 3 * N) * sizeof(float);
+    auto prep = head_decay ? delta_chunk_prep_kernel<true> : delta_chunk_prep_kernel<false>;
+    if (prep_smem > 48 * 1024) cudaFuncSetAttribute(prep, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)prep_smem);
     const dim3 pgrid((unsigned)((max_new + DELTA_CHUNK - 1) / DELTA_CHUNK), (unsigned)n_seqs, (unsigned)H);
-    int e = plm_status_of(launch_pdl(delta_chunk_prep_kernel, pgrid, dim3(256), prep_smem, stream, qn, kn, dec, ws, seq_start, H, N,
-                                     NP, heads_per_group));
+    int e = plm_status_of(launch_pdl(prep, pgrid, dim3(256), prep_smem, stream, qn, kn, dec, ws, seq_start, H, N, NP, heads_per_group));
     if (e != PLM_OK) return e;
 #define DCS(NR_, ST_)                                                                                                     \
     return delta_chunk_launch<NR_, ST_>(ws, beta, v, dtype == PLM_F32 ? 1 : 0, ldv, state, state_stride, y, seq_start, seq_slot, \

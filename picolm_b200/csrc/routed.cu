@@ -10,7 +10,7 @@
 //   weights  w = s_chosen / (sum of the chosen s + 1e-20) * scale, or s_chosen * scale   (s without the correction)
 //   identity the router's last outputs may be experts without tensors whose output is their input: they take part in
 //            scores, groups and choice like the others, are left out of the sort, and enter the weighted sum as w * h
-//   expert   y = W_down (silu(W_gate h) * (W_up h)), no biases
+//   expert   y = W_down (silu(W_gate h) * (W_up h)), or without a gate y = W_down relu(W_up h)^2; no biases
 //   output   out[t] = sum_k w[t, k] y_(e[t, k])(h[t])  (+ gate[t] * shared[t] for an expert every token uses)
 //
 // Everything a later kernel needs of the choice stays on the device (nothing is read on the host, so the step can be
@@ -266,6 +266,7 @@ moe_align_kernel(const int* ids, int n_entries, int E, int BM, int* __restrict__
 // A tile of BM sorted rows times a tile of 64 columns of its expert's weights, k ascending, fp32 sums.
 // MODE 0 (gate and up): row r of the tile is token sorted[...] / top of `a` [T, K]; w is [E][2 N][K], an expert's
 //   N gate rows followed by its N up rows; out[tile * BM + r, n] = silu(g) * u in To.
+// MODE 2 (up, no gate): the same rows of `a`; w is [E][N][K]; out[tile * BM + r, n] = relu(u)^2 in To.
 // MODE 1 (down): row r of the tile is row tile * BM + r of `a` [max_tiles * BM, K]; w is [E][N][K];
 //   out[tile * BM + r, n] = sum in fp32 (the weighted sum per token comes after).
 constexpr int MG_BN = 64, MG_BK = 16;
@@ -273,6 +274,11 @@ constexpr int MG_BN = 64, MG_BK = 16;
 // where gate row n and up row n of an expert lie in its [2 N, K] matrix
 __device__ __forceinline__ int gate_row_of(int n, int N, int interleaved) { return interleaved ? (n >> 6) * 128 + (n & 63) : n; }
 __device__ __forceinline__ int up_row_of(int n, int N, int interleaved) { return interleaved ? (n >> 6) * 128 + 64 + (n & 63) : N + n; }
+
+__device__ __forceinline__ float relu_squared(float z) {
+    const float r = fmaxf(z, 0.f);
+    return r * r;
+}
 
 template <typename Ta, typename Tw, typename To, int BM, int MODE>
 __global__ void __launch_bounds__(256)
@@ -291,7 +297,7 @@ moe_gemm_kernel(const Ta* a, long lda, int top, const Tw* w, To* __restrict__ ou
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
     for (int r = tid; r < BM; r += 256) {
         const int entry = sorted[tile * BM + r];
-        a_off[r] = entry < 0 ? -1 : (MODE == 0 ? (long)(entry / top) * lda : (long)(tile * BM + r) * lda);
+        a_off[r] = entry < 0 ? -1 : (MODE != 1 ? (long)(entry / top) * lda : (long)(tile * BM + r) * lda);
     }
     __syncthreads();
     const Tw* wg = w + (size_t)e * (MODE == 0 ? 2 : 1) * N * K;
@@ -345,6 +351,8 @@ moe_gemm_kernel(const Ta* a, long lda, int top, const Tw* w, To* __restrict__ ou
                 // both branches rounded to the activations' type first, as a product that stores them would
                 const float g = to_f32<To>(from_f32<To>(acc[0][i][j])), u = to_f32<To>(from_f32<To>(acc[MODE == 0 ? 1 : 0][i][j]));
                 o[n] = from_f32<To>(g / (1.0f + expf(-g)) * u);
+            } else if (MODE == 2) {
+                o[n] = from_f32<To>(relu_squared(acc[0][i][j]));
             } else {
                 o[n] = from_f32<To>(acc[0][i][j]);
             }
@@ -395,7 +403,7 @@ moe_gemm_mma_kernel(const bf16* a, long lda, int top, const bf16* w, void* __res
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, c = lane & 3;
     if (tid < BM) {
         const int entry = sorted[tile * BM + tid];
-        a_off[tid] = entry < 0 ? -1 : (MODE == 0 ? (long)(entry / top) * lda : (long)(tile * BM + tid) * lda);
+        a_off[tid] = entry < 0 ? -1 : (MODE != 1 ? (long)(entry / top) * lda : (long)(tile * BM + tid) * lda);
     }
     const bf16* we = w + (size_t)e * NACC * N * K;
     const int n_base = blockIdx.y * MM_BN + warp * MM_NB * 8;
@@ -464,6 +472,8 @@ moe_gemm_mma_kernel(const bf16* a, long lda, int top, const bf16* w, void* __res
                     const float gv = __bfloat162float(__float2bfloat16_rn(acc[0][j][2 * half + i]));
                     const float uv = __bfloat162float(__float2bfloat16_rn(acc[NACC - 1][j][2 * half + i]));
                     reinterpret_cast<bf16*>(out_)[(size_t)(tile * BM + r) * ldo + n] = __float2bfloat16_rn(gv / (1.0f + expf(-gv)) * uv);
+                } else if (MODE == 2) {
+                    reinterpret_cast<bf16*>(out_)[(size_t)(tile * BM + r) * ldo + n] = __float2bfloat16_rn(relu_squared(acc[0][j][2 * half + i]));
                 } else {
                     reinterpret_cast<float*>(out_)[(size_t)(tile * BM + r) * ldo + n] = acc[0][j][2 * half + i];
                 }
@@ -655,7 +665,7 @@ extern "C" int plm_moe_align(const int* ids, int n_entries, int E, int bm, int* 
                                     sorted, where, max_tiles, n_skip));
 }
 
-// mode 0: gate/up with SiLU (a [T, K], out [max_tiles * bm, N] of a's type); mode 1: down (a [max_tiles * bm, K] of
+// mode 0: gate/up with SiLU (a [T, K], out [max_tiles * bm, N] of a's type); mode 2: up with a squared ReLU, likewise; mode 1: down (a [max_tiles * bm, K] of
 // `dtype`, out fp32).  bm 16 or 64.  dtype: a and w, PLM_F32 or PLM_BF16.
 // `interleaved` (mode 0): an expert's gate and up rows come in turns of 64 (64 gate rows, their 64 up rows, ...: the layout
 // of the tensor-core product with the activation in its epilogue) instead of all gate rows before all up rows.
@@ -676,6 +686,9 @@ extern "C" int plm_moe_gemm(const void* a, long lda, int top, const void* w, voi
         if (mode == 1)
             return plm_status_of(launch_pdl(moe_gemm_mma_kernel<1>, mgrid, mnt, smem, stream, (const bf16*)a, lda, top, (const bf16*)w,
                                             out, ldo, tile_expert, sorted, N, K, interleaved));
+        if (mode == 2)
+            return plm_status_of(launch_pdl(moe_gemm_mma_kernel<2>, mgrid, mnt, smem, stream, (const bf16*)a, lda, top, (const bf16*)w,
+                                            out, ldo, tile_expert, sorted, N, K, interleaved));
         return PLM_ERR_UNSUPPORTED;
     }
     const dim3 grid(max_tiles, (N + MG_BN - 1) / MG_BN), nt(256);
@@ -685,9 +698,11 @@ extern "C" int plm_moe_gemm(const void* a, long lda, int top, const void* w, voi
     if (dtype == PLM_F32) {
         if (mode == 0) { if (bm == 16) MG_LAUNCH(float, float, 16, 0); else MG_LAUNCH(float, float, 64, 0); }
         if (mode == 1) { if (bm == 16) MG_LAUNCH(float, float, 16, 1); else MG_LAUNCH(float, float, 64, 1); }
+        if (mode == 2) { if (bm == 16) MG_LAUNCH(float, float, 16, 2); else MG_LAUNCH(float, float, 64, 2); }
     } else if (dtype == PLM_BF16) {
         if (mode == 0) { if (bm == 16) MG_LAUNCH(bf16, bf16, 16, 0); else MG_LAUNCH(bf16, bf16, 64, 0); }
         if (mode == 1) { if (bm == 16) MG_LAUNCH(bf16, float, 16, 1); else MG_LAUNCH(bf16, float, 64, 1); }
+        if (mode == 2) { if (bm == 16) MG_LAUNCH(bf16, bf16, 16, 2); else MG_LAUNCH(bf16, bf16, 64, 2); }
     } else {
         return PLM_ERR_DTYPE;
     }

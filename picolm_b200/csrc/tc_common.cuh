@@ -134,11 +134,20 @@ __device__ __forceinline__ float swiglu_bf16(float g, float u, float limit = 0.f
     return __fdividef(g, 1.0f + e) * u;
 }
 
-// What the bf16 store epilogue applies to a result before it is rounded: nothing, or with -DPLM_STORE_GELU_ERF (a build
-// variant for products with an activation that has no gate behind them) the exact GELU, 0.5 z (1 + erf(z / sqrt 2)),
+// What the bf16 store epilogue applies to a result before it is rounded: nothing, or in a build variant for products with
+// an activation that has no gate behind them: with -DPLM_STORE_RELU2 the square of ReLU, with -DPLM_STORE_GELU_ERF the exact GELU, 0.5 z (1 + erf(z / sqrt 2)),
 // with erfc(x) = t (a1 + t (a2 + t (a3 + t (a4 + t a5)))) e^(-x^2), t = 1 / (1 + p x), x >= 0: formula 7.1.26 of Abramowitz
 // and Stegun's Handbook of Mathematical Functions (absolute error below 1.5e-7, far below the bf16 rounding of results).
+#if defined(PLM_STORE_GELU_ERF) || defined(PLM_STORE_RELU2)
+#define PLM_STORE_ACT
+#endif
 template <typename OutT> __device__ __forceinline__ float store_act(float z) {
+#ifdef PLM_STORE_RELU2
+    if (sizeof(OutT) == 2) {
+        const float r = fmaxf(z, 0.0f);
+        return r * r;
+    }
+#endif
 #ifdef PLM_STORE_GELU_ERF
     if (sizeof(OutT) == 2) {
         const float x = fabsf(z) * 0.70710678118654752f;

@@ -21,10 +21,14 @@ _SIGNATURES = {
     "plm_embed_pair": [_vp, _vp, _vp, _i, _vp, _l, _vp, _vp, _vp, _vp, _i, _i, _i, _l, _l, _l, _f, _vp],
     "plm_joined_post_pre_norm": [_vp, _vp, _vp, _vp, _vp, _f, _vp, _vp, _vp, _i, _i, _i, _f, _f, _f, _f, _vp],
     "plm_heads_store": [_vp, _i, _l, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
-    "plm_decay_step": [_vp, _vp, _vp, _i, _l, _l, _l, _vp, _vp, _l, _vp, _l, _vp, _i, _i, _i, _i, _i, _vp],
+    "plm_embed_norm": [_vp, _vp, _vp, _i, _vp, _i, _i, _i, _f, _vp],
+    "plm_squash": [_vp, _l, _f, _f, _vp],
+    "plm_decay_step": [_vp, _vp, _vp, _i, _l, _l, _l, _vp, _vp, _l, _vp, _l, _vp, _i, _i, _i, _i, _i, _vp, _vp, _vp, _i, _f, _vp],
+    "plm_rotate_rows": [_vp, _vp, _vp, _i, _l, _l, _l, _vp, _vp, _vp, _i, _f, _vp, _vp, _i, _i, _i, _i, _vp],
     "plm_decay_chunk_plan": [_i, _i, _i, _i, _i, _i, _vp],
-    "plm_decay_chunk_scan": [_vp, _vp, _vp, _l, _l, _l, _vp, _vp, _l, _vp, _l, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _i, _vp],
-    "plm_gelu_erf": [_vp, _vp, _i, _l, _vp],
+    "plm_decay_chunk_scan": [_vp, _vp, _vp, _l, _l, _l, _vp, _vp, _l, _vp, _l, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _i, _i, _vp, _vp,
+                             _vp, _i, _f, _vp],
+    "plm_plain_act": [_vp, _vp, _i, _i, _l, _vp],
     "plm_rmsnorm": [_vp, _vp, _vp, _i, _vp, _i, _vp, _i, _i, _f, _vp],
     "plm_post_pre_norm": [_vp, _vp, _vp, _vp, _i, _vp, _i, _i, _i, _f, _f, _vp],
     "plm_swiglu": [_vp, _vp, _i, _i, _i, _i, _f, _f, _vp],
@@ -77,9 +81,9 @@ _SIGNATURES = {
     "plm_causal_conv": [_vp, _i, _l, _vp, _vp, _vp, _l, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp, _i, _vp],
     "plm_rglru_gates": [_vp, _i, _l, _vp, _vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
     "plm_diag_scan": [_vp, _vp, _vp, _i, _l, _vp, _vp, _l, _vp, _vp, _vp, _i, _i, _i, _vp],
-    "plm_delta_prep": [_vp, _l, _vp, _l, _vp, _l, _vp, _l, _i, _vp, _vp, _f, _f, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
-    "plm_delta_chunk_scan": [_vp, _vp, _vp, _vp, _vp, _i, _l, _vp, _l, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
-    "plm_delta_scan": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _l, _vp, _l, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
+    "plm_delta_prep": [_vp, _l, _vp, _l, _vp, _l, _vp, _l, _i, _vp, _vp, _f, _f, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
+    "plm_delta_chunk_scan": [_vp, _vp, _vp, _vp, _vp, _i, _l, _vp, _l, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
+    "plm_delta_scan": [_vp, _vp, _vp, _vp, _vp, _vp, _i, _l, _vp, _l, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp],
     "plm_linear_scan": [_vp, _vp, _vp, _vp, _i, _l, _l, _l, _l, _i, _vp, _vp, _vp, _f, _f, _vp, _l, _vp, _l, _vp, _vp,
                         _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _i, _vp],
     "plm_sigmoid_decay": [_vp, _i, _l, _vp, _f, _vp, _i, _i, _vp],

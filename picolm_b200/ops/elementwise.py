@@ -20,6 +20,31 @@ def embed(tokens: torch.Tensor, table: torch.Tensor, out: Optional[torch.Tensor]
     return out
 
 
+def embed_norm(tokens: torch.Tensor, table: torch.Tensor, weight: torch.Tensor, eps: float) -> torch.Tensor:
+    """out[t, :] = RMSNorm(float(table[tokens[t], :])) with `weight` [d]: the fp32 residual stream of a design whose
+    embedding passes a norm first."""
+    _i32(tokens, "tokens")
+    _dev(table, "table"), _dev(weight, "weight")
+    n, (vocab, d) = tokens.numel(), table.shape
+    if weight.shape != (d,) or weight.dtype != table.dtype:
+        raise KernelError(f"embed_norm: the norm's weight must be [{d}] of {table.dtype}")
+    out = torch.empty((n, d), dtype=torch.float32, device=table.device)
+    _check(_fn("elementwise", "plm_embed_norm")(_p(tokens), _p(table), _p(weight), _dt(table, "table"), _p(out), n, d, vocab,
+                                                float(eps), _stream()), f"embed_norm T={n} d={d}",
+           nbytes=n * d * (4 + table.element_size()))
+    return out
+
+
+def squash(x: torch.Tensor, scale: float, cap: float) -> torch.Tensor:
+    """x = cap * tanh(x * scale / cap) in place for float32 `x` (logits that are scaled and then kept inside -cap .. cap);
+    returns x."""
+    _dev(x, "x")
+    if x.dtype != torch.float32 or not cap > 0:
+        raise KernelError("squash takes float32 values and a positive cap")
+    _check(_fn("elementwise", "plm_squash")(_p(x), x.numel(), float(scale), float(cap), _stream()), "squash", nbytes=8 * x.numel())
+    return x
+
+
 def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype,
             delta: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
             out: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -131,13 +156,23 @@ def joined_post_pre_norm(x: torch.Tensor, a: torch.Tensor, w_a: torch.Tensor, ep
     return out
 
 
-def gelu_erf(x: torch.Tensor) -> torch.Tensor:
-    """0.5 x (1 + erf(x / sqrt 2)) element by element, in x's type (float32 inside)."""
+# activations of a map without a gate: "gelu_erf" 0.5 x (1 + erf(x / sqrt 2)), "relu2" relu(x)^2
+PLAIN_ACTIVATIONS = ("gelu_erf", "relu2")
+
+
+def plain_act(x: torch.Tensor, activation: str) -> torch.Tensor:
+    """An activation of `PLAIN_ACTIVATIONS` element by element, in x's type (float32 inside)."""
     _dev(x, "x")
+    if activation not in PLAIN_ACTIVATIONS:
+        raise KernelError(f"activation {activation!r} without a gate has no kernel; known: {', '.join(PLAIN_ACTIVATIONS)}")
     out = torch.empty_like(x)
-    _check(_fn("elementwise", "plm_gelu_erf")(_p(x), _p(out), _dt(x, "x"), x.numel(), _stream()), "gelu_erf",
-           nbytes=2 * x.numel() * x.element_size())
+    _check(_fn("elementwise", "plm_plain_act")(_p(x), _p(out), _dt(x, "x"), PLAIN_ACTIVATIONS.index(activation), x.numel(), _stream()),
+           activation, nbytes=2 * x.numel() * x.element_size())
     return out
+
+
+def gelu_erf(x: torch.Tensor) -> torch.Tensor:
+    return plain_act(x, "gelu_erf")
 
 
 def gather_rows(x: torch.Tensor, rows: torch.Tensor) -> torch.Tensor:

@@ -10,11 +10,7 @@ from . import chain as _chain
 from ._lib import (SM_COUNT, KernelError, _check, _dev, _dt, _fn, _p, _stream, status_word, stream_space,
                    stream_space_enabled)
 from .chain import LazyRows
-from .elementwise import gelu_erf
-
-
-# activations without a gate that a product can apply to its own results
-PLAIN_ACTIVATIONS = ("gelu_erf",)
+from .elementwise import PLAIN_ACTIVATIONS, plain_act          # (activations a product can apply to its own results)
 
 
 def _work(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, extra: int = 0) -> dict:
@@ -71,7 +67,7 @@ def _gated_library(name: str, flags: tuple, activation: str):
 # activation -> (the variant's name, its compile flag)
 _GATE_VARIANTS = {"gelu_tanh": ("gelu", "-DPLM_GATE_GELU"), "swish_clamped": ("clamped", "-DPLM_GATE_CLAMPED"),
                   # (not a gate: what the store epilogue applies, see `linear_act`)
-                  "gelu_erf": ("gelu_erf", "-DPLM_STORE_GELU_ERF")}
+                  "gelu_erf": ("gelu_erf", "-DPLM_STORE_GELU_ERF"), "relu2": ("relu2", "-DPLM_STORE_RELU2")}
 
 
 def _set_gate_constants(lib, flags, activation: str, limit: float, slope: float) -> None:
@@ -401,7 +397,7 @@ def linear_act(a, w: torch.Tensor, out_dtype: torch.dtype, activation: str):
         if x.shape[0] <= 64:
             return gemm_tc_skinny(x, w, out_dtype, store_act=activation)
         return gemm_tc_wide(x, w, out_dtype, pair=pair_pays(x.shape[0], w.shape[0], x.shape[1], 0), store_act=activation)
-    return gelu_erf(linear(x, w, out_dtype))
+    return plain_act(linear(x, w, out_dtype), activation)
 
 
 def linear(a, w: torch.Tensor, out_dtype: torch.dtype, defer: bool = False):

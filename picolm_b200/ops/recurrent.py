@@ -175,22 +175,30 @@ def decay_chunk_supported(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, key
 
 def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, powers: torch.Tensor,
                state: torch.Tensor, step, heads: int, key_dim: int, value_dim: int,
-               activation: Optional[str] = None) -> torch.Tensor:
+               activation: Optional[str] = None, rotation=None, k_scale: Optional[float] = None) -> torch.Tensor:
     """S_t = d_h S_(t-1) + k_t v_t^T, y_t = S_t^T q_t over each sequence's tokens, with one constant decay a head; float32
     [T, heads * value_dim].  q, k [T, heads * key_dim], v [T, heads * value_dim] (column slices will do); with
     `activation="silu"` they pass SiLU on their way in.  `decay` float32 [heads], `powers` its table (`decay_powers`);
+    `rotation` (`ops.Rotation`, halves paired) turns the leading `rotary_dim` components of every head of q and k by the
+    token's position and `k_scale` multiplies k, on the way in, in float32 and without a rounding behind (either of
+    them given: no activation).
     `state` float32 [slots, >= heads * key_dim * value_dim] is carried on.  Steps with prompts in bfloat16 run 64 tokens
     at a time on the tensor cores where the sizes allow it, steps of single tokens stream the state through once,
     everything else goes token by token (`linear_scan`)."""
     H, N, P = heads, key_dim, value_dim
     T = v.shape[0]
-    if step.is_decode and step.n_tokens == step.n_seqs and P % 4 == 0 and state.stride(0) % 4 == 0 and state.data_ptr() % 16 == 0:
-        return _decay_step(q, k, v, decay, state, step, H, N, P, activation)
-    if step.max_new < DECAY_CHUNK_FROM or not decay_chunk_supported(q, k, v, N, P) or state.stride(0) % 4:
-        return linear_scan(q, k, v, None, DECAY_CONST, decay, None, None, 1.0, 1.0, state, step, H, N, P, activation=activation)
-    ldq, ldk, ldv, lds = _cols(q, "q"), _cols(k, "k"), _cols(v, "v"), _cols(state, "state")
     if q.shape != (T, H * N) or k.shape != (T, H * N) or v.shape != (T, H * P) or activation not in (None, "silu"):
         raise KernelError("decay_scan: q, k, v do not have the shapes the head counts imply, or the activation is not known (silu)")
+    turn = _Turn(rotation, k_scale, activation, step, N) if rotation is not None or k_scale is not None else None
+    if step.is_decode and step.n_tokens == step.n_seqs and P % 4 == 0 and state.stride(0) % 4 == 0 and state.data_ptr() % 16 == 0:
+        return _decay_step(q, k, v, decay, state, step, H, N, P, activation, turn)
+    chunked = decay_chunk_supported(q, k, v, N, P) and state.stride(0) % 4 == 0
+    if turn is not None and not chunked:
+        q, k, v = _turned_rows(q, k, v, turn, step, H, N, P)
+        return linear_scan(q, k, v, None, DECAY_CONST, decay, None, None, 1.0, 1.0, state, step, H, N, P)
+    if turn is None and (step.max_new < DECAY_CHUNK_FROM or not chunked):
+        return linear_scan(q, k, v, None, DECAY_CONST, decay, None, None, 1.0, 1.0, state, step, H, N, P, activation=activation)
+    ldq, ldk, ldv, lds = _cols(q, "q"), _cols(k, "k"), _cols(v, "v"), _cols(state, "state")
     _f32(powers, "powers", H * (DECAY_CHUNK + 1))
     if state.dtype != torch.float32 or state.shape[1] < H * N * P:
         raise KernelError("decay_scan: the state must be float32 with heads * key_dim * value_dim values a row")
@@ -199,27 +207,67 @@ def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.T
     seg_state = torch.empty((step.n_seqs, n_segs, H * N * P), dtype=torch.float32, device=v.device) if n_segs > 1 else None
     _check(_fn("decay_chunk", "plm_decay_chunk_scan")(
         _p(q), _p(k), _p(v), ldq, ldk, ldv, _p(powers), _p(state), lds, _p(y), H * P, _p(step.seq_start), _p(step.seq_slot),
-        step.n_seqs, H, N, P, seg_len, n_segs, _p(seg_state), 1 if activation == "silu" else 0, _stream()),
-        f"decay_chunk_scan T={T} H={H} N={N} P={P}" + (f" in {n_segs} segments" if n_segs > 1 else ""),
+        step.n_seqs, H, N, P, seg_len, n_segs, _p(seg_state), 1 if activation == "silu" else 0, *_turn_args(turn, step, True),
+        _stream()),
+        f"decay_chunk_scan{' rotated' if turn is not None else ''} T={T} H={H} N={N} P={P}" + (f" in {n_segs} segments" if n_segs > 1 else ""),
         kernels=3 if n_segs > 1 else 1,
         nbytes=T * (2 * H * N + H * P) * v.element_size() + T * H * P * 4 + 2 * step.n_seqs * H * N * P * 4,
         flops=2 * T * H * (DECAY_CHUNK // 2 * (N + P) + 2 * N * P))
     return y
 
 
-def _decay_step(q, k, v, decay, state, step, H, N, P, activation):
+class _Turn:
+    """A rotation and a factor on the keys, as `decay_scan`'s kernels take them."""
+    __slots__ = ("cos", "sin", "half", "k_scale")
+
+    def __init__(self, rotation, k_scale, activation, step, key_dim):
+        if activation is not None:
+            raise KernelError("decay_scan: queries and keys are rotated or pass an activation, not both")
+        self.cos = self.sin = None
+        self.half, self.k_scale = 0, 1.0 if k_scale is None else float(k_scale)
+        if rotation is not None and rotation.cos is not None:
+            self.cos, self.sin, self.half = rotation.cos, rotation.sin, rotation.rotary_dim // 2
+            if (rotation.pairing != "half" or 2 * self.half > key_dim or self.cos.dtype != torch.float32
+                    or self.cos.shape[1] != self.half or self.sin.shape != self.cos.shape):
+                raise KernelError("decay_scan: the rotation must pair halves, fit a head, and have float32 tables [positions, rotary_dim / 2]")
+            if step.max_position >= self.cos.shape[0]:
+                raise KernelError(f"position {step.max_position} lies beyond the rotary table")
+
+
+def _turn_args(turn, step, with_flag: bool):
+    flag = [1 if turn is not None else 0] if with_flag else []
+    if turn is None:
+        return flag + [None, None, None, 0, 1.0]
+    return flag + [_p(turn.cos), _p(turn.sin), _p(step.tok_pos), turn.half, turn.k_scale]
+
+
+def _turned_rows(q, k, v, turn, step, H, N, P):
+    """q, k rotated (k scaled) and v, float32 each, for the walk token by token."""
+    ldq, ldk, ldv = _cols(q, "q"), _cols(k, "k"), _cols(v, "v")
+    T = v.shape[0]
+    if not (q.dtype == k.dtype == v.dtype):
+        raise KernelError("decay_scan: q, k and v differ in type")
+    qk = torch.empty((T, 2 * H * N), dtype=torch.float32, device=q.device)
+    vo = torch.empty((T, H * P), dtype=torch.float32, device=q.device) if v.dtype != torch.float32 else None
+    _check(_fn("decay_chunk", "plm_rotate_rows")(
+        _p(q), _p(k), _p(v), _dt(q, "q"), ldq, ldk, ldv, *_turn_args(turn, step, False), _p(qk), _p(vo), T, H, N, P, _stream()),
+        f"rotate_rows T={T} H={H} N={N}", nbytes=T * H * 2 * N * (q.element_size() + 4))
+    return qk[:, :H * N], qk[:, H * N:], vo if vo is not None else v
+
+
+def _decay_step(q, k, v, decay, state, step, H, N, P, activation, turn=None):
     ldq, ldk, ldv, lds = _cols(q, "q"), _cols(k, "k"), _cols(v, "v"), _cols(state, "state")
     T = v.shape[0]
-    if (q.shape != (T, H * N) or k.shape != (T, H * N) or v.shape != (T, H * P) or not (q.dtype == k.dtype == v.dtype)
-            or activation not in (None, "silu")):
-        raise KernelError("decay_scan: q, k, v do not have the shapes the head counts imply, differ in type, or the activation is not known (silu)")
+    if not (q.dtype == k.dtype == v.dtype):
+        raise KernelError("decay_scan: q, k and v differ in type")
     _f32(decay, "decay", H)
     if state.dtype != torch.float32 or state.shape[1] < H * N * P:
         raise KernelError("decay_scan: the state must be float32 with heads * key_dim * value_dim values a row")
     y = torch.empty((T, H * P), dtype=torch.float32, device=v.device)
     _check(_fn("decay_chunk", "plm_decay_step")(
         _p(q), _p(k), _p(v), _dt(v, "v"), ldq, ldk, ldv, _p(decay), _p(state), lds, _p(y), H * P, _p(step.seq_slot), T, H, N, P,
-        1 if activation == "silu" else 0, _stream()), f"decay_step T={T} H={H} N={N} P={P}",
+        1 if activation == "silu" else 0, *_turn_args(turn, step, False), _stream()),
+        f"decay_step{' rotated' if turn is not None else ''} T={T} H={H} N={N} P={P}",
         nbytes=T * H * (8 * N * P + (2 * N + P) * v.element_size() + 4 * P), flops=4 * T * H * N * P)
     return y
 
@@ -428,40 +476,43 @@ def delta_chunk_workspace(n_tokens: int, n_seqs: int, heads: int, key_dim: int) 
 
 
 def delta_prep(q: torch.Tensor, k: torch.Tensor, z: torch.Tensor, b_raw: torch.Tensor, a_log: torch.Tensor,
-               dt_bias: torch.Tensor, l2_eps: float, q_scale: float, heads: int, key_dim: int, heads_per_group: int = 1):
+               dt_bias: torch.Tensor, l2_eps: float, q_scale: float, heads: int, key_dim: int, heads_per_group: int = 1,
+               head_decay: bool = False):
     """What the gated delta rule's recurrence takes, per token in float32 from the convolved projections (all of one
     type, column slices will do): q, k [T, groups * key_dim] made unit vectors per group (`x / sqrt(sum x^2 +
     l2_eps)`, q also times `q_scale`), their product q . k, the decays' logarithms `-exp(a_log[h]) softplus(z + dt_bias)`
-    for z [T, heads * key_dim] (the logarithm: a decay next to 1 keeps its distance from 1), and `sigmoid(b_raw)` for b_raw [T, heads].  Returns (qn, kn, qk, decay, beta)."""
+    for z [T, heads * key_dim] (the logarithm: a decay next to 1 keeps its distance from 1), and `sigmoid(b_raw)` for b_raw [T, heads].  With `head_decay`
+    there is one decay a head: z [T, heads], dt_bias [heads], decay [T, heads].  Returns (qn, kn, qk, decay, beta)."""
     T = q.shape[0]
     H, N = heads, key_dim
     if H % heads_per_group:
         raise KernelError("delta_prep: heads is not a multiple of heads_per_group")
     G = H // heads_per_group
+    ND = 1 if head_decay else N
     ldq, ldk, ldz, ldb = _cols(q, "q"), _cols(k, "k"), _cols(z, "z"), _cols(b_raw, "b_raw")
-    if (tuple(q.shape) != (T, G * N) or tuple(k.shape) != (T, G * N) or tuple(z.shape) != (T, H * N)
+    if (tuple(q.shape) != (T, G * N) or tuple(k.shape) != (T, G * N) or tuple(z.shape) != (T, H * ND)
             or tuple(b_raw.shape) != (T, H) or not (q.dtype == k.dtype == z.dtype == b_raw.dtype)):
         raise KernelError("delta_prep: q, k, z, b_raw do not have the shapes the head counts imply, or differ in type")
-    _f32(a_log, "a_log", H), _f32(dt_bias, "dt_bias", H * N)
+    _f32(a_log, "a_log", H), _f32(dt_bias, "dt_bias", H * ND)
     dev = q.device
     qn = torch.empty((T, G * N), dtype=torch.float32, device=dev)
     kn = torch.empty((T, G * N), dtype=torch.float32, device=dev)
     qk = torch.empty((T, G), dtype=torch.float32, device=dev)
-    dec = torch.empty((T, H * N), dtype=torch.float32, device=dev)
+    dec = torch.empty((T, H * ND), dtype=torch.float32, device=dev)
     beta = torch.empty((T, H), dtype=torch.float32, device=dev)
     _check(_fn("recurrent", "plm_delta_prep")(
         _p(q), ldq, _p(k), ldk, _p(z), ldz, _p(b_raw), ldb, _dt(q, "q"), _p(a_log), _p(dt_bias), float(l2_eps),
-        float(q_scale), _p(qn), _p(kn), _p(qk), _p(dec), _p(beta), T, G, H, N, _stream()), f"delta_prep T={T} H={H} N={N}",
-        nbytes=T * ((2 * G + H) * N * (q.element_size() + 4)))
+        float(q_scale), _p(qn), _p(kn), _p(qk), _p(dec), _p(beta), T, G, H, N, 1 if head_decay else 0, _stream()), f"delta_prep T={T} H={H} N={N}",
+        nbytes=T * ((2 * G * N + H * ND) * (q.element_size() + 4)))
     return qn, kn, qk, dec, beta
 
 
 def delta_scan(qn: torch.Tensor, kn: torch.Tensor, qk: torch.Tensor, decay: torch.Tensor, beta: torch.Tensor,
                v: torch.Tensor, state: torch.Tensor, step, heads: int, key_dim: int, value_dim: int,
-               heads_per_group: int = 1) -> torch.Tensor:
+               heads_per_group: int = 1, head_decay: bool = False) -> torch.Tensor:
     """The gated delta rule over each sequence's tokens, per head, state S [key_dim, value_dim] in float32:
       S <- diag(exp(decay_t)) S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
-    (the read-out sees the token's own write).  qn, kn, qk, decay (its logarithm), beta as `delta_prep` returns them; v [T, heads *
+    (the read-out sees the token's own write; with `head_decay` one decay a head).  qn, kn, qk, decay (its logarithm), beta as `delta_prep` returns them; v [T, heads *
     value_dim] (a column slice will do); `state` float32 [slots, >= heads * key_dim * value_dim] with contiguous
     rows holds S as [heads, key_dim, value_dim] and is carried on.  Returns o, float32 [T, heads * value_dim].
     A step whose longest sequence brings `DELTA_CHUNK_FROM` tokens or more runs chunk by chunk (two kernels: what does
@@ -472,8 +523,9 @@ def delta_scan(qn: torch.Tensor, kn: torch.Tensor, qk: torch.Tensor, decay: torc
     if H % heads_per_group:
         raise KernelError("delta_scan: heads is not a multiple of heads_per_group")
     G = H // heads_per_group
+    ND = 1 if head_decay else N
     ldv = _cols(v, "v")
-    for t, n, cols in ((qn, "qn", G * N), (kn, "kn", G * N), (qk, "qk", G), (decay, "decay", H * N), (beta, "beta", H)):
+    for t, n, cols in ((qn, "qn", G * N), (kn, "kn", G * N), (qk, "qk", G), (decay, "decay", H * ND), (beta, "beta", H)):
         _dev(t, n)
         if t.dtype != torch.float32 or tuple(t.shape) != (T, cols):
             raise KernelError(f"delta_scan: {n} must be float32 [{T}, {cols}]")
@@ -491,14 +543,14 @@ def delta_scan(qn: torch.Tensor, kn: torch.Tensor, qk: torch.Tensor, decay: torc
         ws = torch.empty((floats,), dtype=torch.float32, device=v.device)
         _check(_fn("recurrent", "plm_delta_chunk_scan")(
             _p(qn), _p(kn), _p(decay), _p(beta), _p(v), _dt(v, "v"), ldv, _p(state), lds, _p(y), _p(ws), _p(step.seq_start),
-            _p(step.seq_slot), step.n_seqs, int(step.max_new), H, N, P, heads_per_group, _stream()),
+            _p(step.seq_slot), step.n_seqs, int(step.max_new), H, N, P, heads_per_group, 1 if head_decay else 0, _stream()),
             f"delta_chunk_scan T={T} H={H} N={N} P={P}", kernels=2,
             nbytes=2 * floats * 4 + T * H * P * (4 + v.element_size()) + 2 * step.n_seqs * H * N * P * 4,
             flops=T * H * (6 * N * P + 6 * 32 * N + 4 * 32 * P))
         return y
     _check(_fn("recurrent", "plm_delta_scan")(
         _p(qn), _p(kn), _p(qk), _p(decay), _p(beta), _p(v), _dt(v, "v"), ldv, _p(state), lds, _p(y), _p(step.seq_start),
-        _p(step.seq_slot), step.n_seqs, H, N, P, heads_per_group, _stream()), f"delta_scan T={T} H={H} N={N} P={P}",
-        nbytes=T * (2 * G * N + 2 * H * N) * 4 + T * H * P * (4 + v.element_size()) + 2 * step.n_seqs * H * N * P * 4,
+        _p(step.seq_slot), step.n_seqs, H, N, P, heads_per_group, 1 if head_decay else 0, _stream()), f"delta_scan T={T} H={H} N={N} P={P}",
+        nbytes=T * (2 * G * N + H * N + H * ND) * 4 + T * H * P * (4 + v.element_size()) + 2 * step.n_seqs * H * N * P * 4,
         flops=8 * T * H * N * P)
     return y

@@ -8,6 +8,7 @@ from typing import Optional, Tuple
 import torch
 
 from ._lib import KernelError, _check, _dev, _dt, _fn, _i32, _p, _stream, status_word
+from .gemm import _gated_library
 
 
 def router_logits(h: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
@@ -115,6 +116,21 @@ def moe_gate_up(h: torch.Tensor, w_gate_up: torch.Tensor, pairs: SortedPairs, in
     return out
 
 
+def moe_up(h: torch.Tensor, w_up: torch.Tensor, pairs: SortedPairs) -> torch.Tensor:
+    """relu(W_up[e] h)^2 for every sorted pair, experts without a gate: `h` [T, d], `w_up` [E, F, d], both of one type;
+    [rows, F] of that type, in sorted order (the kernels of `moe_gate_up`)."""
+    _dev(h, "h"), _dev(w_up, "w_up")
+    E, F, d = w_up.shape
+    if h.dtype != w_up.dtype or h.shape != (pairs.n_tokens, d):
+        raise KernelError("moe_up: h [T, d] and w_up [E, F, d] of one type are expected")
+    out = torch.empty((pairs.rows, F), dtype=h.dtype, device=h.device)
+    _check(_fn("routed", "plm_moe_gemm")(
+        _p(h), d, pairs.top, _p(w_up), _p(out), F, _dt(h, "h"), 2, _p(pairs.tile_expert), _p(pairs.sorted),
+        pairs.max_tiles, pairs.bm, F, d, 0, _stream()), f"moe_up tiles<={pairs.max_tiles}x{pairs.bm} F={F} d={d}",
+        flops=2 * pairs.n_tokens * pairs.top * F * d, nbytes=w_up.numel() * w_up.element_size())
+    return out
+
+
 def moe_down(act: torch.Tensor, w_down: torch.Tensor, pairs: SortedPairs) -> torch.Tensor:
     """W_down[e] act for every sorted pair: `act` [rows, F] in sorted order, `w_down` [E, d, F]; float32 [rows, d]."""
     _dev(act, "act"), _dev(w_down, "w_down")
@@ -176,24 +192,36 @@ def moe_combine(y: torch.Tensor, pairs: SortedPairs, weights: torch.Tensor, shar
     return out
 
 
-def moe_tc_supported(h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor) -> bool:
-    """Whether the experts' products can run on tcgen05 (`moe_gate_up_tc`, `moe_down_tc`): bfloat16, an inner width
-    that is a multiple of 64, rows that TMA can address."""
-    E, F2, d = w_gate_up.shape
-    F = F2 // 2
-    return (h.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16 and w_down.dtype == torch.bfloat16
-            and F % 64 == 0 and d % 8 == 0 and d >= 64 and w_gate_up.data_ptr() % 16 == 0 and w_down.data_ptr() % 16 == 0)
+def moe_tc_supported(h: torch.Tensor, w_in: torch.Tensor, w_down: torch.Tensor) -> bool:
+    """Whether the experts' products can run on tcgen05 (`moe_gate_up_tc` or `moe_up_tc`, `moe_down_tc`): bfloat16, rows
+    that TMA can address, an inner width that is a multiple of 64 (without a gate: of 8 from 64 on).  `w_in`: [E, 2F, d]
+    with a gate, [E, F, d] without one."""
+    d = w_in.shape[2]
+    F = w_down.shape[2]
+    wide = F % 64 == 0 if w_in.shape[1] == 2 * F else F % 8 == 0 and F >= 64
+    return (h.dtype == torch.bfloat16 and w_in.dtype == torch.bfloat16 and w_down.dtype == torch.bfloat16
+            and wide and d % 8 == 0 and d >= 64 and w_in.data_ptr() % 16 == 0 and w_down.data_ptr() % 16 == 0)
 
 
-def _grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, pairs: SortedPairs, what: str) -> torch.Tensor:
+def _grouped(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int, pairs: SortedPairs, what: str,
+             store_act: Optional[str] = None) -> torch.Tensor:
     E, N, K = w.shape
     if pairs.bm != 128 or x.shape != (pairs.rows, K) or x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError(f"{what}: tiles of 128 sorted rows [rows, {K}] in bfloat16 are expected")
-    _check(_fn("gemm_tc_wide", "plm_gemm_tc_wide_grouped")(
+    lib, flags = _gated_library("gemm_tc_wide", (), store_act or "silu")
+    _check(_fn(lib, "plm_gemm_tc_wide_grouped", flags)(
         _p(x), _p(w), _p(out), _dt(out, "out"), epilogue, pairs.rows, N, K, K, K, out.shape[1], E, _p(pairs.tile_expert),
         _p(status_word(x.device)), _stream()), f"{what} tiles<={pairs.max_tiles}x128 N={N} K={K}",
         flops=2 * pairs.n_tokens * pairs.top * N * K, nbytes=w.numel() * 2)
     return out
+
+
+def moe_up_tc(x_sorted: torch.Tensor, w_up: torch.Tensor, pairs: SortedPairs) -> torch.Tensor:
+    """`moe_up` on tcgen05 for tiles of 128 rows: `x_sorted` [rows, d] from `moe_gather`, `w_up` [E, F, d]; the squared
+    ReLU in the product's epilogue; [rows, F] bfloat16."""
+    _dev(x_sorted, "x_sorted"), _dev(w_up, "w_up")
+    out = torch.empty((pairs.rows, w_up.shape[1]), dtype=torch.bfloat16, device=x_sorted.device)
+    return _grouped(x_sorted, w_up, out, 0, pairs, "moe_up_tc", store_act="relu2")
 
 
 def moe_gate_up_tc(x_sorted: torch.Tensor, w_gate_up: torch.Tensor, pairs: SortedPairs) -> torch.Tensor:

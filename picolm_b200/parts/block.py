@@ -210,7 +210,8 @@ class ParallelNormBlock(Arrangement):
     """Mixer and feed-forward side by side, each behind a norm of its own of the same x:
     `x += scale * (mixer(filter(norm_a(x))) + feed_forward(norm_b(x)))`.  The feed-forward with its norm and the
     filter (family "row_filter": something done to the mixer's input alone) are optional; `scale` is the layer's
-    `params["residual_scale"]` (default 1).
+    `params["residual_scale"]` (default 1).  A feed-forward without a norm of its own reads what the mixer's norm makes:
+    `h = norm(x); x += scale * (mixer(filter(h)) + feed_forward(h))`.
 
     Both norms are RMS norms here, so that one pass over a row serves both (and a `token_shift` filter with them:
     `ops.norm_pair_shift`); other norms run one after the other.  A feed-forward that can (`adds_to_stream`) puts
@@ -234,7 +235,7 @@ class ParallelNormBlock(Arrangement):
 
     def _fused_norms(self) -> bool:
         from .norm import RMSNorm
-        norms = [self.mixer_norm] + ([self.feed_forward_norm] if "feed_forward" in self.named else [])
+        norms = [self.mixer_norm] + ([self.feed_forward_norm] if "feed_forward_norm" in self.named else [])
         filt = self.named.get("mixer_filter")
         return (all(isinstance(n, RMSNorm) and n.weight.dtype == torch.float32 for n in norms)
                 and len({float(n.params["eps"]) for n in norms}) == 1 and (filt is None or isinstance(filt, TokenShift)))
@@ -247,7 +248,12 @@ class ParallelNormBlock(Arrangement):
         if keep_rows is not None and keep_rows.numel() == 0:
             has_ff = False                                            # nothing reads what this layer adds to the stream
         h_ff = None
-        if self._fused_norms():
+        shared = has_ff and "feed_forward_norm" not in self.named     # one norm's rows for both
+        if shared or not has_ff and filt is None:
+            h = h_ff = self.mixer_norm.forward(stream)                # (adds what the layer before left in its own pass)
+            if filt is not None:
+                h = filt.forward(h, step, filt_cache)
+        elif self._fused_norms():
             settle(stream, None)                                      # x += what the layer before left
             h, h_ff = ops.norm_pair_shift(
                 stream.x, self.mixer_norm.weight, float(self.mixer_norm.params["eps"]), dt,
@@ -268,12 +274,17 @@ class ParallelNormBlock(Arrangement):
             stream.pending = delta
             stream.narrow(keep_rows)
             delta, stream.pending = stream.pending, None
-            if has_ff:
+            if shared:
+                h_ff = ops.gather_rows(h_ff, keep_rows)
+            elif has_ff:
                 h_ff = self.feed_forward_norm.forward(stream)
+        if not has_ff and self.scale == 1.0:
+            stream.pending = delta                                    # a product that has not run: left to the next norm
+            return
         if hasattr(delta, "compute"):
             delta = delta.compute()
         if not has_ff:
-            stream.pending = delta if self.scale == 1.0 else ops.scaled_sum(delta, self.scale, delta, 0.0)
+            stream.pending = ops.scaled_sum(delta, self.scale, delta, 0.0)
             return
         if getattr(self.feed_forward, "adds_to_stream", False):
             self.feed_forward.forward(h_ff, step, add=delta, out_scale=self.scale, into=stream.x)
@@ -287,12 +298,15 @@ class ParallelNormBlock(Arrangement):
 def parallel_norm_layer(prefix: str, mixer: PartSpec, mixer_norm: PartSpec, feed_forward: PartSpec = None,
                         feed_forward_norm: PartSpec = None, mixer_filter: PartSpec = None, residual_scale: float = 1.0,
                         cache_of=None) -> LayerSpec:
-    """The spec of a `parallel_norm` layer; without `feed_forward` the layer only mixes.  `mixer_filter`: a part of
+    """The spec of a `parallel_norm` layer; without `feed_forward` the layer only mixes, without `feed_forward_norm` the
+    feed-forward reads the mixer's norm.  `mixer_filter`: a part of
     the "row_filter" family between the mixer's norm and the mixer."""
     parts = {"mixer_norm": ("norm", mixer_norm)}
     if mixer_filter is not None:
         parts["mixer_filter"] = ("row_filter", mixer_filter)          # (in front of the mixer: the order of the layer's caches)
     parts["mixer"] = ("mixer", mixer)
     if feed_forward is not None:
-        parts.update({"feed_forward_norm": ("norm", feed_forward_norm), "feed_forward": ("feed_forward", feed_forward)})
+        if feed_forward_norm is not None:
+            parts["feed_forward_norm"] = ("norm", feed_forward_norm)
+        parts["feed_forward"] = ("feed_forward", feed_forward)
     return LayerSpec(prefix, "parallel_norm", parts, cache_of=cache_of, params={"residual_scale": float(residual_scale)})

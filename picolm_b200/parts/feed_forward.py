@@ -69,7 +69,7 @@ class GatedMLP(Part):
 @register_part("feed_forward", "mlp")
 class PlainMLP(Part):
     """Two maps with an activation between them, `W_down act(W_up h)`, no gate and no biases.  params: hidden_size,
-    intermediate_size, activation ("gelu_erf": 0.5 z (1 + erf(z / sqrt 2))), up_name/down_name (relative tensor names)."""
+    intermediate_size, activation ("gelu_erf": 0.5 z (1 + erf(z / sqrt 2)), "relu2": relu(z)^2), up_name/down_name (relative tensor names)."""
 
     def __init__(self, params, runtime):
         super().__init__(params, runtime)
@@ -110,7 +110,8 @@ class RoutedMLP(Part):
     {"size", "prefix", "gate"}: the shared expert's inner width, its tensors' prefix, and the name under that prefix of
     the [1, hidden] row whose sigmoid multiplies the shared expert's result per token; None: no such gate).
 
-    Optional: scores ("sigmoid", or "softmax": over all router outputs, or "logits": the choice goes by the logits plus the
+    Optional: activation ("silu", the gated default; "relu2": experts without a gate, `W_down relu(W_up h)^2`, and no
+    gate_name), scores ("sigmoid", or "softmax": over all router outputs, or "logits": the choice goes by the logits plus the
     tensor `correction_name`, a bias of the router, and the weights are the softmax over the chosen ones), group_score ("top2", or "max": a group's
     score is its best choice score), normalize (False: the weights are the chosen scores as they are, times
     `route_scale`), identity (a number: the router has that many outputs more, behind the experts', for experts
@@ -146,8 +147,13 @@ class RoutedMLP(Part):
                              f"kept={self.keep} do not fit together")
         if self.top > self.keep * (self.n_out // self.n_groups):
             raise ValueError(f"routed_mlp: {self.keep} groups of {self.n_out // self.n_groups} experts cannot give {self.top} choices")
+        if p.get("activation", "silu") not in ("silu", "relu2"):
+            raise ValueError(f"routed_mlp: experts with the activation {p['activation']!r} have no kernel; known: silu (gated), relu2")
+        self.gated = p.get("activation", "silu") == "silu"
         self.shared = None
         sh = p.get("shared")
+        if sh and not self.gated:
+            raise ValueError("routed_mlp: a shared expert is a gated one")
         if sh:
             self.shared = GatedMLP({"hidden_size": self.d, "intermediate_size": int(sh["size"]), "activation": "silu",
                                     "gate_name": p["gate_name"], "up_name": p["up_name"], "down_name": p["down_name"]}, runtime)
@@ -161,7 +167,8 @@ class RoutedMLP(Part):
         if p.get("correction_name"):
             specs[p["correction_name"]] = WeightSpec((self.n_out,), init="normal")
         for e in range(self.E):
-            specs[self._expert(e, "gate_name")] = WeightSpec((self.F, self.d))
+            if self.gated:
+                specs[self._expert(e, "gate_name")] = WeightSpec((self.F, self.d))
             specs[self._expert(e, "up_name")] = WeightSpec((self.F, self.d))
             specs[self._expert(e, "down_name")] = WeightSpec((self.d, self.F))
         if self.shared is not None:
@@ -187,9 +194,14 @@ class RoutedMLP(Part):
         self.correction = (tensors[p["correction_name"]].to(torch.float32).contiguous() if p.get("correction_name") else None)
         # [E, 2F, d]: an expert's gate rows, then its up rows (in turns of 64 where the inner width allows it: the
         # layout of the tensor-core product with the activation in its epilogue, which every kernel here reads); [E, d, F]
+        if not self.gated:
+            self.interleaved = False
+            self.w_in = torch.stack([tensors[self._expert(e, "up_name")] for e in range(self.E)]).contiguous()          # [E, F, d]
+            self.w_down = torch.stack([tensors[self._expert(e, "down_name")] for e in range(self.E)]).contiguous()
+            return
         gates, ups = [tensors[self._expert(e, "gate_name")] for e in range(self.E)], [tensors[self._expert(e, "up_name")] for e in range(self.E)]
         self.interleaved = self.F % 64 == 0
-        self.w_gate_up = torch.stack([ops.interleave_gate_up(g, u) if self.interleaved else torch.cat([g, u])
+        self.w_in = torch.stack([ops.interleave_gate_up(g, u) if self.interleaved else torch.cat([g, u])
                                       for g, u in zip(gates, ups)]).contiguous()
         self.w_down = torch.stack([tensors[self._expert(e, "down_name")] for e in range(self.E)]).contiguous()
 
@@ -200,7 +212,7 @@ class RoutedMLP(Part):
     def weight_bytes_for(self, tokens: int) -> int:
         """What a decode step of `tokens` tokens reads at most: each token's `top` experts, all different until all
         experts are in use."""
-        per = (self.w_gate_up.numel() + self.w_down.numel()) // self.E * self.w_down.element_size()
+        per = (self.w_in.numel() + self.w_down.numel()) // self.E * self.w_down.element_size()
         return (self.w_router.numel() * self.w_router.element_size() + min(self.E, tokens * self.top) * per
                 + (self.shared.weight_bytes() if self.shared is not None else 0))
 
@@ -213,17 +225,19 @@ class RoutedMLP(Part):
                                             float(self.params["route_scale"]), self.gate_col, scores=self.scores,
                                             group_score=self.group_score, normalize=self.normalize)
         skip = self.identity
-        if self.interleaved and T * self.top >= 64 * self.E and ops.moe_tc_supported(h, self.w_gate_up, self.w_down):
+        if (self.interleaved or not self.gated) and T * self.top >= 64 * self.E and ops.moe_tc_supported(h, self.w_in, self.w_down):
             # many pairs an expert (prompts): tiles of 128 rows on tcgen05, the tokens' rows laid out in sorted order first
             pairs = ops.moe_align(ids, self.E, 128, skip)
-            act = ops.moe_gate_up_tc(ops.moe_gather(h, pairs), self.w_gate_up, pairs)
+            rows = ops.moe_gather(h, pairs)
+            act = ops.moe_gate_up_tc(rows, self.w_in, pairs) if self.gated else ops.moe_up_tc(rows, self.w_in, pairs)
             y = ops.moe_down_tc(act, self.w_down, pairs)
         else:
             # few pairs an expert (decode steps): small tiles, so that a tile's padding costs little; bfloat16 on
             # mma.sync, float32 on the CUDA cores (which take tiles of 64 rows where experts have many)
             bm = 16 if (h.dtype == torch.bfloat16 or T * self.top <= 16 * self.E) else 64
             pairs = ops.moe_align(ids, self.E, bm, skip)
-            act = ops.moe_gate_up(h, self.w_gate_up, pairs, interleaved=self.interleaved)
+            act = (ops.moe_gate_up(h, self.w_in, pairs, interleaved=self.interleaved) if self.gated
+                   else ops.moe_up(h, self.w_in, pairs))
             y = ops.moe_down(act, self.w_down, pairs)
         shared = None
         if self.shared is not None:

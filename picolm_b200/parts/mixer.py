@@ -45,7 +45,9 @@ class Attention(Part):
       qk_norm       {"eps", "q_name", "k_name"}: queries and keys are divided by their root mean square over ALL heads
                     at once and multiplied by those weights ([H * head_dim], [G * head_dim]), after the bias and
                     before the rotation; with "per_head": True the root mean square is each head's own and the
-                    weights are [head_dim], shared by the heads
+                    weights are [head_dim], shared by the heads.  With "weights": False there are none (and no names).
+                    (The root mean square is the same before and after the rotation, so without weights, or with
+                    weights equal on rotated pairs, the norm may as well stand behind it.)
       values_from_keys  True: there is no value projection; the keys as projected (bias added, before norm and
                     rotation) serve as values
       sink_name     a tensor [num_heads]: the softmax's denominator of head h also holds exp(sink[h]), a term with no
@@ -98,6 +100,7 @@ class Attention(Part):
         self.vd = int(p.get("value_dim") or self.hd)
         self.bias = bool(p.get("bias", False))
         self.qk_norm = p.get("qk_norm")
+        self.norm_weights = bool(self.qk_norm and self.qk_norm.get("weights", True))
         self.per_head_norm = bool(self.qk_norm and self.qk_norm.get("per_head", False))
         self.own_kv = bool(p.get("own_kv", True))
         self.v_from_k = bool(p.get("values_from_keys", False))
@@ -154,7 +157,7 @@ class Attention(Part):
             sfx = p.get("bias_suffix", ".b")
             for name in self._names() + [p["o_name"]]:
                 specs[name + sfx] = WeightSpec((specs[name].shape[0],), init="normal")
-        if self.qk_norm is not None:
+        if self.norm_weights:
             specs[self.qk_norm["q_name"]] = WeightSpec((hd if self.per_head_norm else H * hd,), init="ones_normal")
             if self.own_kv:
                 specs[self.qk_norm["k_name"]] = WeightSpec((hd if self.per_head_norm else G * hd,), init="ones_normal")
@@ -193,7 +196,12 @@ class Attention(Part):
             sfx = p.get("bias_suffix", ".b")
             self.b_qkv = torch.cat([tensors[n + sfx].to(torch.float32) for n in self._names()]).contiguous()
             self.b_o = tensors[p["o_name"] + sfx].to(torch.float32).contiguous()
-        if self.qk_norm is not None:
+        if self.qk_norm is not None and not self.norm_weights:
+            n_q, n_k = (self.hd, self.hd) if self.per_head_norm else (self.H * self.hd, self.G * self.hd)
+            self.w_qn = torch.ones(n_q, dtype=self.runtime.dtype, device=self.w_o.device)
+            if self.own_kv:
+                self.w_kn = torch.ones(n_k, dtype=self.runtime.dtype, device=self.w_o.device)
+        elif self.qk_norm is not None:
             self.w_qn = tensors[self.qk_norm["q_name"]].to(self.runtime.dtype).contiguous()
             if self.own_kv:
                 self.w_kn = tensors[self.qk_norm["k_name"]].to(self.runtime.dtype).contiguous()

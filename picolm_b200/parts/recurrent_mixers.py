@@ -12,7 +12,7 @@ import torch
 
 from .. import ops
 from ..cache.spec import CacheSpec
-from .base import Part, WeightSpec, register_part
+from .base import Part, WeightSpec, build_part, register_part
 from .mixer import _stack_rows
 
 
@@ -205,6 +205,62 @@ class LightningAttention(_StateMixer):
         return ops.linear(gated, self.w_o, torch.float32, defer=True)
 
 
+@register_part("mixer", "retention")
+class Retention(_StateMixer):
+    """Linear attention with one constant decay a head over rotated queries and keys.  params: hidden_size, heads, dim
+    (key size of a head), vdim, decay (a number per head), eps, position (a PartSpec of the position family: a rotation
+    that pairs halves, or none), k_scale (a factor on the keys behind the rotation; default dim^(-1/2)).
+    `q = R_t W_q h`, `k = k_scale R_t W_k h`, `v = W_v h`; per head `S_t = decay_h S_(t-1) + k_t v_t^T`,
+    `o_t = S_t^T q_t`; each head's o is divided by its root mean square over vdim (no weight), the heads are
+    concatenated, multiplied by `silu(W_g h)` and projected.
+
+    Tensors: q, k [heads dim, hidden], v, g [heads vdim, hidden], o [hidden, heads vdim]."""
+
+    def __init__(self, params, runtime):
+        super().__init__(params, runtime)
+        p = self.params
+        self.d, self.H, self.N, self.P, self.eps = p["hidden_size"], p["heads"], p["dim"], p["vdim"], float(p["eps"])
+        self.k_scale = float(p["k_scale"]) if p.get("k_scale") is not None else self.N ** -0.5
+        if len(p["decay"]) != self.H:
+            raise ValueError(f"retention: {len(p['decay'])} decays for {self.H} heads")
+        pos = p.get("position")
+        self.position = build_part("position", pos, runtime) if pos is not None and pos.kind != "none" else None
+        if self.position is not None and (not hasattr(self.position, "rotation") or self.position.params.get("pairing") != "half"):
+            raise ValueError("retention: the position encoding must be a rotation that pairs halves, or none")
+
+    def weight_specs(self):
+        HN, HP, d = self.H * self.N, self.H * self.P, self.d
+        return {"q": WeightSpec((HN, d)), "k": WeightSpec((HN, d)), "v": WeightSpec((HP, d)), "g": WeightSpec((HP, d)),
+                "o": WeightSpec((d, HP))}
+
+    def load(self, tensors):
+        self.w_h = _stack_rows([tensors[n] for n in ("q", "k", "v", "g")])       # one product for everything that reads h
+        self.w_o = tensors["o"]
+        decay = [float(x) for x in self.params["decay"]]
+        self.decay = torch.tensor(decay, dtype=torch.float32, device=self.w_o.device)
+        self.powers = ops.decay_powers(decay).to(self.w_o.device)
+
+    def weight_bytes(self):
+        return sum(t.numel() * t.element_size() for t in (self.w_h, self.w_o))
+
+    def cache_spec(self):
+        return CacheSpec.state((self.H * self.N * self.P,))
+
+    def prepare(self, max_seq_tokens: int) -> None:
+        if self.position is not None:
+            self.position.prepare(max_seq_tokens)
+
+    def forward(self, h, step, cache):
+        dt = self.runtime.dtype
+        HN, HP = self.H * self.N, self.H * self.P
+        proj = ops.linear(h, self.w_h, dt)
+        q, k, v, g = proj[:, :HN], proj[:, HN:2 * HN], proj[:, 2 * HN:2 * HN + HP], proj[:, 2 * HN + HP:]
+        o = ops.decay_scan(q, k, v, self.decay, self.powers, cache.state, step, self.H, self.N, self.P,
+                           rotation=self.position.rotation() if self.position is not None else None, k_scale=self.k_scale)
+        gated = ops.gated_norm(o, dt, eps=self.eps, group=self.P, gate=g, gate_mode=ops.GATE_AFTER_NORM, activation="silu")
+        return ops.linear(gated, self.w_o, torch.float32, defer=True)
+
+
 @register_part("mixer", "rglru")
 class GatedDiagonalRecurrence(_StateMixer):
     """A recurrent block around a real-gated diagonal linear recurrence.  params: hidden_size, width (channels of the
@@ -269,18 +325,21 @@ class GatedDiagonalRecurrence(_StateMixer):
 
 @register_part("mixer", "gated_delta")
 class GatedDeltaRule(_StateMixer):
-    """The delta rule with a decay per key channel.  params: hidden_size, heads, kv_heads (query/key heads; head h
-    uses q/k head h // (heads / kv_heads)), dim (key size), vdim, conv (taps), rank (None: as the checkpoint's a1 and
-    g1 have it), eps (of the read-out's norm), l2_eps (inside the root of the unit norm, default 1e-6).
+    """The delta rule with a decay.  params: hidden_size, heads, kv_heads (query/key heads; head h uses q/k head
+    h // (heads / kv_heads)), dim (key size), vdim, conv (taps), eps (of the read-out's norm), l2_eps (inside the root of
+    the unit norm, default 1e-6), decay ("channel", the default: one per head and key channel, through a bottleneck; or
+    "head": one a head, straight from h), gate ("bottleneck", the default, or "full": one matrix), gate_activation
+    ("sigmoid", the default, or "silu"), rank (of the bottlenecks; None: as the checkpoint's a1 and g1 have it).
     q, k, v each pass a depthwise causal convolution (no bias) and SiLU; q and k are made unit vectors per head and q
-    is multiplied by dim^(-1/2); `beta = sigmoid(W_b h)` per head; the decay per head and key channel is
-    `exp(-exp(A_log_h) softplus(W_a2 (W_a1 h) + dt_bias))`.  Per head, S [dim, vdim] from zero:
+    is multiplied by dim^(-1/2); `beta = sigmoid(W_b h)` per head; the decay is `exp(-exp(A_log_h) softplus(z + dt_bias))`
+    with `z = W_a2 (W_a1 h)` per head and key channel, or `z = W_a h` per head.  Per head, S [dim, vdim] from zero:
     `S <- diag(decay) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q`.  Each head's o is divided by its root
-    mean square over vdim, times `norm` [vdim] (shared), times `sigmoid(W_g2 (W_g1 h))`, then projected.
+    mean square over vdim, times `norm` [vdim] (shared), times `act(W_g2 (W_g1 h))` or `act(W_g h)`, then projected.
 
     Tensors: q, k [kv_heads dim, hidden], v [heads vdim, hidden], q.conv, k.conv, v.conv [channels, taps], b [heads,
-    hidden], A_log [heads], a1 [rank, hidden], a2 [heads dim, rank], dt_bias [heads dim], g1 [rank', hidden], g2
-    [heads vdim, rank'], norm [vdim], o [hidden, heads vdim]."""
+    hidden], A_log [heads], norm [vdim], o [hidden, heads vdim]; a decay per channel: a1 [rank, hidden], a2 [heads dim,
+    rank], dt_bias [heads dim], per head: a [heads, hidden], dt_bias [heads]; a gate through a bottleneck: g1 [rank',
+    hidden], g2 [heads vdim, rank'], in full: g [heads vdim, hidden]."""
 
     def __init__(self, params, runtime):
         super().__init__(params, runtime)
@@ -288,6 +347,9 @@ class GatedDeltaRule(_StateMixer):
         self.d, self.H, self.G, self.N, self.P = p["hidden_size"], p["heads"], p["kv_heads"], p["dim"], p["vdim"]
         self.taps, self.rank, self.eps = p["conv"], p.get("rank"), float(p["eps"])
         self.l2_eps = float(p.get("l2_eps", 1e-6))
+        self.head_decay = {"channel": False, "head": True}[p.get("decay", "channel")]
+        self.full_gate = {"bottleneck": False, "full": True}[p.get("gate", "bottleneck")]
+        self.gate_activation = p.get("gate_activation", "sigmoid")
         if self.H % self.G:
             raise ValueError("gated_delta: heads must be a multiple of kv_heads")
         self.conv_channels = 2 * self.G * self.N + self.H * self.P
@@ -295,33 +357,54 @@ class GatedDeltaRule(_StateMixer):
         self.n_conv = (self.taps - 1) * self.conv_channels
 
     def weight_specs(self):
-        GN, HN, HP, d, r = self.G * self.N, self.H * self.N, self.H * self.P, self.d, self.rank or -1
+        H, GN, HN, HP, d, r = self.H, self.G * self.N, self.H * self.N, self.H * self.P, self.d, self.rank or -1
         conv = dict(init="normal_scaled", scale=0.4)
-        return {
+        specs = {
             "q": WeightSpec((GN, d)), "k": WeightSpec((GN, d)), "v": WeightSpec((HP, d)),
             "q.conv": WeightSpec((GN, self.taps), **conv), "k.conv": WeightSpec((GN, self.taps), **conv),
             "v.conv": WeightSpec((HP, self.taps), **conv),
-            "b": WeightSpec((self.H, d)), "A_log": WeightSpec((self.H,), init="uniform", lo=-2.0, hi=0.5),
-            "a1": WeightSpec((r, d)), "a2": WeightSpec((HN, r), init="normal_scaled", scale=0.5),
-            "dt_bias": WeightSpec((HN,), init="uniform", lo=-3.0, hi=0.0),
-            "g1": WeightSpec((r, d)), "g2": WeightSpec((HP, r), init="normal_scaled", scale=0.5),
+            "b": WeightSpec((H, d)), "A_log": WeightSpec((H,), init="uniform", lo=-2.0, hi=0.5),
+            "dt_bias": WeightSpec((H if self.head_decay else HN,), init="uniform", lo=-3.0, hi=0.0),
             "norm": WeightSpec((self.P,), init="ones_normal"),
             "o": WeightSpec((d, HP)),
         }
+        if self.head_decay:
+            specs["a"] = WeightSpec((H, d))
+        else:
+            specs.update({"a1": WeightSpec((r, d)), "a2": WeightSpec((HN, r), init="normal_scaled", scale=0.5)})
+        if self.full_gate:
+            specs["g"] = WeightSpec((HP, d))
+        else:
+            specs.update({"g1": WeightSpec((r, d)), "g2": WeightSpec((HP, r), init="normal_scaled", scale=0.5)})
+        return specs
 
     def load(self, tensors):
-        # one projection for everything that reads h: rows [q | k | v | b | a1 | g1]
-        self.w_h = _stack_rows([tensors[n] for n in ("q", "k", "v", "b", "a1", "g1")])
-        self.r_a, self.r_g = tensors["a1"].shape[0], tensors["g1"].shape[0]
-        self.w_a2, self.w_g2, self.w_o = tensors["a2"], tensors["g2"], tensors["o"]
-        if self.w_a2.shape[1] != self.r_a or self.w_g2.shape[1] != self.r_g:
-            raise ValueError("gated_delta: a2 / g2 do not take as many columns as a1 / g1 have rows")
+        # one projection for everything that reads h: rows [q | k | v | g (in full) | b | a or a1 | g1]
+        names = ["q", "k", "v"] + ["g"] * self.full_gate + ["b", "a" if self.head_decay else "a1"] + ["g1"] * (not self.full_gate)
+        rows = [tensors[n] for n in names]
+        if self.full_gate:
+            # rows of zeros up to a multiple of eight columns: the product's rows then start on 16-byte boundaries
+            spare = -sum(t.shape[0] for t in rows) % 8
+            if spare:
+                rows.append(torch.zeros((spare, self.d), dtype=rows[0].dtype, device=rows[0].device))
+        self.w_h = _stack_rows(rows)
+        self.w_o = tensors["o"]
+        self.w_a2 = self.w_g2 = None
+        self.r_a = self.H if self.head_decay else tensors["a1"].shape[0]
+        if not self.head_decay:
+            self.w_a2 = tensors["a2"]
+            if self.w_a2.shape[1] != self.r_a:
+                raise ValueError("gated_delta: a2 does not take as many columns as a1 has rows")
+        if not self.full_gate:
+            self.w_g2 = tensors["g2"]
+            if self.w_g2.shape[1] != tensors["g1"].shape[0]:
+                raise ValueError("gated_delta: g2 does not take as many columns as g1 has rows")
         self.conv_w = self._f32(torch.cat([tensors[n].to(torch.float32) for n in ("q.conv", "k.conv", "v.conv")]).t())
         self.a_log, self.dt_bias = self._f32(tensors["A_log"]), self._f32(tensors["dt_bias"])
         self.norm_w = self._f32(tensors["norm"])
 
     def weight_bytes(self):
-        return sum(t.numel() * t.element_size() for t in (self.w_h, self.w_a2, self.w_g2, self.w_o))
+        return sum(t.numel() * t.element_size() for t in (self.w_h, self.w_a2, self.w_g2, self.w_o) if t is not None)
 
     def cache_spec(self):
         # one row per sequence: S as [heads, dim, vdim], then the convolution's last inputs
@@ -336,14 +419,19 @@ class GatedDeltaRule(_StateMixer):
         GN, HP, H, C = self.G * self.N, self.H * self.P, self.H, self.conv_channels
         proj = ops.linear(h, self.w_h, dt)
         qkv = ops.causal_conv(proj[:, :C], self.conv_w, None, cache.state[:, self.n_state:], step)
-        b_raw = proj[:, C:C + H]
-        a1, g1 = proj[:, C + H:C + H + self.r_a], proj[:, C + H + self.r_a:]
-        z = self._narrow_product(a1, self.w_a2, dt)
-        gate = self._narrow_product(g1, self.w_g2, dt)
+        at = C
+        if self.full_gate:
+            gate, at = proj[:, C:C + HP], C + HP
+        b_raw, z, rest = proj[:, at:at + H], proj[:, at + H:at + H + self.r_a], proj[:, at + H + self.r_a:]
+        if not self.head_decay:
+            z = self._narrow_product(z, self.w_a2, dt)
+        if not self.full_gate:
+            gate = self._narrow_product(rest, self.w_g2, dt)
         qn, kn, qk, decay, beta = ops.delta_prep(qkv[:, :GN], qkv[:, GN:2 * GN], z, b_raw, self.a_log, self.dt_bias,
-                                                 self.l2_eps, self.N ** -0.5, H, self.N, heads_per_group=H // self.G)
+                                                 self.l2_eps, self.N ** -0.5, H, self.N, heads_per_group=H // self.G,
+                                                 head_decay=self.head_decay)
         o = ops.delta_scan(qn, kn, qk, decay, beta, qkv[:, 2 * GN:], cache.state[:, :self.n_state], step, H, self.N,
-                           self.P, heads_per_group=H // self.G)
+                           self.P, heads_per_group=H // self.G, head_decay=self.head_decay)
         gated = ops.gated_norm(o, dt, weight=self.norm_w, eps=self.eps, group=self.P, weight_per_group=True, gate=gate,
-                               gate_mode=ops.GATE_AFTER_NORM, activation="sigmoid")
+                               gate_mode=ops.GATE_AFTER_NORM, activation=self.gate_activation)
         return ops.linear(gated, self.w_o, torch.float32, defer=True)
