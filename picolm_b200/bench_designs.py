@@ -1,9 +1,10 @@
-"""Throughput of another design (Potuzen, Kunulorn, Tebasun, Fupapel, Dobepel) beside the Llama decoder (Tebasun: beside Potuzen, the
+"""Throughput of another design (Potuzen, Kunulorn, Tebasun, Fupapel, Dobepel, Laperax) beside the Llama decoder (Tebasun: beside Potuzen, the
 other design whose layers are recurrences and attention in turn; Fupapel: beside Kunulorn, the other design of chunked
-attention and routed feed-forwards; Dobepel: beside Tebasun, the other design of attention and a recurrence side by side) at equal layer sizes (random weights): prefill
+attention and routed feed-forwards; Dobepel: beside Tebasun, the other design of attention and a recurrence side by side;
+Laperax: beside Dobepel, the other design with a constant-decay recurrence and routed feed-forwards) at equal layer sizes (random weights): prefill
 tokens/s of one prompt and decode tokens/s of a batch, at a few sizes that resemble a real model's layers,
 and, with `kernels=True`, the device time of every kind of launch with the fraction of the memory's or the
-tensor cores' measured rate that it reaches.  `bench.py --design potuzen|kunulorn|tebasun|fupapel|dobepel` calls this."""
+tensor cores' measured rate that it reaches.  `bench.py --design potuzen|kunulorn|tebasun|fupapel|dobepel|laperax` calls this."""
 from __future__ import annotations
 
 import json
@@ -12,6 +13,8 @@ import statistics
 import sys
 import tempfile
 import time
+
+DESIGNS = ("potuzen", "kunulorn", "tebasun", "fupapel", "dobepel", "laperax")
 
 # name -> (width, feed-forward, layers, vocabulary, the Llama twin's (heads, kv heads, head size))
 SIZES = {
@@ -119,6 +122,23 @@ def dobepel_config(width: int, ff: int, layers: int, vocab: int) -> dict:
                        for i in range(layers)]}
 
 
+def laperax_config(width: int, ff: int, layers: int, vocab: int) -> dict:
+    """Layers in turn: two of retention (Dobepel's recurrent heads: width / 256 of 128 x 256, every component rotated),
+    attention (Dobepel's: width / 128 heads of 128 over a quarter as many key heads, half of each head rotated, a window of
+    4,096 positions) and a delta rule (Tebasun's: width / 256 heads of 128 x 128); every layer routes to 4 of 32 experts
+    (16 at the larger size), each two maps of 3/8 of the dense width, so that a token's arithmetic equals a gated dense layer's."""
+    H = width // 256
+    mlp = {"kind": "moe", "expert": {"ff": 3 * ff // 8}, "router": {"experts": 32 if width <= 2048 else 16, "top": 4, "scale": 2.0}}
+    ret = {"type": "retention", "mixer": {"heads": H, "dim": 128, "vdim": 256, "rot": {"base": 500000.0, "dims": 128},
+                                          "decay": [1.0 - 2.0 ** (-5.0 - 6.0 * h / max(1, H - 1)) for h in range(H)]}}
+    att = {"type": "attention", "mixer": {"heads": width // 128, "kv_heads": width // 512, "dim": 128, "vdim": 128, "scale": 0.12,
+                                          "rot": {"base": 500000.0, "dims": 64}, "mask": {"size": 4096}}}
+    delta = {"type": "delta", "mixer": {"heads": H, "kv_heads": width // 512, "dim": 128, "vdim": 128, "conv": 4}}
+    turn = [ret, ret, att, delta]
+    return {"architecture": "Laperax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_scale": 0.5, "logit_softcap": 30.0,
+            "layers": [dict(turn[i % 4], mlp=mlp) for i in range(layers)]}
+
+
 def llama_config(width: int, ff: int, layers: int, vocab: int, heads) -> dict:
     H, G, hd = heads
     return {"architectures": ["LlamaForCausalLM"], "model_type": "llama", "num_hidden_layers": layers, "hidden_size": width,
@@ -206,10 +226,10 @@ def _table(rows, top=20):
 
 
 def run(design: str, sizes, prompt_tokens: int, batch: int, steps: int, warmup: int, kernels: bool) -> dict:
-    if design not in ("potuzen", "kunulorn", "tebasun", "fupapel", "dobepel"):
-        raise ValueError(f"no design {design!r} to compare (known: potuzen, kunulorn, tebasun, fupapel, dobepel)")
-    beside = {"tebasun": "potuzen", "fupapel": "kunulorn", "dobepel": "tebasun"}.get(design, "llama")
-    result = {"design": design, "beside": {"potuzen": "Potuzen", "kunulorn": "Kunulorn", "tebasun": "Tebasun"}.get(beside, "LlamaForCausalLM"), "dtype": "bf16",
+    if design not in DESIGNS:
+        raise ValueError(f"no design {design!r} to compare (known: {', '.join(DESIGNS)})")
+    beside = {"tebasun": "potuzen", "fupapel": "kunulorn", "dobepel": "tebasun", "laperax": "dobepel"}.get(design, "llama")
+    result = {"design": design, "beside": {"potuzen": "Potuzen", "kunulorn": "Kunulorn", "tebasun": "Tebasun", "dobepel": "Dobepel"}.get(beside, "LlamaForCausalLM"), "dtype": "bf16",
               "data": "synthetic (random weights and tokens)",
               "prompt_tokens": prompt_tokens, "decode_batch": batch, "steps": steps, "warmup": warmup, "sizes": {}}
     for name in sizes:
@@ -219,11 +239,13 @@ def run(design: str, sizes, prompt_tokens: int, batch: int, steps: int, warmup: 
                   "kunulorn": lambda: kunulorn_config(width, ff, layers, vocab, heads),
                   "tebasun": lambda: tebasun_config(width, ff, layers, vocab),
                   "fupapel": lambda: fupapel_config(width, ff, layers, vocab, heads),
-                  "dobepel": lambda: dobepel_config(width, ff, layers, vocab)}[design]()
+                  "dobepel": lambda: dobepel_config(width, ff, layers, vocab),
+                  "laperax": lambda: laperax_config(width, ff, layers, vocab)}[design]()
         ours = _measure(config, prompt_tokens, batch, steps, warmup, kernels)
         twin_config = {"potuzen": lambda: potuzen_config(width, ff, layers, vocab),
                        "kunulorn": lambda: kunulorn_config(width, ff, layers, vocab, heads),
                        "tebasun": lambda: tebasun_config(width, ff, layers, vocab),
+                       "dobepel": lambda: dobepel_config(width, ff, layers, vocab),
                        "llama": lambda: llama_config(width, ff, layers, vocab, heads)}[beside]()
         twin = _measure(twin_config, prompt_tokens, batch, steps, warmup, kernels)
         result["sizes"][name] = {
