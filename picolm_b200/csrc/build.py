@@ -44,8 +44,9 @@ LIBRARIES: Dict[str, List[str]] = {
     "recurrent": ["recurrent.cu"],
     "routed": ["routed.cu"],
     "decay_chunk": ["decay_chunk.cu"],
+    "delta_chunk": ["delta_chunk.cu"],
 }
-HEADERS = ["common.cuh", "tc_common.cuh", "gemm_tc_static.h"]
+HEADERS = ["common.cuh", "tc_common.cuh", "mma_common.cuh", "gemm_tc_static.h"]
 
 # Libraries that are specialised at compile time.  At run time only the variant a
 # model needs is built (`attention_variant`); the build check builds these.

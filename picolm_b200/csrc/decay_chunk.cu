@@ -23,7 +23,7 @@
 // (FINAL; WHOLE where there is one segment).
 //
 // Steps of single tokens take decay_step_kernel, which streams the state through once.
-#include "common.cuh"
+#include "mma_common.cuh"
 
 namespace {
 
@@ -49,32 +49,7 @@ struct Args {
     float* seg_state;                                  // [seq][segment][H][N][P]
 };
 
-__device__ __forceinline__ uint32_t smem_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
-__device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm_x4_t(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t bits(__nv_bfloat162 h) { return *reinterpret_cast<uint32_t*>(&h); }
-// two floats as bf16 pairs hi + lo
-__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-    hi = bits(h);
-    lo = bits(__floats2bfloat162_rn(a - __low2float(h), b - __high2float(h)));
-}
 __device__ __forceinline__ float silu_f(float x) { return __fdividef(x, 1.f + __expf(-x)); }      // (rounded to bf16 right away)
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool full) {        // 16 bytes, or zeros
-    const int n = full ? 16 : 0;
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
-}
 
 // eight activations of a row: SiLU where asked for, rounded to bf16
 __device__ __forceinline__ uint4 act8(uint4 raw, bool silu) {
@@ -83,7 +58,7 @@ __device__ __forceinline__ uint4 act8(uint4 raw, bool silu) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const __nv_bfloat162 h = *reinterpret_cast<const __nv_bfloat162*>(w + i);
-        w[i] = bits(__floats2bfloat162_rn(silu_f(__low2float(h)), silu_f(__high2float(h))));
+        w[i] = bf16_bits(__floats2bfloat162_rn(silu_f(__low2float(h)), silu_f(__high2float(h))));
     }
     return raw;
 }
@@ -91,11 +66,6 @@ __device__ __forceinline__ uint4 act8(uint4 raw, bool silu) {
 template <int NP, bool ROT> constexpr size_t smem_bytes() {
     // q and k (rotated: in two terms), v; the state in two terms; rows as they arrive; the powers
     return (size_t)((ROT ? 4 : 2) * C * (NP + 8) + C * LDV + 2 * NP * LDV + C * (2 * NP + PT)) * sizeof(bf16) + (POW_N + 3) / 4 * 4 * sizeof(float);
-}
-
-__device__ __forceinline__ float2 unpack(uint32_t w) {
-    const __nv_bfloat162 h = *reinterpret_cast<const __nv_bfloat162*>(&w);
-    return make_float2(__low2float(h), __high2float(h));
 }
 
 // Eight pairs (u, v) of a row turned by their angles (turn: whether there are any), times `scale`, as two bf16 terms each.
@@ -106,7 +76,7 @@ __device__ __forceinline__ void turn8(const bf16* row, int cu, int cv, bool turn
     uint32_t uh[4], ul[4], vh[4], vl[4];
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-        const float2 x = unpack(uw[i]), y = unpack(vw[i]);
+        const float2 x = bf16_pair(uw[i]), y = bf16_pair(vw[i]);
         float2 p = x, q = y;
         if (turn) {
             p = make_float2(rope_first(x.x, y.x, c[2 * i], sn[2 * i]), rope_first(x.y, y.y, c[2 * i + 1], sn[2 * i + 1]));
@@ -393,9 +363,9 @@ __global__ void __launch_bounds__(NT, 1) decay_chunk_kernel(const Args a) {
                 for (int i = 0; i < 4; ++i) {          // registers 0, 1: tokens pc, pc + 1 of the sixteen; 2, 3: eight later
                     const int tok = sb * 16 + pc + (i >> 1) * 8;
                     const float g0 = tok < n ? pw[n - 1 - tok] : 0.f, g1 = tok + 1 < n ? pw[n - 2 - tok] : 0.f;
-                    float2 x = unpack(ka[i]);
+                    float2 x = bf16_pair(ka[i]);
                     if (ROT) {
-                        const float2 y = unpack(kl[i]);
+                        const float2 y = bf16_pair(kl[i]);
                         x = make_float2(x.x + y.x, x.y + y.y);
                     }
                     split2(g0 * x.x, g1 * x.y, ah[i], al[i]);

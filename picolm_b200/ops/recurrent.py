@@ -464,6 +464,16 @@ def diag_scan(a: torch.Tensor, x: torch.Tensor, y_raw: torch.Tensor, y_bias: Opt
     return out
 
 
+_head_chunk_bytes = {}
+
+
+def delta_head_chunk_supported(v: torch.Tensor, state: torch.Tensor, key_dim: int, value_dim: int) -> bool:
+    """Whether the delta rule with one decay a head can run prompts on the tensor cores: values in bfloat16, a key size
+    that is a multiple of 16 up to 128, a value size that is a multiple of 8."""
+    return (v.dtype == torch.bfloat16 and key_dim % 16 == 0 and key_dim <= 128 and value_dim % 8 == 0
+            and state.stride(0) % 2 == 0 and state.data_ptr() % 16 == 0)
+
+
 DELTA_CHUNK_FROM = 16      # tokens of a step's longest sequence from which the delta rule runs chunk by chunk
 
 
@@ -516,8 +526,8 @@ def delta_scan(qn: torch.Tensor, kn: torch.Tensor, qk: torch.Tensor, decay: torc
     value_dim] (a column slice will do); `state` float32 [slots, >= heads * key_dim * value_dim] with contiguous
     rows holds S as [heads, key_dim, value_dim] and is carried on.  Returns o, float32 [T, heads * value_dim].
     A step whose longest sequence brings `DELTA_CHUNK_FROM` tokens or more runs chunk by chunk (two kernels: what does
-    not depend on the state for all chunks side by side, then a walk over each sequence's chunks); shorter portions
-    and single tokens run token by token."""
+    not depend on the state for all chunks side by side, then a walk over each sequence's chunks; with one decay a head and
+    values in bfloat16 on the tensor cores, 64 tokens at a time); shorter portions and single tokens run token by token."""
     H, N, P = heads, key_dim, value_dim
     T = v.shape[0]
     if H % heads_per_group:
@@ -538,7 +548,21 @@ def delta_scan(qn: torch.Tensor, kn: torch.Tensor, qk: torch.Tensor, decay: torc
         raise KernelError("delta_scan: the state must be float32 with heads * key_dim * value_dim values a row")
     y = torch.empty((T, H * P), dtype=torch.float32, device=v.device)
     set_bounds("recurrent", n_seqs=step.n_seqs, device=v.device)
-    if step.max_new >= DELTA_CHUNK_FROM and not (step.is_decode and step.n_tokens == step.n_seqs):
+    prompts = step.max_new >= DELTA_CHUNK_FROM and not (step.is_decode and step.n_tokens == step.n_seqs)
+    if prompts and head_decay and delta_head_chunk_supported(v, state, N, P):
+        per = _head_chunk_bytes.get((N, P))
+        if per is None:
+            per = _head_chunk_bytes[N, P] = _fn("delta_chunk", "plm_delta_head_chunk_bytes")(N, P)
+        nbytes = (T // 64 + step.n_seqs + 1) * H * per
+        ws = torch.empty((nbytes,), dtype=torch.uint8, device=v.device)
+        _check(_fn("delta_chunk", "plm_delta_head_chunk_scan")(
+            _p(qn), _p(kn), _p(decay), _p(beta), _p(v), ldv, _p(state), lds, _p(y), _p(ws), _p(step.seq_start), _p(step.seq_slot),
+            step.n_seqs, int(step.max_new), H, N, P, heads_per_group, _stream()),
+            f"delta_head_chunk_scan T={T} H={H} N={N} P={P}", kernels=2,
+            nbytes=T * (8 * G * N + H * P * (4 + v.element_size())) + 2 * step.n_seqs * H * N * P * 4,
+            flops=2 * T * H * (3 * N * P + 64 // 2 * (2 * N + N + 2 * P)))
+        return y
+    if prompts:
         floats = delta_chunk_workspace(T, step.n_seqs, H, N)
         ws = torch.empty((floats,), dtype=torch.float32, device=v.device)
         _check(_fn("recurrent", "plm_delta_chunk_scan")(

@@ -143,9 +143,9 @@ def unit_attention(h, w, m, eps, get):
 
 
 # ------------------------------------------------------------------- delta rule
-def delta_rule(q, k, v, g, beta):
+def delta_rule(q, k, v, g, beta, with_state=False):
     """One head.  q, k [T, N], v [T, P], g, beta [T]: S <- g_t S; u = beta_t (v_t - S^T k_t); S <- S + k_t u^T;
-    o_t = S^T q_t.  Returns o [T, P]."""
+    o_t = S^T q_t.  Returns o [T, P] (and the last S)."""
     T, N = k.shape
     S = torch.zeros(N, v.shape[1], dtype=q.dtype)
     out = torch.zeros(T, v.shape[1], dtype=q.dtype)
@@ -154,7 +154,7 @@ def delta_rule(q, k, v, g, beta):
         u = beta[t] * (v[t] - S.T @ k[t])
         S = S + torch.outer(k[t], u)
         out[t] = S.T @ q[t]
-    return out
+    return (out, S) if with_state else out
 
 
 def fading_delta(h, w, m, eps, get):

@@ -230,15 +230,20 @@ def test_rotated_recurrence_refuses_what_it_cannot_do():
 
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("N,Pv,H,hpg", [(12, 20, 4, 2), (32, 64, 3, 3), (64, 40, 2, 1), (100, 128, 2, 2), (200, 24, 1, 1), (1, 5, 2, 1)])
+@pytest.mark.parametrize("N,Pv,H,hpg", [(12, 20, 4, 2), (32, 64, 3, 3), (64, 40, 2, 1), (100, 128, 2, 2), (200, 24, 1, 1), (1, 5, 2, 1),
+                                        (16, 8, 2, 2), (48, 72, 4, 2), (128, 136, 2, 1), (112, 64, 2, 2)])
 def test_delta_rule_with_one_decay_a_head(dtype, N, Pv, H, hpg):
-    """Unit queries and keys, decays and write strengths, and the recurrence chunk by chunk and token by token, from zero
-    and from a state; decays from next to 1 to next to 0."""
+    """Unit queries and keys, decays and write strengths, and the recurrence chunk by chunk (in bfloat16 on the tensor
+    cores where the sizes allow it) and token by token, from zero and from a state: outputs and states; decays from next to 1
+    to next to 0; neighbouring keys that are nearly the same."""
     from picolm_b200 import ops
     G = H // hpg
     lens, slots = [230, 1, 67], [3, 0, 1]
     g = torch.Generator().manual_seed(N + Pv)
     rows = [torch.randn(n, 2 * G * N + H * Pv + 2 * H + 8, generator=g).to(dtype) for n in lens]
+    for r in rows:                                         # a key like the one before, over a chunk's border too
+        for lo, hi in ((20, 26), (62, 67)):
+            r[lo:hi, 4 + G * N:4 + 2 * G * N] = r[lo:lo + 1, 4 + G * N:4 + 2 * G * N].clone()
     a_log = torch.linspace(-9.0, 1.5, H) if H > 1 else torch.tensor([-2.0])
     bias = torch.randn(H, generator=g)
 
@@ -249,7 +254,7 @@ def test_delta_rule_with_one_decay_a_head(dtype, N, Pv, H, hpg):
             o += n
         return out
 
-    want = []
+    want, states = [], []
     for r in rows:
         q, k, v, z, b = (t.double() for t in parts(r))
         n = len(r)
@@ -257,7 +262,9 @@ def test_delta_rule_with_one_decay_a_head(dtype, N, Pv, H, hpg):
         q = q / torch.sqrt((q * q).sum(-1, keepdim=True) + 1e-6) * N ** -0.5
         k = k / torch.sqrt((k * k).sum(-1, keepdim=True) + 1e-6)
         fade = torch.exp(-torch.exp(a_log.double()) * P.softplus(z + bias.double()))
-        want.append(torch.cat([P.delta_rule(q[:, h // hpg], k[:, h // hpg], v[:, h], fade[:, h], torch.sigmoid(b[:, h])) for h in range(H)], dim=1))
+        heads = [P.delta_rule(q[:, h // hpg], k[:, h // hpg], v[:, h], fade[:, h], torch.sigmoid(b[:, h]), with_state=True) for h in range(H)]
+        want.append(torch.cat([o for o, _ in heads], dim=1))
+        states.append(torch.stack([S for _, S in heads]).reshape(-1))
     state = torch.zeros(5, H * N * Pv + 4, device=DEV)
     for name, cuts in (("whole", [[(0, 230), (0, 1), (0, 67)]]),
                        ("cut", [[(0, 33), (0, 1), (0, 2)], [(33, 34), None, (2, 40)], [(34, 200), None, (40, 41)]]
@@ -276,8 +283,11 @@ def test_delta_rule_with_one_decay_a_head(dtype, N, Pv, H, hpg):
                 got[i][c[0]:c[1]] = y[o:o + c[1] - c[0]]
                 o += c[1] - c[0]
         for i in range(3):
+            tol = 2e-5 if dtype == torch.float32 or N % 16 or N > 128 or Pv % 8 else 1e-4
             err = (got[i].double() - want[i]).abs().max()
-            assert err < 2e-5 * max(1.0, want[i].abs().max()), f"{name}, sequence {i}: {err:.2e}"
+            assert err < tol * want[i].abs().max(), f"{name}, sequence {i}: {err:.2e}"
+            err = (state[slots[i], :H * N * Pv].cpu().double() - states[i]).abs().max()
+            assert err < tol * states[i].abs().max(), f"{name}, state of sequence {i}: {err:.2e}"
         assert (state[:, H * N * Pv:] == 0).all() and (state[[2, 4]] == 0).all()
 
 
