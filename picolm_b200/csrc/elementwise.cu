@@ -54,6 +54,7 @@ embed_norm_kernel(const int* tok, const Tw* table, const Tw* w, float* __restric
     if (id < 0 || id >= vocab) id = 0;   // ids are checked on the host; never read outside the table
     const Tw* row = table + (size_t)id * d;
     float ss = 0.f;
+#pragma unroll 8
     for (int i = threadIdx.x; i < d; i += NT) {
         const float v = to_f32<Tw>(row[i]);
         embed_row[i] = v;                           // (read back by the same thread)
@@ -62,6 +63,7 @@ embed_norm_kernel(const int* tok, const Tw* table, const Tw* w, float* __restric
     ss = block_sum<NT>(ss, red);
     const float scale = 1.0f / sqrtf(ss / (float)d + eps);
     float* o = out + (size_t)t * d;
+#pragma unroll 8
     for (int i = threadIdx.x; i < d; i += NT) o[i] = embed_row[i] * scale * to_f32<Tw>(w[i]);
 }
 
